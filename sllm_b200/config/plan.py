@@ -98,6 +98,9 @@ class ModelPlan:
     embedding_norm_name: str | None = None
     pass_vectors_name: str | None = None     # tensor [passes, hidden]: what a run with `reentry` = t adds to the stream
     passes: int = 0
+    token_table_name: str | None = None      # tensor [vocab, token_table_width]: vectors that belong to a token, for parts that ask for it
+    token_table_width: int = 0
+    logit_softcap: float | None = None       # logits become softcap tanh(logits / softcap)
 
     def validate(self) -> None:
         from .errors import ConfigError

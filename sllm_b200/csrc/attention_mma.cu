@@ -44,6 +44,9 @@ struct AttnParams {
   int max_pages, page_size, nq, nkv, window, num_splits, total_tokens;
   int block;     // > 0: a query sees only keys of its own block of this many positions (counted from 0)
   float scale_log2;              // scale * log2(e)
+  float cap_log2, cap_slope;     // > 0: capped scores, cap * log2(e) and 2 scale log2(e) / cap (see softcap_log2)
+  const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
+  int gate_ld;
   const float* sink;             // [nq] or null: exp(sink_h) joins the softmax's denominator (no key, no value, not scaled)
   // pooled blocks beside a window (pool > 0; needs window > 0 and num_splits == 1): a query at position i also sees entry b
   // of the pooled cache (same page geometry) for every b < (i - window + 1) / pool; these entries are walked as key tiles
@@ -272,7 +275,8 @@ __global__ void __launch_bounds__(AttThreads<DECODE>::value) attention_mma_kerne
         const int key = kbase + n * 8 + 2 * t4 + (c & 1);
         const int i = c >> 1;
         const bool seen = pooled_tile ? key < nb_r[i] : (key < hi_r[i] && key >= lo_r[i]);
-        const float v = seen ? s[n][c] * p.scale_log2 : -INFINITY;
+        const float sl = p.cap_log2 > 0.f ? softcap_log2(s[n][c], p.cap_slope, p.cap_log2) : s[n][c] * p.scale_log2;
+        const float v = seen ? sl : -INFINITY;
         s[n][c] = v;
         mx[i] = fmaxf(mx[i], v);
       }
@@ -333,7 +337,8 @@ __global__ void __launch_bounds__(AttThreads<DECODE>::value) attention_mma_kerne
       if (row >= rows_total) continue;
       const size_t orow = (size_t)(q0 + row / G) * p.nq + kvh * G + row % G;
       if (p.sink != nullptr && p.num_splits == 1) l_r[i] += exp2f(p.sink[kvh * G + row % G] * 1.4426950408889634f - m_r[i]);
-      const float inv = l_r[i] > 0.f ? (p.num_splits > 1 ? 1.f : p.out_scale) / l_r[i] : 0.f;
+      float inv = l_r[i] > 0.f ? (p.num_splits > 1 ? 1.f : p.out_scale) / l_r[i] : 0.f;
+      if (p.gate != nullptr && p.num_splits == 1) inv *= sigmoid_f32(p.gate[(size_t)(q0 + row / G) * p.gate_ld + kvh * G + row % G]);
       if (p.out_ld > 0 && p.num_splits == 1) {
         __nv_bfloat16* po = p.out + (size_t)(q0 + row / G) * p.out_ld + p.out_off + (size_t)(kvh * G + row % G) * p.vdim;
 #pragma unroll
@@ -392,7 +397,8 @@ __global__ void __launch_bounds__(AttThreads<DECODE>::value) attention_mma_kerne
         acc.x += v.x * f[w]; acc.y += v.y * f[w]; acc.z += v.z * f[w]; acc.w += v.w * f[w];
       }
       if (p.sink != nullptr && p.num_splits == 1) lt += exp2f(p.sink[kvh * G + row % G] * 1.4426950408889634f - mt);
-      const float inv = lt > 0.f ? (p.num_splits > 1 ? 1.f : p.out_scale) / lt : 0.f;
+      float inv = lt > 0.f ? (p.num_splits > 1 ? 1.f : p.out_scale) / lt : 0.f;
+      if (p.gate != nullptr && p.num_splits == 1) inv *= sigmoid_f32(p.gate[(size_t)(q0 + row / G) * p.gate_ld + kvh * G + row % G]);
       const size_t orow = (size_t)(q0 + row / G) * p.nq + kvh * G + row % G;
       if (p.out_ld > 0 && p.num_splits == 1) {
         if (d4 < p.vdim) {
@@ -416,7 +422,8 @@ template <int HD>
 __global__ void attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                              __nv_bfloat16* __restrict__ out, int rows, int num_splits,
                                              const int* __restrict__ tile_seq, const int* __restrict__ q_start, int nq,
-                                             const float* __restrict__ sink, int out_ld, int out_off, int vdim, float out_scale) {
+                                             const float* __restrict__ sink, int out_ld, int out_off, int vdim, float out_scale,
+                                             const float* __restrict__ gate, int gate_ld) {
   // One CTA per (tile, query head, token of the tile's request): the rows the decode form wrote and no others, so
   // that a step's other rows (a prompt portion's, the prefill form's) are neither read nor touched.  The step's
   // description is read before the wait for the kernel before.
@@ -434,7 +441,8 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o, const
     tot += l == -INFINITY ? 0.f : exp2f(l - mt);
   }
   if (sink != nullptr) tot += exp2f(sink[blockIdx.y] * 1.4426950408889634f - mt);
-  const float inv = tot > 0.f ? out_scale / tot : 0.f;
+  float inv = tot > 0.f ? out_scale / tot : 0.f;
+  if (gate != nullptr) inv *= sigmoid_f32(gate[(size_t)(q0 + (int)blockIdx.z) * gate_ld + blockIdx.y]);
   // (out_ld > 0: the row of token t and head h lies at out + t * out_ld + out_off + h * vdim and holds vdim channels)
   __nv_bfloat16* po = out_ld > 0 ? out + (size_t)(q0 + (int)blockIdx.z) * out_ld + out_off + (size_t)blockIdx.y * vdim : out + (size_t)row * HD;
   const int lim = out_ld > 0 ? vdim : HD;
@@ -470,7 +478,7 @@ static int launch_attention(const AttnParams& p, int tiles, cudaStream_t stream)
     const int G = p.nq / p.nkv;
     launch_kernel(attention_combine_kernel<HD>, dim3((unsigned)tiles, (unsigned)p.nq, (unsigned)(16 / G > 0 ? 16 / G : 1)), HD >= 128 ? 128 : 64, 0, stream,
                   (const float*)p.part_o, (const float*)p.part_lse, p.out, p.total_tokens * p.nq, p.num_splits, p.tile_seq,
-                  p.q_start, p.nq, p.sink, p.out_ld, p.out_off, p.vdim, p.out_scale);
+                  p.q_start, p.nq, p.sink, p.out_ld, p.out_off, p.vdim, p.out_scale, p.gate, p.gate_ld);
     rc = launch_status("attention_combine");
   }
   return rc;
@@ -490,7 +498,9 @@ SLLM_EXPORT int sllm_attention_mma(const void* q, const void* k_cache, const voi
                                    float* part_lse, const int* block_tables, int max_pages, const int* q_start,
                                    const int* ctx_len, const int* tile_seq, const int* tile_row0, int tiles,
                                    int decode, int num_splits, int total_tokens, int nq, int nkv, int hd,
-                                   int page_size, float scale, int window, int block, const float* sink, cudaStream_t stream) {
+                                   int page_size, float scale, int window, int block, const float* sink, float softcap, const float* gate,
+                                   int gate_ld, cudaStream_t stream) {
+  SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_mma: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_mma: bad head counts nq=%d nkv=%d", nq, nkv);
   SLLM_REQUIRE(sllm_attention_mma_supports(hd), "attention_mma: head_dim=%d is not one of 16, 32, 64, 128", hd);
   SLLM_REQUIRE(page_size > 0 && max_pages > 0 && tiles >= 0 && total_tokens >= 0, "attention_mma: bad sizes");
@@ -505,6 +515,8 @@ SLLM_EXPORT int sllm_attention_mma(const void* q, const void* k_cache, const voi
   p.num_splits = num_splits; p.total_tokens = total_tokens;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
+  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
+  p.gate = gate; p.gate_ld = gate_ld;
   p.pk_cache = p.pv_cache = nullptr; p.pool_tables = nullptr; p.pool_max_pages = p.pool = 0;
   p.out_ld = p.out_off = p.vdim = 0; p.out_scale = 1.f;
 #define DISPATCH(HD_)                                                             \
@@ -547,6 +559,7 @@ SLLM_EXPORT int sllm_attention_mma_pooled(const void* q, const void* k_cache, co
   p.num_splits = num_splits; p.total_tokens = total_tokens;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
+  p.cap_log2 = p.cap_slope = 0.f; p.gate = nullptr; p.gate_ld = 0;
   p.pk_cache = (const __nv_bfloat16*)pk_cache; p.pv_cache = (const __nv_bfloat16*)pv_cache; p.pool_tables = pool_tables;
   p.pool_max_pages = pool_max_pages; p.pool = pool;
   p.out_ld = out_ld; p.out_off = out_off; p.vdim = vdim; p.out_scale = out_scale;

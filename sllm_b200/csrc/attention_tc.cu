@@ -78,6 +78,9 @@ struct AttnTcParams {
   float* part_o;
   float* part_lse;
   const float* sink;             // [nq] or null: exp(sink_h) joins the softmax's denominator (no key, no value, not scaled)
+  float cap_log2, cap_slope;     // CAP: capped scores, cap * log2(e) and 2 scale log2(e) / cap (see softcap_log2)
+  const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
+  int gate_ld;
 };
 
 constexpr int TC_BM = 128, TC_BN = 64;
@@ -132,7 +135,8 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
   return d;
 }
 
-template <int HD, int RT>
+// CAP: a score becomes cap * tanh(score / cap) before the softmax
+template <int HD, int RT, bool CAP>
 __global__ void __launch_bounds__(TcLayout<HD, RT>::THREADS, RT == 1 ? 2 : 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                     const __grid_constant__ CUtensorMap run_k, const __grid_constant__ CUtensorMap run_v,
@@ -441,7 +445,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           mx = max3(mx, __uint_as_float(s0[i]), __uint_as_float(s1[i]));
         }
       }
-      mx *= p.scale_log2;
+      // (the cap's curve rises, so the maximum of the capped scores is the capped maximum; no key: -inf stays)
+      if constexpr (CAP) mx = mx == -INFINITY ? mx : softcap_log2(mx, p.cap_slope, p.cap_log2);
+      else mx *= p.scale_log2;
       const bool grow = mx > m_used + TC_RESCALE_STEP;      // also the first tile with a key (m_used = -inf)
       // Only a rescale of O waits for the product of the tile before it (O must not change under it).
       // The barrier is the one behind that product, s_free of its buffer: its phases go by every
@@ -472,6 +478,26 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
       uint32_t pk[32];                                      // column i: keys 2i (low half) and 2i+1
       float2 sums = make_float2(0.f, 0.f);                  // of the even and of the odd keys
+      if constexpr (CAP) {
+        // 2^(capped score - max) = 2^(cap - max - 2 cap / (2^(slope s) + 1)); the two reciprocals of a pair come from one
+        const bool edge = kbase + TC_BN > hi;
+        const float top = p.cap_log2 + neg_m, two_cap = -2.0f * p.cap_log2;
+        auto capped_pair = [&](uint32_t sa, uint32_t sb, int key) {
+          const float2 z = fma_x2(__uint_as_float(sa), __uint_as_float(sb), p.cap_slope, 0.f);
+          // (beyond 2^60 the quotient is nothing; the bound keeps the product of the two finite)
+          const float2 d = add_x2(make_float2(ex2(fminf(z.x, 60.f)), ex2(fminf(z.y, 60.f))), make_float2(1.f, 1.f));
+          const float rr = __fdividef(1.0f, d.x * d.y);
+          const float2 x = fma_x2(d.y * rr, d.x * rr, two_cap, top);
+          return make_float2(edge && key >= hi ? 0.f : ex2(x.x), edge && key + 1 >= hi ? 0.f : ex2(x.y));
+        };
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float2 e01 = capped_pair(s0[2 * i], s0[2 * i + 1], kbase + 2 * i), e23 = capped_pair(s1[2 * i], s1[2 * i + 1], kbase + 32 + 2 * i);
+          sums = add_x2(sums, add_x2(e01, e23));
+          pk[i] = pack2(e01.x, e01.y);
+          pk[16 + i] = pack2(e23.x, e23.y);
+        }
+      } else {
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const float2 x01 = fma_x2(__uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]), p.scale_log2, neg_m);
@@ -480,6 +506,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         sums = add_x2(sums, add_x2(e01, e23));
         pk[i] = pack2(e01.x, e01.y);
         pk[16 + i] = pack2(e23.x, e23.y);
+      }
       }
       l += sums.x + sums.y;
       tmem_st32(t_lane + b * TC_BN, pk);
@@ -499,7 +526,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     if (ok && my_tiles > 0) {
       tc_fence_after();
       if (p.sink != nullptr && p.num_splits == 1 && valid) l += exp2f(p.sink[kvh * G + row % G] * 1.4426950408889634f - m_used);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate != nullptr && p.num_splits == 1 && valid) inv *= sigmoid_f32(p.gate[(size_t)(q0 + row / G) * p.gate_ld + kvh * G + row % G]);
       __nv_bfloat16* po = nullptr;
       if (valid) po = p.out + orow * HD;
       float* pp = p.num_splits > 1 ? p.part_o + ((size_t)blockIdx.z * p.total_tokens * p.nq + orow) * HD : nullptr;
@@ -538,7 +566,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 template <int HD>
 __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                             __nv_bfloat16* __restrict__ out, int rows, int num_splits, int nq,
-                                            const float* __restrict__ sink) {
+                                            const float* __restrict__ sink, const float* __restrict__ gate, int gate_ld) {
   pdl_launch_dependents();       // a short kernel: the successor may be set up behind it
   pdl_wait();
   const int row = blockIdx.x;
@@ -551,7 +579,8 @@ __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, co
     tot += l == -INFINITY ? 0.f : exp2f(l - mt);
   }
   if (sink != nullptr) tot += exp2f(sink[row % nq] * 1.4426950408889634f - mt);
-  const float inv = tot > 0.f ? 1.f / tot : 0.f;
+  float inv = tot > 0.f ? 1.f / tot : 0.f;
+  if (gate != nullptr) inv *= sigmoid_f32(gate[(size_t)(row / nq) * gate_ld + row % nq]);
   for (int d = threadIdx.x; d < HD; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s) {
@@ -598,24 +627,24 @@ static bool tc_cache_map(const void* base, long long rows, int ps, int hd, CUten
   return true;
 }
 
-template <int HD, int RT>
+template <int HD, int RT, bool CAP>
 static int launch_tc(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& rk, const CUtensorMap& rv,
                      const AttnTcParams& p, int tiles, cudaStream_t stream) {
   constexpr int smem = TcLayout<HD, RT>::SMEM;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tc_kernel<HD, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attention_tc_kernel<HD, RT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
       set_error("attention_tc: cannot raise the shared memory limit");
       return SLLM_ERR_LAUNCH;
     }
     configured = true;
   }
   dim3 grid((unsigned)tiles * p.nkv, 1, p.num_splits);
-  launch_kernel(attention_tc_kernel<HD, RT>, grid, TcLayout<HD, RT>::THREADS, (size_t)smem, stream, mk, mv, rk, rv, p);
+  launch_kernel(attention_tc_kernel<HD, RT, CAP>, grid, TcLayout<HD, RT>::THREADS, (size_t)smem, stream, mk, mv, rk, rv, p);
   int rc = launch_status("attention_tc");
   if (rc != SLLM_OK || p.num_splits == 1) return rc;
   launch_kernel(attention_tc_combine_kernel<HD>, p.total_tokens * p.nq, HD >= 128 ? 128 : 64, 0, stream,
-                (const float*)p.part_o, (const float*)p.part_lse, p.out, p.total_tokens * p.nq, p.num_splits, p.nq, p.sink);
+                (const float*)p.part_o, (const float*)p.part_lse, p.out, p.total_tokens * p.nq, p.num_splits, p.nq, p.sink, p.gate, p.gate_ld);
   return launch_status("attention_tc_combine");
 }
 
@@ -641,7 +670,8 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
                                   const int* tile_seq, const int* tile_row0, int tiles, int row_tiles, int nq, int nkv,
                                   int hd, int page_size, float scale, int num_splits, int tiles_per_split, int total_tokens,
                                   float* part_o, float* part_lse, const int* seq_row, const int* page_shift, const float* sink,
-                                  int* status, cudaStream_t stream) {
+                                  float softcap, const float* gate, int gate_ld, int* status, cudaStream_t stream) {
+  SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_tc: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE((seq_row == nullptr) == (page_shift == nullptr), "attention_tc: parts of requests need both their row and their first page");
   SLLM_REQUIRE(row_tiles == 1 || row_tiles == 2, "attention_tc: row_tiles=%d must be 1 or 2", row_tiles);
   SLLM_REQUIRE(num_splits >= 1 && num_splits <= 65535 && tiles_per_split >= 1, "attention_tc: bad context split %d x %d",
@@ -672,7 +702,12 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
   p.num_splits = num_splits; p.tiles_per_split = num_splits == 1 ? (1 << 30) / TC_BN : tiles_per_split;
   p.total_tokens = total_tokens; p.part_o = part_o; p.part_lse = part_lse; p.seq_row = seq_row; p.page_shift = page_shift;
   p.sink = sink;
+  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
+  p.gate = gate; p.gate_ld = gate_ld;
+  SLLM_REQUIRE(softcap == 0.f || row_tiles == 1, "attention_tc: capped scores run in the form of one row tile a CTA");
+  if (softcap > 0.f)
+    return hd == 128 ? launch_tc<128, 1, true>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 1, true>(mk, mv, rk, rv, p, tiles, stream);
   if (row_tiles == 2)
-    return hd == 128 ? launch_tc<128, 2>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 2>(mk, mv, rk, rv, p, tiles, stream);
-  return hd == 128 ? launch_tc<128, 1>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 1>(mk, mv, rk, rv, p, tiles, stream);
+    return hd == 128 ? launch_tc<128, 2, false>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 2, false>(mk, mv, rk, rv, p, tiles, stream);
+  return hd == 128 ? launch_tc<128, 1, false>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 1, false>(mk, mv, rk, rv, p, tiles, stream);
 }

@@ -51,6 +51,9 @@ struct AttnTmaParams {
   int page_runs;                 // the run maps are valid: a tile of pages with consecutive ids is fetched as one box
   float scale_log2;
   const float* sink;             // [nq] or null: exp(sink_h) joins the softmax's denominator (no key, no value, not scaled)
+  float cap_log2, cap_slope;     // CAP: capped scores, cap * log2(e) and 2 scale log2(e) / cap (see softcap_log2)
+  const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
+  int gate_ld;
 };
 
 // Byte offset of the 16-byte chunk `chunk` (of the head's HD/8) of key row `row` within a stage's K or V.
@@ -62,7 +65,8 @@ __device__ __forceinline__ int swz(int row, int chunk) {
   return unit * 128 + (((chunk & 7) ^ (unit & 7)) << 4);
 }
 
-template <int HD>
+// CAP: a score becomes cap * tanh(score / cap) before the softmax
+template <int HD, bool CAP>
 __global__ void __launch_bounds__(TA_THREADS)
 attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const __grid_constant__ CUtensorMap run_k, const __grid_constant__ CUtensorMap run_v,
@@ -284,7 +288,8 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           for (int c = 0; c < 4; ++c) {
             const int key = kbase + n * 8 + 2 * t4 + (c & 1);
             const int i = c >> 1;
-            const float v = (key < hi_r[i] && key >= lo_r[i]) ? sc[n][c] * p.scale_log2 : -INFINITY;
+            const float sl = CAP ? softcap_log2(sc[n][c], p.cap_slope, p.cap_log2) : sc[n][c] * p.scale_log2;
+            const float v = (key < hi_r[i] && key >= lo_r[i]) ? sl : -INFINITY;
             sc[n][c] = v;
             mx[i] = fmaxf(mx[i], v);
           }
@@ -293,7 +298,7 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
-            sc[n][c] *= p.scale_log2;
+            sc[n][c] = CAP ? softcap_log2(sc[n][c], p.cap_slope, p.cap_log2) : sc[n][c] * p.scale_log2;
             mx[c >> 1] = fmaxf(mx[c >> 1], sc[n][c]);
           }
       }
@@ -384,7 +389,8 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           acc.x += v.x * f[w]; acc.y += v.y * f[w]; acc.z += v.z * f[w]; acc.w += v.w * f[w];
         }
         if (p.sink != nullptr && p.num_splits == 1) lt += exp2f(p.sink[kvh * G + row % G] * 1.4426950408889634f - mt);
-        const float inv = lt > 0.f ? 1.f / lt : 0.f;
+        float inv = lt > 0.f ? 1.f / lt : 0.f;
+        if (p.gate != nullptr && p.num_splits == 1) inv *= sigmoid_f32(p.gate[(size_t)(q0 + row / G) * p.gate_ld + kvh * G + row % G]);
         const size_t orow = (size_t)(q0 + row / G) * p.nq + kvh * G + row % G;
         if (p.num_splits > 1) {
           float* po = p.part_o + ((size_t)split * p.total_tokens * p.nq + orow) * HD + d4;
@@ -413,7 +419,7 @@ template <int HD>
 __global__ void attention_tma_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                              __nv_bfloat16* __restrict__ out, int rows, int num_splits,
                                              const int* __restrict__ tile_seq, const int* __restrict__ q_start, int nq,
-                                             const float* __restrict__ sink) {
+                                             const float* __restrict__ sink, const float* __restrict__ gate, int gate_ld) {
   // One CTA per (tile, query head, token of the tile's request): the rows the decode form wrote and no others, so
   // that a step's other rows (a prompt portion's, the prefill form's) are neither read nor touched.  The step's
   // description is read before the wait for the kernel before.  The ranges' weights are found by the threads side
@@ -456,7 +462,8 @@ __global__ void attention_tma_combine_kernel(const float* __restrict__ part_o, c
   tot = red[1][0];
   for (int i = 1; i < warps; ++i) tot += red[1][i];
   if (sink != nullptr) tot += exp2f(sink[blockIdx.y] * 1.4426950408889634f - mt);
-  const float inv = tot > 0.f ? 1.f / tot : 0.f;
+  float inv = tot > 0.f ? 1.f / tot : 0.f;
+  if (gate != nullptr) inv *= sigmoid_f32(gate[(size_t)(q0 + (int)blockIdx.z) * gate_ld + blockIdx.y]);
   // a warp takes every warps-th range, its lanes the row's columns in pairs; then the warps' sums are added
   float2 acc[VEC];
 #pragma unroll
@@ -524,20 +531,20 @@ constexpr size_t ta_smem(int hd) {
   return (size_t)TA_STAGES * 2 * TA_BN * hd * 2 + 16 * (hd + 8) * 2 + 2 * TA_STAGES * 8 + 16 + TA_BT_CACHE * 4 + 1024;
 }
 
-template <int HD>
+template <int HD, bool CAP>
 static int launch_ta(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& rk, const CUtensorMap& rv,
                      const AttnTmaParams& p, int tiles, cudaStream_t stream) {
   constexpr size_t smem = ta_smem(HD);
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tma_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attention_tma_decode_kernel<HD, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       set_error("attention_tma: cannot raise the shared memory limit");
       return SLLM_ERR_LAUNCH;
     }
     configured = true;
   }
   dim3 grid((unsigned)tiles * p.nkv, 1, p.num_splits);
-  launch_kernel(attention_tma_decode_kernel<HD>, grid, TA_THREADS, smem, stream, mk, mv, rk, rv, p);
+  launch_kernel(attention_tma_decode_kernel<HD, CAP>, grid, TA_THREADS, smem, stream, mk, mv, rk, rv, p);
   int rc = launch_status("attention_tma");
   if (rc != SLLM_OK) return rc;
   if (p.num_splits > 1) {
@@ -546,7 +553,7 @@ static int launch_ta(const CUtensorMap& mk, const CUtensorMap& mv, const CUtenso
     const int merge_warps = p.num_splits < TA_MERGE_WARPS ? (p.num_splits > 2 ? p.num_splits : 2) : TA_MERGE_WARPS;
     launch_kernel(attention_tma_combine_kernel<HD>, dim3((unsigned)tiles, (unsigned)p.nq, (unsigned)(16 / G > 0 ? 16 / G : 1)),
                   32 * merge_warps, 0, stream, (const float*)p.part_o, (const float*)p.part_lse, p.out, p.total_tokens * p.nq,
-                  p.num_splits, p.tile_seq, p.q_start, p.nq, p.sink);
+                  p.num_splits, p.tile_seq, p.q_start, p.nq, p.sink, p.gate, p.gate_ld);
     rc = launch_status("attention_tma_combine");
   }
   return rc;
@@ -576,7 +583,8 @@ SLLM_EXPORT int sllm_attention_tma_decode(const void* q, const void* k_cache, co
                                           int max_pages, const int* q_start, const int* ctx_len, const int* tile_seq,
                                           const int* tile_row0, int tiles, int num_splits, int total_tokens, int nq,
                                           int nkv, int hd, int page_size, float scale, int window, int block, const float* sink,
-                                          int* status, cudaStream_t stream) {
+                                          float softcap, const float* gate, int gate_ld, int* status, cudaStream_t stream) {
+  SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_tma: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_tma: bad head counts nq=%d nkv=%d", nq, nkv);
   SLLM_REQUIRE(sllm_attention_tma_supports(hd, page_size), "attention_tma: head_dim=%d page_size=%d not taken", hd, page_size);
   SLLM_REQUIRE(max_pages > 0 && tiles >= 0 && total_tokens >= 0 && num_pages > 0, "attention_tma: bad sizes");
@@ -603,6 +611,8 @@ SLLM_EXPORT int sllm_attention_tma_decode(const void* q, const void* k_cache, co
   p.status = status; p.max_pages = max_pages; p.page_size = page_size; p.nq = nq; p.nkv = nkv; p.window = window; p.block = block;
   p.num_splits = num_splits; p.total_tokens = total_tokens; p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
-
-  return hd == 128 ? launch_ta<128>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64>(mk, mv, rk, rv, p, tiles, stream);
+  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
+  p.gate = gate; p.gate_ld = gate_ld;
+  if (softcap > 0.f) return hd == 128 ? launch_ta<128, true>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, true>(mk, mv, rk, rv, p, tiles, stream);
+  return hd == 128 ? launch_ta<128, false>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, false>(mk, mv, rk, rv, p, tiles, stream);
 }

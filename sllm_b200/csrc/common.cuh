@@ -30,6 +30,14 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
   return __float2bfloat16_rn(v);   // round to nearest even, as the reference's to_bf16 does
 }
 
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// cap * tanh(score / cap) in the log2 domain, from the raw dot product: tanh(y) = 1 - 2 / (e^(2y) + 1), so the result is
+// cap_log2 - 2 cap_log2 / (2^(raw * slope) + 1) with slope = 2 scale log2(e) / cap.  Its error is absolute, about 2^-22 of the cap.
+__device__ __forceinline__ float softcap_log2(float raw, float slope, float cap_log2) {
+  return cap_log2 - __fdividef(2.0f * cap_log2, exp2f(raw * slope) + 1.0f);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -55,6 +63,28 @@ __device__ __forceinline__ float block_sum(float v, float* red /* >= 33 floats *
   }
   __syncthreads();
   return red[32];
+}
+
+// ---- activations a product's epilogue (or the kernel behind a product) applies to a plain, ungated result ----------------
+#define SLLM_ACT_NONE 0
+#define SLLM_ACT_RELU2 1       // max(v, 0)^2
+#define SLLM_ACT_TOKEN 2       // gelu_tanh(v) times the token's own entry of a table
+
+// For SLLM_ACT_TOKEN: column n of row m is multiplied by table[ids[m]][off + n] (rows of `ld`, V of them; ids outside are
+// clamped, the host validates them).
+struct TokenTable {
+  const void* table = nullptr;     // bfloat16 in the bfloat16 products, the stored type elsewhere
+  const int* ids = nullptr;
+  int off = 0, ld = 0, V = 0;
+};
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float relu2_f32(float v) { v = fmaxf(v, 0.f); return v * v; }
+__device__ __forceinline__ size_t token_row(const TokenTable& t, int m) {
+  int id = t.ids[m];
+  id = id < 0 ? 0 : (id >= t.V ? t.V - 1 : id);
+  return (size_t)id * t.ld + t.off;
 }
 
 void set_error(const char* msg);   // remembers the text for sllm_last_error()

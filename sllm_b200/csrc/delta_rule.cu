@@ -34,6 +34,9 @@
 //       through silu first: mode 2's walk with d = decay_h on every row.
 //   linear attention whose forget gate also writes (mode 4):  S <- diag(f) S + (1 - f) v^T;  o = S^T silu(q)  with
 //       f = lower + (1 - lower) sigmoid(z + bias) per key channel: mode 2's walk with d = f and k = 1 - f.
+//   retention (an instance of its own, ROT):  S <- decay_h S + k v^T;  o = S^T q  with q and k rotated by position over their
+//       first `rot` channels (channel i with i + rot/2, cos and sin from a table) and k then times k_scale: the loader warps
+//       rotate, the walk reads one decay for the whole head.
 //
 // A second kernel finishes the mixer's output: each head's o over its root mean square, times a gain,
 // times sigmoid(gate logit), in the compute dtype.
@@ -44,6 +47,7 @@ namespace sllm {
 constexpr int DR_COMPUTE = 128;   // threads that walk the tokens (as many again prepare the next chunk)
 constexpr int DR_THREADS = 2 * DR_COMPUTE;
 constexpr int DR_MAX_CHUNK = 16;
+constexpr int DR_RETENTION = 5;
 
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
 
@@ -63,12 +67,17 @@ struct DeltaParams {
   const float* a_log;      // mode 1: [H]
   const float* dt_bias;    // mode 1: [H]
   float r_scale, inv_tau;  // the read-out's factor; mode 2: 1 / tau
+  // retention: the head's decay is a_log[h]
+  const int* positions = nullptr;      // [T]
+  const float* table = nullptr;        // [max_pos][2][rot / 2], cos then sin
+  int rot = 0, max_pos = 0;
+  float k_scale = 1.f;
 };
 
 // RPT: rows of a column per lane (dk <= 8 * RPT = DKP, the padded key size).
 constexpr int DR_SPLIT = 8;
 
-template <int RPT, int CB>
+template <int RPT, int CB, bool ROT>
 __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParams p) {
   constexpr int SPLIT = DR_SPLIT, COLS = DR_COMPUTE / SPLIT * CB, DKP = RPT * SPLIT, PER_LANE = (DKP + 31) / 32;
   constexpr int VPL = (COLS + 31) / 32;       // values of v a loader lane brings
@@ -81,6 +90,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
   const int tid = threadIdx.x, lane = tid & 31;
   const bool loader = tid >= DR_COMPUTE;
   const int nchunks = (t_end - t_begin + chunk - 1) / chunk;
+  const float head_decay = ROT ? __ldg(p.a_log + h) : 0.f;
 
   // a loader warp prepares token after token of chunk c: rows of u, d, a*u, k, r (zeros beyond dk) and v's slice
   auto prepare = [&](int c) {
@@ -92,6 +102,54 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
     constexpr int TPW = DR_MAX_CHUNK / (DR_COMPUTE / 32);       // tokens of a chunk per loader warp
     const int lw = (tid - DR_COMPUTE) >> 5;
     float k[TPW][PER_LANE], a[TPW][PER_LANE], d[TPW][PER_LANE], r[TPW][PER_LANE], v[TPW][VPL];
+    if constexpr (ROT) {
+      float kp[TPW][PER_LANE], rp[TPW][PER_LANE], cs[TPW][PER_LANE], sn[TPW][PER_LANE];      // the partners of k and r, and the angle
+      const int half = p.rot >> 1;
+#pragma unroll
+      for (int q = 0; q < TPW; ++q) {
+        const int tt = lw + q * (DR_COMPUTE / 32);
+        const bool tok = tt < nt;
+        const int t = t0 + (tok ? tt : 0);
+        const float* row = p.proj + (size_t)t * p.ld;
+        int pos = p.rot > 0 ? p.positions[t] : 0;
+        pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+        const float* tab = p.table + (size_t)pos * p.rot;
+#pragma unroll
+        for (int m = 0; m < PER_LANE; ++m) {
+          const int i = lane + 32 * m;
+          const bool in = tok && i < dk, turned = in && i < p.rot;
+          const int j = i < half ? i + half : i - half, a_i = i < half ? i : i - half;
+          k[q][m] = in ? __ldg(row + p.off_k + h * dk + i) : 0.f;
+          r[q][m] = in ? __ldg(row + p.off_r + h * dk + i) : 0.f;
+          kp[q][m] = turned ? __ldg(row + p.off_k + h * dk + j) : 0.f;
+          rp[q][m] = turned ? __ldg(row + p.off_r + h * dk + j) : 0.f;
+          cs[q][m] = turned ? __ldg(tab + a_i) : 1.f;
+          sn[q][m] = turned ? (i < half ? -__ldg(tab + half + a_i) : __ldg(tab + half + a_i)) : 0.f;
+        }
+#pragma unroll
+        for (int m = 0; m < VPL; ++m) {
+          const int j = c0 + lane + 32 * m;
+          v[q][m] = (tok && lane + 32 * m < COLS && j < dv) ? __ldg(row + p.off_v + h * dv + j) : 0.f;
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < TPW; ++q) {
+        const int tt = lw + q * (DR_COMPUTE / 32);
+        if (tt >= nt) break;
+#pragma unroll
+        for (int m = 0; m < PER_LANE; ++m) {
+          const int i = lane + 32 * m;
+          if (i < DKP) {
+            s_k[tt * DKP + i] = fmaf(k[q][m], cs[q][m], kp[q][m] * sn[q][m]) * p.k_scale;
+            s_r[tt * DKP + i] = fmaf(r[q][m], cs[q][m], rp[q][m] * sn[q][m]);
+          }
+        }
+#pragma unroll
+        for (int m = 0; m < VPL; ++m)
+          if (lane + 32 * m < COLS) s_v[tt * COLS + lane + 32 * m] = v[q][m];
+      }
+      return;
+    }
     // every load of the warp's tokens first, then the arithmetic: the loads of all of them are in flight together
 #pragma unroll
     for (int q = 0; q < TPW; ++q) {
@@ -252,7 +310,19 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
         }
 #pragma unroll
         for (int cc = 0; cc < CB; ++cc) us[cc] = ut[cc] = o[cc] = o2[cc] = 0.f;
-        if (p.mode == 0) {
+        if constexpr (ROT) {
+#pragma unroll
+          for (int n = 0; n < RPT; n += 2) {
+            const float ka = k[n * SPLIT], kb = k[(n + 1) * SPLIT], ra = r[n * SPLIT], rb = r[(n + 1) * SPLIT];
+#pragma unroll
+            for (int cc = 0; cc < CB; ++cc) {
+              s[n][cc] = fmaf(ka, vv[cc], head_decay * s[n][cc]);
+              s[n + 1][cc] = fmaf(kb, vv[cc], head_decay * s[n + 1][cc]);
+              o[cc] = fmaf(s[n][cc], ra, o[cc]);
+              o2[cc] = fmaf(s[n + 1][cc], rb, o2[cc]);
+            }
+          }
+        } else if (p.mode == 0) {
 #pragma unroll
           for (int n = 0; n < RPT; n += 2) {
             const float ua = u[n * SPLIT], ub = u[(n + 1) * SPLIT];
@@ -371,7 +441,8 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
 }
 
 // out[t, h*dv + j] = o[t, h, j] / sqrt(mean_j(o[t, h, :]^2) + eps) * gain[h*dv + j] * act(gate[t, h*dv + j]), act the sigmoid
-// (gate_act 0) or z * sigmoid(z) (gate_act 1), or no gate at all (gate_act 2: `proj` is not read); a warp per (t, h).
+// (gate_act 0) or z * sigmoid(z) (gate_act 1), or no gate at all (gate_act 2: `proj` is not read); `gain` may be null (ones);
+// a warp per (t, h).
 template <typename TO>
 __global__ void delta_out_kernel(const float* __restrict__ o, const float* __restrict__ gain, const float* __restrict__ proj,
                                  int ld, int off_g, float eps, TO* __restrict__ out, int rows, int H, int dv, int gate_act,
@@ -390,7 +461,7 @@ __global__ void delta_out_kernel(const float* __restrict__ o, const float* __res
   const float* g = proj + (size_t)t * ld + off_g + h * dv;
   for (int j = lane; j < dv; j += 32) {
     const float gate = gate_act == 2 ? 1.0f : (gate_act == 1 ? g[j] * sigmoidf_(g[j]) : sigmoidf_(g[j]));
-    out[(size_t)t * out_ld + out_off + h * dv + j] = from_f32<TO>(x[j] * inv * gain[h * dv + j] * gate);
+    out[(size_t)t * out_ld + out_off + h * dv + j] = from_f32<TO>(x[j] * inv * (gain != nullptr ? gain[h * dv + j] : 1.0f) * gate);
   }
 }
 
@@ -412,7 +483,7 @@ delta_out_wide_kernel(const float* __restrict__ o, const float* __restrict__ gai
   const float* g = proj + (size_t)t * ld + off_g + h * dv;
   for (int j = threadIdx.x; j < dv; j += blockDim.x) {
     const float gate = gate_act == 2 ? 1.0f : (gate_act == 1 ? g[j] * sigmoidf_(g[j]) : sigmoidf_(g[j]));
-    out[(size_t)t * out_ld + out_off + h * dv + j] = from_f32<TO>(x[j] * inv * gain[h * dv + j] * gate);
+    out[(size_t)t * out_ld + out_off + h * dv + j] = from_f32<TO>(x[j] * inv * (gain != nullptr ? gain[h * dv + j] : 1.0f) * gate);
   }
 }
 
@@ -422,7 +493,7 @@ using namespace sllm;
 
 SLLM_EXPORT int sllm_delta_rule_supports(int dk, int dv) { return dk >= 1 && dk <= 256 && dv >= 1 && dv <= 65535 * 16; }
 
-template <int RPT, int CB>
+template <int RPT, int CB, bool ROT>
 static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   constexpr int DKP = RPT * DR_SPLIT, DR_COLS = DR_COMPUTE / DR_SPLIT * CB;
   const size_t per_token = (size_t)(5 * DKP + DR_COLS) * sizeof(float);
@@ -433,7 +504,7 @@ static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   const size_t smem = 2 * per_token * chunk;
   static size_t allowed = 48 * 1024;          // (per instantiation: what the kernel has been told it may use)
   if (smem > allowed) {
-    if (cudaFuncSetAttribute(delta_rule_kernel<RPT, CB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(delta_rule_kernel<RPT, CB, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       cudaGetLastError();
       set_error("delta_rule: the kernel's shared memory could not be raised");
       return SLLM_ERR_LAUNCH;
@@ -441,7 +512,7 @@ static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
     allowed = smem;
   }
   const dim3 grid((unsigned)S, (unsigned)p.H, (unsigned)((p.dv + DR_COLS - 1) / DR_COLS));
-  launch_kernel(delta_rule_kernel<RPT, CB>, grid, DR_THREADS, smem, stream, p);
+  launch_kernel(delta_rule_kernel<RPT, CB, ROT>, grid, DR_THREADS, smem, stream, p);
   return launch_status("delta_rule");
 }
 
@@ -469,7 +540,9 @@ static int dispatch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   const int dk = p.dk, dv = p.dv;
   // enough (request, head, 64 columns) for every SM: four columns a lane; else one, in four times the CTAs
   const bool wide = (long)S * p.H * ((dv + 63) / 64) >= (long)num_sms();
-#define SLLM_DR(RPT_) return wide ? launch_delta_rule<RPT_, 4>(p, S, stream) : launch_delta_rule<RPT_, 1>(p, S, stream)
+#define SLLM_DR(RPT_)                                                                                                         \
+  return p.mode == DR_RETENTION ? (wide ? launch_delta_rule<RPT_, 4, true>(p, S, stream) : launch_delta_rule<RPT_, 1, true>(p, S, stream)) \
+                                : (wide ? launch_delta_rule<RPT_, 4, false>(p, S, stream) : launch_delta_rule<RPT_, 1, false>(p, S, stream))
   if (dk <= 16) SLLM_DR(2);
   if (dk <= 32) SLLM_DR(4);
   if (dk <= 64) SLLM_DR(8);
@@ -550,6 +623,28 @@ SLLM_EXPORT int sllm_forget_gate_attention(const float* proj, int ld, int off_q,
   p.chunk = 1; p.max_q = max_q;
   p.mode = 4; p.hdiv = 1; p.gates = nullptr; p.ldg = p.off_b = p.off_dt = 0; p.a_log = lower; p.dt_bias = nullptr;
   p.r_scale = 1.f; p.inv_tau = 1.f;
+  return dispatch_delta_rule(p, S, stream);
+}
+
+// Retention (a fixed decay per head, `decay` [H]; q and k rotated by position, k times k_scale) over q | k | v columns of
+// `proj` [T, ld]; rot == 0: no rotation, positions and table unused.
+SLLM_EXPORT int sllm_retention(const float* proj, int ld, int off_q, int off_k, int off_v, const float* decay, const int* positions,
+                               const float* table, int rot, int max_pos, float k_scale, float* state, const int* q_start,
+                               const int* state_slots, float* out, int S, int H, int dk, int dv, int max_q, cudaStream_t stream) {
+  SLLM_REQUIRE(S >= 0 && H > 0 && H <= 65535, "retention: bad sizes S=%d H=%d", S, H);
+  SLLM_REQUIRE(sllm_delta_rule_supports(dk, dv), "retention: a head of %d key and %d value channels is outside 1..256 keys", dk, dv);
+  SLLM_REQUIRE(off_q >= 0 && off_k >= 0 && off_v >= 0 && off_q + H * dk <= ld && off_k + H * dk <= ld && off_v + H * dv <= ld,
+               "retention: columns outside the product's %d", ld);
+  SLLM_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dk && (rot == 0 || (positions && table && max_pos > 0)),
+               "retention: %d rotated channels of %d need an even number, positions and a table", rot, dk);
+  if (S == 0) return SLLM_OK;
+  DeltaParams p;
+  p.proj = proj; p.decay = proj; p.a_bias = nullptr; p.state = state; p.q_start = q_start; p.state_slots = state_slots;
+  p.out = out; p.ld = ld; p.off_r = off_q; p.off_k = off_k; p.off_v = off_v; p.off_a = 0; p.H = H; p.dk = dk; p.dv = dv;
+  p.chunk = 1; p.max_q = max_q;
+  p.mode = DR_RETENTION; p.hdiv = 1; p.gates = nullptr; p.ldg = p.off_b = p.off_dt = 0; p.a_log = decay; p.dt_bias = nullptr;
+  p.r_scale = 1.f; p.inv_tau = 1.f;
+  p.positions = positions; p.table = table; p.rot = rot; p.max_pos = max_pos > 0 ? max_pos : 1; p.k_scale = k_scale;
   return dispatch_delta_rule(p, S, stream);
 }
 

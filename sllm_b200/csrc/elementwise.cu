@@ -366,6 +366,47 @@ __global__ void rope_kv_write_vec_kernel(const TI* __restrict__ qkv, const float
   }
 }
 
+// ---------------------------------------------------------------------------
+// x[i] = cap * tanh(x[i] / cap), in place (a model's capped logits)
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, size_t n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t step = (size_t)gridDim.x * blockDim.x;
+  size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if ((reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+    for (; i < n / 4; i += step) {
+      float4 v = reinterpret_cast<float4*>(x)[i];
+      v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+      reinterpret_cast<float4*>(x)[i] = v;
+    }
+    i = n / 4 * 4 + (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  }
+  for (; i < n; i += step) x[i] = cap * tanhf(x[i] / cap);
+}
+
+// ---------------------------------------------------------------------------
+// out[t, n] = max(x, 0)^2, or gelu_tanh(x) * table[ids[t], off + n]: behind products whose kernel has no such epilogue
+// ---------------------------------------------------------------------------
+template <typename TI, typename TT, typename TO>
+__global__ void __launch_bounds__(256)
+plain_act_kernel(const TI* __restrict__ x, TO* __restrict__ out, int T, int N, int act, const TokenTable token) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t total = (size_t)T * N;
+  for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
+    const float v = to_f32(x[e]);
+    float y;
+    if (act == SLLM_ACT_RELU2) {
+      y = relu2_f32(v);
+    } else {
+      const int t = (int)(e / N), n = (int)(e % N);
+      y = gelu_tanh_f32(v) * to_f32(reinterpret_cast<const TT*>(token.table)[token_row(token, t) + n]);
+    }
+    out[e] = from_f32<TO>(y);
+  }
+}
+
 }  // namespace sllm
 
 using namespace sllm;
@@ -494,4 +535,32 @@ SLLM_EXPORT int sllm_rope_kv_write(const void* qkv, int in_dtype, int parts, siz
   else SLLM_REQUIRE(false, "rope_kv_write: unsupported dtypes %d -> %d", in_dtype, cache_dtype);
 #undef LAUNCH
   return launch_status("rope_kv_write");
+}
+
+SLLM_EXPORT int sllm_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  SLLM_REQUIRE(n >= 0 && cap > 0.f, "softcap: %lld values, cap %f", n, cap);
+  if (n == 0) return SLLM_OK;
+  const long long blocks = (n / 4 + 255) / 256 + 1;
+  launch_kernel(softcap_kernel, (unsigned)(blocks > 2048 ? 2048 : blocks), 256, 0, stream, x, (size_t)n, cap);
+  return launch_status("softcap");
+}
+
+// act: SLLM_ACT_RELU2, or SLLM_ACT_TOKEN with a table of the output's dtype
+SLLM_EXPORT int sllm_plain_act(const void* x, int in_dtype, void* out, int out_dtype, int T, int N, int act, const void* token_table,
+                               const int* token_ids, int token_off, int token_ld, int token_rows, cudaStream_t stream) {
+  SLLM_REQUIRE(T >= 0 && N > 0 && (act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN), "plain_act: bad sizes T=%d N=%d act=%d", T, N, act);
+  SLLM_REQUIRE(act != SLLM_ACT_TOKEN || (token_table && token_ids && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld),
+               "plain_act: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
+  if (T == 0) return SLLM_OK;
+  TokenTable tt;
+  tt.table = token_table; tt.ids = token_ids; tt.off = token_off; tt.ld = token_ld; tt.V = token_rows;
+  const size_t total = (size_t)T * N;
+  const unsigned blocks = (unsigned)((total + 255) / 256 > 8192 ? 8192 : (total + 255) / 256);
+#define PA(TI_, TO_) launch_kernel(plain_act_kernel<TI_, TO_, TO_>, blocks, 256, 0, stream, (const TI_*)x, (TO_*)out, T, N, act, tt)
+  if (in_dtype == SLLM_F32 && out_dtype == SLLM_F32) PA(float, float);
+  else if (in_dtype == SLLM_F32 && out_dtype == SLLM_BF16) PA(float, __nv_bfloat16);
+  else if (in_dtype == SLLM_BF16 && out_dtype == SLLM_BF16) PA(__nv_bfloat16, __nv_bfloat16);
+  else SLLM_REQUIRE(false, "plain_act: unsupported dtypes %d -> %d", in_dtype, out_dtype);
+#undef PA
+  return launch_status("plain_act");
 }

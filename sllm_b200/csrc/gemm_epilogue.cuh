@@ -11,6 +11,8 @@ namespace sllm {
 #define TG_EPI_BF16 1
 #define TG_EPI_SILU 2
 #define TG_EPI_GELU 4      // like TG_EPI_SILU with gelu_tanh(gate + bias) * (up + bias), the bias interleaved like the columns
+#define TG_EPI_RELU2 5     // bfloat16 out[M, N] = max(product, 0)^2 (no bias)
+#define TG_EPI_TOKEN 6     // bfloat16 out[M, N] = gelu_tanh(product) * the token's entry of a table (no bias); see TgExtra::token
 #define TG_EPI_RESID 3     // residual[M, N] (float32) += the product (+ bias), in place; see TgExtra
 
 // What an epilogue may do beyond its store, for the RMSNorm that a prompt portion's products take apart
@@ -30,6 +32,7 @@ struct TgExtra {
   __nv_bfloat16* xg = nullptr;
   float* ssq_out = nullptr;
   int stride_out = 0;
+  TokenTable token;            // TG_EPI_TOKEN
 };
 
 // the factor of row m (1 where nothing is owed); the partial sums are added in index order
@@ -43,6 +46,21 @@ __device__ __forceinline__ float tg_row_scale(const TgExtra& e, int m, int M) {
 __device__ __forceinline__ void tg_scale(uint32_t (&r)[32], float s) {
 #pragma unroll
   for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * s);
+}
+
+// what TG_EPI_RELU2 and TG_EPI_TOKEN do to the columns n .. n + 31 of row m before the bfloat16 store
+template <int EPI>
+__device__ __forceinline__ void tg_activate(uint32_t (&r)[32], int m, int n, int M, int N, const TgExtra& e) {
+  if constexpr (EPI == TG_EPI_RELU2) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(relu2_f32(__uint_as_float(r[i])));
+  } else if constexpr (EPI == TG_EPI_TOKEN) {
+    if (m >= M) return;
+    const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(e.token.table) + token_row(e.token, m) + n;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      r[i] = __float_as_uint(n + i < N ? gelu_tanh_f32(__uint_as_float(r[i])) * __bfloat162float(row[i]) : 0.f);
+  }
 }
 
 // The epilogue warps run one to a scheduler with nothing to hide a dependent instruction behind, so what they
@@ -138,7 +156,7 @@ __device__ __forceinline__ void tg_store_chunk(const uint32_t (&r)[32], int m, i
 // lane hands it to the TMA unit, which writes whole lines and clips what lies outside the matrix.
 // A box is 32 float32, 64 bfloat16 or (SiLU form) 128 accumulator columns wide.
 template <int EPI> struct TgBox {
-  static constexpr int ACC_COLS = (EPI == TG_EPI_F32 || EPI == TG_EPI_RESID) ? 32 : (EPI == TG_EPI_BF16 ? 64 : 128);   // accumulator columns a box covers
+  static constexpr int ACC_COLS = (EPI == TG_EPI_F32 || EPI == TG_EPI_RESID) ? 32 : (tg_gated(EPI) ? 128 : 64);   // accumulator columns a box covers
   static constexpr int ELEM = (EPI == TG_EPI_F32 || EPI == TG_EPI_RESID) ? 4 : 2;
 };
 

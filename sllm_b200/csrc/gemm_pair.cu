@@ -256,6 +256,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
         }
         if (m >= M) continue;
         if (extra.ssq_in != nullptr) tg_scale(r, row_scale);
+        tg_activate<EPI>(r, m, n0 + c0, M, N, extra);
         if constexpr (EPI == TG_EPI_F32)
           tg_store_chunk<EPI>(r, m, n0 + c0, N, split == 0 ? bias : nullptr, reinterpret_cast<float*>(out) + (size_t)split * M * N);
         else if constexpr (EPI != TG_EPI_RESID)
@@ -476,6 +477,7 @@ gemm_pair_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
             tmem_ld32(tmem_base + ((uint32_t)(quarter * 32) << 16) + h * 256 + c0 + 32 * sub, r);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (extra.ssq_in != nullptr) tg_scale(r, row_scale);
+            tg_activate<EPI>(r, m, n + 32 * sub, M, N, extra);
             if constexpr (EPI == TG_EPI_RESID) {
               if (n + 32 * sub < N) tg_resid_box(r, box, lane, row0, n + 32 * sub, M, N, bias, extra, sq);      // (warp-uniform)
             } else {
@@ -595,7 +597,8 @@ SLLM_EXPORT int sllm_gemm_pair_supports(int M, int N, int K) {
 
 // The same product and epilogues as sllm_gemm_tcgen05 (0: float32 out[M, N] (+bias); 1: bfloat16; 2: bfloat16
 // out[M, N/2] = silu(gate) * up for W rows interleaved in blocks of 8), by pairs of CTAs on 256 x 256 tiles, and
-// 3: residual[M, N] (float32) += the product (+bias) in place (`out` is ignored).
+// 3: residual[M, N] (float32) += the product (+bias) in place (`out` is ignored); 4: 2 with the tanh form of GELU; 5: bfloat16
+// max(product, 0)^2; 6: bfloat16 gelu_tanh(product) times token_table[token_ids[m]][token_off + n].
 // `wide`: 0 tiles of 256 x 256; 1 tiles of 256 x 512 (for matrices with few rows of W); 2 tiles of 256 x 128 (for results
 // with few tiles); 448, 384, 320: tiles of 256 x that many columns (epilogues 0 and 3; where they fill the pairs of SMs
 // better than 512-wide ones).
@@ -631,12 +634,21 @@ SLLM_EXPORT int sllm_gemm_pair_splits(int K, int want) {
 SLLM_EXPORT int sllm_gemm_pair(const void* A, const void* W, const float* bias, void* out, int M, int N, int K,
                                int epilogue, int wide, int want_splits, const float* ssq_in, int parts_in, int stride_in, float eps_in,
                                int width_in, float* residual, const float* gain, void* xg_out, float* ssq_out, int stride_out,
+                               const void* token_table, const int* token_ids, int token_off, int token_ld, int token_rows,
                                int* status, cudaStream_t stream) {
   SLLM_REQUIRE(sllm_gemm_pair_supports(M, N, K), "gemm_pair: sizes M=%d N=%d K=%d (K must be a multiple of 8)", M, N, K);
   SLLM_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_pair: operands must be 16-byte aligned");
   SLLM_REQUIRE(status != nullptr, "gemm_pair: a status word is required");
   SLLM_REQUIRE(!tg_gated(epilogue) || N % 16 == 0, "gemm_pair: the gated epilogues need N %% 16 == 0");
   TgExtra extra;
+  SLLM_REQUIRE((epilogue != TG_EPI_RELU2 && epilogue != TG_EPI_TOKEN) || bias == nullptr, "gemm_pair: epilogue %d takes no bias", epilogue);
+  if (epilogue == TG_EPI_TOKEN) {
+    SLLM_REQUIRE(token_table != nullptr && token_ids != nullptr && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld,
+                 "gemm_pair: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
+    SLLM_REQUIRE(wide == 0 || wide == 2, "gemm_pair: the tokens' table goes with tiles of 256 or 128 columns");
+    extra.token.table = token_table; extra.token.ids = token_ids; extra.token.off = token_off; extra.token.ld = token_ld;
+    extra.token.V = token_rows;
+  }
   if (ssq_in != nullptr) {
     SLLM_REQUIRE(parts_in >= 1 && stride_in >= parts_in && width_in >= 1, "gemm_pair: a table of %d partial sums (row stride %d) over width %d",
                  parts_in, stride_in, width_in);
@@ -685,6 +697,10 @@ SLLM_EXPORT int sllm_gemm_pair(const void* A, const void* W, const float* bias, 
     case TG_EPI_BF16: GO(TG_EPI_BF16)
     case TG_EPI_SILU: GO(TG_EPI_SILU)
     case TG_EPI_GELU: GO(TG_EPI_GELU)
+    case TG_EPI_RELU2: GO(TG_EPI_RELU2)
+    case TG_EPI_TOKEN:
+      return wide == 2 ? launch_tp<TG_EPI_TOKEN, 128>(ma, mw, bias, out, M, N, K, status, stream, extra, ksplits, kb_per_split)
+                       : launch_tp<TG_EPI_TOKEN, 256>(ma, mw, bias, out, M, N, K, status, stream, extra, ksplits, kb_per_split);
     case TG_EPI_RESID: GO(TG_EPI_RESID)
   }
 #undef GO

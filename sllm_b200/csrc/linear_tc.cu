@@ -46,6 +46,7 @@ struct LtCfg {
 #define LT_EPI_F32 0
 #define LT_EPI_BF16 1
 #define LT_EPI_SILU 2
+#define LT_EPI_RELU2 3     // bfloat16 max(product, 0)^2
 
 template <int BN, int EPI>
 __global__ void __launch_bounds__(192, 1)
@@ -213,7 +214,10 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
               __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out) + n;
 #pragma unroll
               for (int j = 0; j < 32; ++j)
-                if (c0 + j < M) o[(size_t)(c0 + j) * N] = __float2bfloat16_rn(__uint_as_float(r[j]) + bv);
+                if (c0 + j < M) {
+                  const float v = __uint_as_float(r[j]) + bv;
+                  o[(size_t)(c0 + j) * N] = __float2bfloat16_rn(EPI == LT_EPI_RELU2 ? relu2_f32(v) : v);
+                }
             }
           }
         }
@@ -280,7 +284,7 @@ SLLM_EXPORT int sllm_linear_tc_splits(int K, int want) {
 
 // epilogue 0: float32 out[splits, M, N] (bias in the first slice); 1: bfloat16 out[M, N] (+bias; one
 // slice); 2: bfloat16 out[M, N/2] = silu(gate) * up for W rows interleaved in blocks of 8 (N a multiple
-// of 16; one slice).  `status` as for sllm_gemm_tcgen05 (codes 31 producer, 32 MMA issuer, 33 epilogue).
+// of 16; one slice); 3: bfloat16 max(product (+bias), 0)^2 (one slice).  `status` as for sllm_gemm_tcgen05 (codes 31 producer, 32 MMA issuer, 33 epilogue).
 SLLM_EXPORT int sllm_linear_tc(const void* x, const void* W, const float* bias, void* out, int M, int N, int K, int want_splits,
                                int epilogue, int* status, cudaStream_t stream) {
   SLLM_REQUIRE(M >= 1 && M <= 128 && N >= 8 && K >= 8 && K % 8 == 0, "linear_tc: sizes M=%d N=%d K=%d (M <= 128, K a multiple of 8)", M, N, K);
@@ -302,12 +306,14 @@ SLLM_EXPORT int sllm_linear_tc(const void* x, const void* W, const float* bias, 
       case LT_EPI_F32: LT_LAUNCH(64, LT_EPI_F32);
       case LT_EPI_BF16: LT_LAUNCH(64, LT_EPI_BF16);
       case LT_EPI_SILU: LT_LAUNCH(64, LT_EPI_SILU);
+      case LT_EPI_RELU2: LT_LAUNCH(64, LT_EPI_RELU2);
     }
   } else {
     switch (epilogue) {
       case LT_EPI_F32: LT_LAUNCH(128, LT_EPI_F32);
       case LT_EPI_BF16: LT_LAUNCH(128, LT_EPI_BF16);
       case LT_EPI_SILU: LT_LAUNCH(128, LT_EPI_SILU);
+      case LT_EPI_RELU2: LT_LAUNCH(128, LT_EPI_RELU2);
     }
   }
 #undef LT_LAUNCH

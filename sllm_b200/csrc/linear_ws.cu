@@ -10,6 +10,7 @@
 // partial tiles are added through shared memory in warp order (a fixed order), and since the CTA
 // holds complete sums the epilogue can finish the layer's job:
 //   store      out[M, N] (+ bias), float32 or bfloat16
+//              optionally through an activation: max(v, 0)^2, or gelu_tanh(v) times the token's own entry of a table
 //   residual   residual[M, N] += y (+ bias): the float32 stream is updated in place, so the next
 //              norm has nothing to add
 //   rotary     for the fused q|k|v matrix of an attention layer: bias, rotary encoding and the write
@@ -98,7 +99,7 @@ template <int NT, int EPI, typename OUT, bool SCALED>
 __global__ void __launch_bounds__(WS_WARPS * 32, 2)
 linear_ws_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ W,
                  const float* __restrict__ bias, OUT* __restrict__ out, float* __restrict__ residual,
-                 int M, int N, int K, const WsRope rope, const WsNorm norm) {
+                 int M, int N, int K, const WsRope rope, const WsNorm norm, const int act, const TokenTable token) {
   constexpr int WS_DEPTH = ws_depth(NT);
   __shared__ float red[WS_WARPS][16][8 * NT + 1];
   __shared__ float row_scale[8 * NT];
@@ -278,6 +279,8 @@ linear_ws_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __res
         if (row == 0 && tok < M) norm.ssq_out[(size_t)tok * ((gridDim.x + 3) & ~3) + blockIdx.x] = sq;
       }
     } else if (valid) {
+      if (act == SLLM_ACT_RELU2) v = relu2_f32(v);
+      else if (act == SLLM_ACT_TOKEN) v = gelu_tanh_f32(v) * __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(token.table)[token_row(token, tok) + n]);
       out[(size_t)tok * N + n] = from_f32<OUT>(v);
     }
   }
@@ -299,12 +302,13 @@ static int ws_ctas(int N, int K, bool rope) {
 
 template <int NT, int EPI, typename OUT>
 static int launch_ws(const __nv_bfloat16* x, const __nv_bfloat16* W, const float* bias, void* out, float* residual,
-                     int M, int N, int K, cudaStream_t stream, const WsRope& rope = WsRope{}, const WsNorm& norm = WsNorm{}) {
+                     int M, int N, int K, cudaStream_t stream, const WsRope& rope = WsRope{}, const WsNorm& norm = WsNorm{},
+                     int act = SLLM_ACT_NONE, const TokenTable& token = TokenTable{}) {
   const int ctas = ws_ctas(N, K, EPI == WS_EPI_ROPE);
   if (norm.ssq_in != nullptr)
-    launch_kernel(linear_ws_kernel<NT, EPI, OUT, true>, ctas, WS_WARPS * 32, 0, stream, x, W, bias, (OUT*)out, residual, M, N, K, rope, norm);
+    launch_kernel(linear_ws_kernel<NT, EPI, OUT, true>, ctas, WS_WARPS * 32, 0, stream, x, W, bias, (OUT*)out, residual, M, N, K, rope, norm, act, token);
   else
-    launch_kernel(linear_ws_kernel<NT, EPI, OUT, false>, ctas, WS_WARPS * 32, 0, stream, x, W, bias, (OUT*)out, residual, M, N, K, rope, norm);
+    launch_kernel(linear_ws_kernel<NT, EPI, OUT, false>, ctas, WS_WARPS * 32, 0, stream, x, W, bias, (OUT*)out, residual, M, N, K, rope, norm, act, token);
   return launch_status("linear_ws");
 }
 
@@ -333,9 +337,17 @@ static bool ws_norm_in(WsNorm& n, const float* ssq_in, int parts_in, float eps_i
 // squares of the stream's rows (width_in wide): each row of the product is multiplied by rsqrt(sum / width_in + eps_in).
 // gain != null (residual epilogue only): also write xg_out [M, N] = bfloat16(residual * gain) and
 // ssq_out [M][sllm_linear_ws_parts(N, K) rounded up to 4], the next norm's input in the same form.
+// act: what the plain result passes before its store (SLLM_ACT_*; SLLM_ACT_TOKEN with the bfloat16 table of the tokens).
 SLLM_EXPORT int sllm_linear_ws(const void* x, const void* W, const float* bias, void* out, int out_dtype, float* residual,
                                int M, int N, int K, const float* ssq_in, int parts_in, float eps_in, int width_in,
-                               const float* gain, void* xg_out, float* ssq_out, cudaStream_t stream) {
+                               const float* gain, void* xg_out, float* ssq_out, int act, const void* token_table, const int* token_ids,
+                               int token_off, int token_ld, int token_rows, cudaStream_t stream) {
+  SLLM_REQUIRE(act == SLLM_ACT_NONE || ((act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN) && residual == nullptr),
+               "linear_ws: activation %d (0 none, 1 relu squared, 2 gelu times the tokens' table), not with a residual", act);
+  SLLM_REQUIRE(act != SLLM_ACT_TOKEN || (token_table && token_ids && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld),
+               "linear_ws: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
+  TokenTable tt;
+  tt.table = token_table; tt.ids = token_ids; tt.off = token_off; tt.ld = token_ld; tt.V = token_rows;
   SLLM_REQUIRE(sllm_linear_ws_supports(M, N, K), "linear_ws: sizes M=%d N=%d K=%d (needs M<=32, K%%32==0)", M, N, K);
   SLLM_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)W & 15) == 0, "linear_ws: operands must be 16-byte aligned");
   SLLM_REQUIRE(residual != nullptr || out != nullptr, "linear_ws: no destination");
@@ -350,8 +362,8 @@ SLLM_EXPORT int sllm_linear_ws(const void* x, const void* W, const float* bias, 
   const __nv_bfloat16* wb = (const __nv_bfloat16*)W;
 #define GO(NT_)                                                                                                        \
   if (residual) return launch_ws<NT_, WS_EPI_RESID, float>(xb, wb, bias, nullptr, residual, M, N, K, stream, WsRope{}, nm);          \
-  if (out_dtype == SLLM_BF16) return launch_ws<NT_, WS_EPI_STORE, __nv_bfloat16>(xb, wb, bias, out, nullptr, M, N, K, stream, WsRope{}, nm); \
-  return launch_ws<NT_, WS_EPI_STORE, float>(xb, wb, bias, out, nullptr, M, N, K, stream, WsRope{}, nm);
+  if (out_dtype == SLLM_BF16) return launch_ws<NT_, WS_EPI_STORE, __nv_bfloat16>(xb, wb, bias, out, nullptr, M, N, K, stream, WsRope{}, nm, act, tt); \
+  return launch_ws<NT_, WS_EPI_STORE, float>(xb, wb, bias, out, nullptr, M, N, K, stream, WsRope{}, nm, act, tt);
   if (M <= 8) { GO(1) }
   if (M <= 16) { GO(2) }
   GO(4)

@@ -1,7 +1,8 @@
 // Kernels of layers that wrap each sublayer in two norms, and of the small recurrent and gated units such layers hold.
 //
 //   * post_add_norm: a sublayer's output is normed BEFORE it joins the stream, and the stream is normed for the next
-//     reader in the same pass:  stream += term / rms(term) * post_gain;  h = stream / rms(stream) * pre_gain.  Either
+//     reader in the same pass:  stream += term / rms(term) * post_gain;  h = stream / rms(stream) * pre_gain (or, without
+//     a pre_gain, h = the stream itself in the reader's dtype).  Either
 //     half may be absent (the first norm of a model has no term; the last sublayer has no reader).  A CTA per token,
 //     float32 throughout; `term` may be a stack of k-split partial sums.  post_add_norm_conv: where every request
 //     brings one token, the reader's input convolution rides along: h + conv(h) from the request's state row, which the
@@ -111,6 +112,14 @@ post_add_norm_kernel(float* __restrict__ stream, const float* __restrict__ term,
     float y[PER];
     float ss = post_add_regs<PER>(x, term, base, parts, part_stride, post_gain, post_eps, W, red, y);
     if (h == nullptr) return;
+    if (pre_gain == nullptr) {                  // (the reader takes the stream as it is)
+#pragma unroll
+      for (int k = 0; k < PER; ++k) {
+        const int i = threadIdx.x + k * 256;
+        if (i < W) h[base + i] = from_f32<TO>(y[k]);
+      }
+      return;
+    }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)W + pre_eps);
 #pragma unroll
@@ -121,6 +130,10 @@ post_add_norm_kernel(float* __restrict__ stream, const float* __restrict__ term,
   } else {
     float ss = post_add(x, term, base, parts, part_stride, post_gain, post_eps, W, red);
     if (h == nullptr) return;
+    if (pre_gain == nullptr) {
+      for (int i = threadIdx.x; i < W; i += blockDim.x) h[base + i] = from_f32<TO>(x[i]);
+      return;
+    }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)W + pre_eps);
     for (int i = threadIdx.x; i < W; i += blockDim.x) h[base + i] = from_f32<TO>(x[i] * inv * pre_gain[i]);
@@ -408,7 +421,6 @@ SLLM_EXPORT int sllm_post_add_norm(float* stream_, const float* term, int parts,
                                    cudaStream_t stream) {
   SLLM_REQUIRE(T >= 0 && W > 0, "post_add_norm: bad sizes T=%d W=%d", T, W);
   SLLM_REQUIRE(term == nullptr || (post_gain != nullptr && parts >= 1), "post_add_norm: a term needs its gain");
-  SLLM_REQUIRE(h == nullptr || pre_gain != nullptr, "post_add_norm: a normed output needs its gain");
   SLLM_REQUIRE(term != nullptr || h != nullptr, "post_add_norm: nothing to do");
   if (T == 0) return SLLM_OK;
 #define PAN(TO_, PER_)                                                                                                      \

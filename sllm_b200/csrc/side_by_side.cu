@@ -302,16 +302,17 @@ SLLM_EXPORT int sllm_qk_norm_rope_kv_write(const float* qkv, int ld, const float
   SLLM_REQUIRE((q_gain == nullptr) == (k_gain == nullptr), "qk_norm_rope: query and key heads are normed together or not at all");
   SLLM_REQUIRE(T >= 0 && nq > 0 && nkv > 0 && dim > 0 && vdim > 0, "qk_norm_rope: bad sizes T=%d nq=%d nkv=%d dim=%d vdim=%d", T, nq, nkv, dim, vdim);
   SLLM_REQUIRE(D >= dim && D >= vdim, "qk_norm_rope: the cache's head of %d is smaller than a key of %d or a value of %d", D, dim, vdim);
-  SLLM_REQUIRE(ld >= (nq + nkv) * dim + nkv * vdim, "qk_norm_rope: the product's %d columns are fewer than q|k|v", ld);
+  SLLM_REQUIRE(ld >= nq * dim + (slot_mapping != nullptr ? nkv * (dim + vdim) : 0), "qk_norm_rope: the product's %d columns are fewer than q|k|v", ld);
   SLLM_REQUIRE(rot >= 0 && rot <= dim && rot % 2 == 0, "qk_norm_rope: rotary_dim=%d must be even and <= %d", rot, dim);
   SLLM_REQUIRE(rot == 0 || (table != nullptr && max_pos > 0), "qk_norm_rope: rotary table missing");
   SLLM_REQUIRE(slot_mapping == nullptr || (page_size > 0 && num_pages > 0 && k_cache && v_cache), "qk_norm_rope: cache arguments missing");
   if (T == 0) return SLLM_OK;
-  const long items = (long)T * (nq + 2 * nkv);
+  const int nkv_w = slot_mapping != nullptr ? nkv : 0;        // (a borrowed cache: queries alone; the product may hold no keys and values)
+  const long items = (long)T * (nq + 2 * nkv_w);
   const unsigned blocks = (unsigned)((items + 3) / 4);
 #define LAUNCH(TC)                                                                                                        \
   launch_kernel(qk_norm_rope_kv_write_kernel<TC>, blocks, 128, 0, stream, qkv, ld, q_gain, k_gain, q_mul, eps, positions, table, rot, \
-                max_pos, nq, nkv, dim, vdim, D, slot_mapping, page_size, num_pages, (TC*)k_cache, (TC*)v_cache, (TC*)q_out, T)
+                max_pos, nq, nkv_w, dim, vdim, D, slot_mapping, page_size, num_pages, (TC*)k_cache, (TC*)v_cache, (TC*)q_out, T)
   if (cache_dtype == SLLM_F32) LAUNCH(float);
   else if (cache_dtype == SLLM_BF16) LAUNCH(__nv_bfloat16);
   else SLLM_REQUIRE(false, "qk_norm_rope: unknown dtype %d", cache_dtype);

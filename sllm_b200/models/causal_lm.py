@@ -11,10 +11,10 @@ from .. import ops
 from ..config.plan import ModelPlan
 from ..parts import delta_rule as _delta_rule, experts as _experts, latent_attention as _latent  # noqa: F401
 from ..parts import linear_attention as _linear_attention, parallel as _parallel, side_by_side as _side_by_side  # noqa: F401
-from ..parts import gated_recurrence as _gated_recurrence, sandwich as _sandwich  # noqa: F401
+from ..parts import gated_recurrence as _gated_recurrence, output_norm as _output_norm, sandwich as _sandwich  # noqa: F401
 from ..parts import standard as _standard  # noqa: F401  (each import registers its parts)
-from ..parts.base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, SHIFTS,
-                          LayerCache, OwedNorm, SlotState, StepContext, TensorSpec, flatten_needs, join_name)
+from ..parts.base import (BLOCKS, COMPLETE, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, SHIFTS,
+                          LayerCache, SlotState, StepContext, TensorSpec, flatten_needs, join_name)
 
 
 FAMILIES = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "norm": NORMS, "shift": SHIFTS}
@@ -54,6 +54,7 @@ class CausalLM:
         self.final_norm = NORMS.build(plan.final_norm, **kw)
         self.embedding_norm = NORMS.build(plan.embedding_norm, **kw) if plan.embedding_norm is not None else None
         self.pass_vectors = None   # [passes, H] float32
+        self.token_table = None    # [V, width] compute dtype: vectors that belong to a token
         self.position = POSITIONS.build(plan.position, **kw) if plan.position is not None else None
         self.embedding = None      # [V, H] compute dtype
         self.head = None           # [V, H] compute dtype (the embedding itself when tied)
@@ -79,6 +80,8 @@ class CausalLM:
             specs.append(TensorSpec(p.head_name, (p.vocab_size, p.hidden_size), role="matrix"))
         if p.pass_vectors_name is not None:
             specs.append(TensorSpec(p.pass_vectors_name, (p.passes, p.hidden_size), role="bias"))
+        if p.token_table_name is not None:
+            specs.append(TensorSpec(p.token_table_name, (p.vocab_size, p.token_table_width), role="embedding"))
         return specs
 
     def ignored_tensor_names(self):
@@ -92,6 +95,11 @@ class CausalLM:
             part.bind(lambda rel, _p=prefix: fetch(join_name(_p, rel)))
         if p.pass_vectors_name is not None:
             self.pass_vectors = fetch(p.pass_vectors_name).to(device=self.device, dtype=torch.float32).contiguous()
+        if p.token_table_name is not None:
+            self.token_table = fetch(p.token_table_name).to(device=self.device, dtype=self.dtype).contiguous()
+            for _, part in self._named_parts():
+                if hasattr(part, "adopt_token_table"):
+                    part.adopt_token_table(self.token_table)
         if p.head_name is None:
             self.head = self.embedding
         else:
@@ -152,11 +160,12 @@ class CausalLM:
                 # the norm that reads the stream next: this block's last product may prepare its input
                 kw["next_norm"] = getattr(self.layers[runs[i + 1].layer].block, "first_norm", None)
             delta = block.forward(residual, delta, step, caches[i], self.position, write_cache=e.cache_from is None, **kw)
-        if isinstance(delta, OwedNorm):          # (a block handed one on although nothing asked: take the stream as it is)
+        if isinstance(delta, COMPLETE):          # (a block handed one on although nothing asked: take the stream as it is)
             delta = None
         if step.logit_rows.numel() == 0:
             return torch.empty((0, self.plan.vocab_size), dtype=torch.float32, device=self.device)
         res_rows = ops.gather_rows(residual, step.logit_rows)
         delta_rows = ops.gather_rows(delta, step.logit_rows) if delta is not None else None
         x = self.final_norm.add_norm(res_rows, delta_rows)
-        return ops.linear(x, self.head, None, torch.float32)
+        logits = ops.linear(x, self.head, None, torch.float32)
+        return ops.softcap_(logits, self.plan.logit_softcap) if self.plan.logit_softcap is not None else logits

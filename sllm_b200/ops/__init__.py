@@ -208,7 +208,7 @@ GATE_ACTS = {"sigmoid": 0, "silu": 1, "none": 2}
 
 def delta_out(o, gain, proj, off_g: int, eps: float, heads: int, dv: int, out_dtype, gate_act: str = "sigmoid", out=None,
               out_off: int = 0) -> torch.Tensor:
-    """Each head's ``o`` over its root mean square, times ``gain`` (``[heads*dv]``), times ``sigmoid`` (or ``silu``) of
+    """Each head's ``o`` over its root mean square, times ``gain`` (``[heads*dv]``; None: ones), times ``sigmoid`` (or ``silu``) of
     the gate logits (columns ``off_g`` of ``proj``), in ``out_dtype``; with ``gate_act`` ``none`` there is no gate and
     ``proj`` may be None.  ``out``: a wider tensor whose columns ``out_off ..`` receive the result."""
     if gate_act == "none":
@@ -309,7 +309,7 @@ def qk_norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, positions, table, rot
     """From a float32 product ``[T, (nq+nkv)*dim + nkv*vdim]``: every query and key head over its root mean square times
     its gain (``[dim]``, shared by the heads), then rotated; values as they are.  The queries come back ``[T, nq*D]`` in
     ``out_dtype`` with D the cache's head size (>= dim and vdim; zeros beyond); keys and values go to ``slot_mapping`` in
-    the pages (not written when ``slot_mapping`` is None).  With both gains None the heads are not normed; ``q_mul``
+    the pages (not written when ``slot_mapping`` is None: the product may then end behind the queries' columns).  With both gains None the heads are not normed; ``q_mul``
     (float32 ``[nq]``) multiplies each query head.  ``col_off``: the column of ``qkv`` at which q|k|v start (a product that
     holds other projections too)."""
     _chk(qkv, q_gain, k_gain, q_mul, positions, table, slot_mapping, k_cache, v_cache)
@@ -323,7 +323,7 @@ def qk_norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, positions, table, rot
             raise KernelError("qk_norm_rope_kv_write: rotary table must be float32 [positions, 2, rotary_dim/2]")
         max_pos = table.shape[0]
     q = torch.empty((T, nq * D), dtype=out_dtype, device=qkv.device)
-    if col_off < 0 or col_off + (nq + nkv) * dim + nkv * vdim > ld:
+    if col_off < 0 or col_off + nq * dim + (nkv * (dim + vdim) if slot_mapping is not None else 0) > ld:
         raise KernelError("qk_norm_rope_kv_write: q|k|v lie outside the product's columns")
     call("sllm_qk_norm_rope_kv_write", _p(qkv) + 4 * int(col_off), ld, _p(q_gain), _p(k_gain), _p(q_mul), float(eps), _p(positions), _p(table), int(rotary_dim),
          max_pos, nq, nkv, dim, vdim, D, _p(slot_mapping), page_size, num_pages, _p(k_cache), _p(v_cache), _p(q),
@@ -454,6 +454,31 @@ def post_add_norm(stream, term, post_gain, post_eps: float, pre_gain, pre_eps: f
     return h
 
 
+def post_add_copy(stream, term, post_gain, post_eps: float, out_dtype=None):
+    """``stream += term / rms(term) * post_gain`` (skipped when ``term`` is None), for a reader that takes the stream as it is:
+    returns the stream in ``out_dtype`` (the stream itself where that is float32, None where ``out_dtype`` is None)."""
+    _chk(stream, term, post_gain)
+    T, W = stream.shape
+    if stream.dtype != torch.float32 or (term is not None and tuple(term.shape[-2:]) != (T, W)):
+        raise KernelError("post_add_copy: a float32 stream [T, W] and a term that fits it")
+    h = None
+    if out_dtype is not None and out_dtype != torch.float32:
+        h = torch.empty((T, W), dtype=out_dtype, device=stream.device)
+    if term is not None or h is not None:
+        call("sllm_post_add_norm", _p(stream), *_term(term), _p(post_gain), float(post_eps), None, 0.0, _p(h),
+             _dtc(out_dtype) if h is not None else F32, T, W, _stream())
+    return stream if out_dtype == torch.float32 else h
+
+
+def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(x / cap)`` in place on a float32 tensor."""
+    _chk(x)
+    if x.dtype != torch.float32:
+        raise KernelError("softcap_: float32 values")
+    call("sllm_softcap", _p(x), x.numel(), float(cap), _stream())
+    return x
+
+
 def post_add_norm_conv(stream, term, post_gain, post_eps: float, pre_gain, pre_eps: float, weight, state, step, out_dtype):
     """`post_add_norm` and `short_conv_add` of its result in one launch, for a step in which every request brings ONE token:
     the normed row stays in the CTA, ``out = h + conv(h)`` reads the request's row of ``state`` (float32 ``[slots, W, taps-1]``)
@@ -501,6 +526,28 @@ def decay_linear_attention(proj, offs, decay, state, step, heads: int, dk: int, 
     off_q, off_k, off_v = (int(o) for o in offs)
     call("sllm_decay_linear_attention", _p(proj), ld, off_q, off_k, off_v, _p(decay), _p(state), _p(step.q_start),
          _p(step.state_slots), _p(out), step.num_seqs, heads, dk, dv, int(step.max_q_len), _stream())
+    return out
+
+
+def retention(proj, offs, decay, table, rotary_dim: int, k_scale: float, state, step, heads: int, dk: int, dv: int) -> torch.Tensor:
+    """S <- decay_h S + k v^T; o = S^T q over the step's tokens from and into ``state`` (float32 ``[slots, heads, dk, dv]``), with
+    q and k rotated by position over their first ``rotary_dim`` channels (channel i with i + rotary_dim/2; ``table`` float32
+    ``[positions, 2, rotary_dim/2]``, None: no rotation) and k then times ``k_scale``.  ``proj`` float32 ``[T, ld]`` holds q, k, v
+    at columns ``offs``; ``decay`` float32 ``[heads]``.  Returns ``o`` float32 ``[T, heads*dv]``."""
+    _chk(proj, decay, table, state)
+    T, ld = proj.shape
+    if proj.dtype != torch.float32 or decay.dtype != torch.float32 or state.dtype != torch.float32:
+        raise KernelError("retention: everything that enters the recurrence is float32")
+    if tuple(decay.shape) != (heads,) or tuple(state.shape[1:]) != (heads, dk, dv):
+        raise KernelError(f"retention: decay {tuple(decay.shape)} or state {tuple(state.shape)} does not fit {heads} heads of {dk}x{dv}")
+    rot = int(rotary_dim) if table is not None else 0
+    if rot and (table.dtype != torch.float32 or tuple(table.shape[1:]) != (2, rot // 2)):
+        raise KernelError("retention: rotary table must be float32 [positions, 2, rotary_dim/2]")
+    out = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
+    off_q, off_k, off_v = (int(o) for o in offs)
+    call("sllm_retention", _p(proj), ld, off_q, off_k, off_v, _p(decay), _p(step.positions), _p(table), rot, table.shape[0] if rot else 0,
+         float(k_scale), _p(state), _p(step.q_start), _p(step.state_slots), _p(out), step.num_seqs, heads, dk, dv, int(step.max_q_len),
+         _stream())
     return out
 
 
@@ -609,15 +656,33 @@ def stream_supports(M: int, N: int, K: int) -> bool:
     return not linear_tc_supports(M, N, K)
 
 
+PLAIN_ACTS = {None: 0, "relu2": 1, "token": 2}      # SLLM_ACT_* of the kernels: activations of a plain (ungated) result
+
+
+class TokenColumns:
+    """Columns ``off ..`` of a table with a row per token id (``table [V, ld]`` in the compute dtype), at the step's ``ids``
+    (int32 ``[T]``): what the ``token`` activation multiplies by."""
+    __slots__ = ("table", "ids", "off")
+
+    def __init__(self, table, ids, off: int):
+        self.table, self.ids, self.off = table, ids, int(off)
+
+    def args(self):
+        return _p(self.table), _p(self.ids), self.off, self.table.shape[1], self.table.shape[0]
+
+
+_NO_TOKEN = (None, None, 0, 0, 0)
+
+
 def linear_stream(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False, act: "str | None" = None):
     """The weight-streaming kernel for at most 64 tokens.  With ``splits`` > 1 the result is
     a float32 stack ``[splits', M, N]`` of partial sums (bias in the first) that the consumer
     adds; with ``silu`` the matrix is gate|up interleaved in blocks of 8 and the result is
     ``silu(gate) * up`` of width N/2; with ``act="gelu_tanh"`` it is ``gelu_tanh(gate + bias) * (up + bias)``
-    (the bias interleaved like the rows)."""
-    if act not in (None, "gelu_tanh") or (act and silu):
-        raise KernelError(f"linear_stream: gated epilogue {act!r}")
-    gated = silu or act is not None
+    (the bias interleaved like the rows); with ``act="relu2"`` the plain result's ``max(v, 0)^2`` (bfloat16)."""
+    if act not in (None, "gelu_tanh", "relu2") or (act and silu):
+        raise KernelError(f"linear_stream: epilogue {act!r}")
+    gated = silu or act == "gelu_tanh"
     _chk(x, w, bias)
     M, K = x.shape
     N = w.shape[0]
@@ -632,7 +697,7 @@ def linear_stream(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False,
     else:
         out = torch.empty((M, N // 2 if gated else N), dtype=out_dtype, device=x.device)
     call("sllm_linear_stream", _p(x), _p(w), _p(bias), _p(out), _dtc(out_dtype), _p(partial), M, N, K,
-         real if real > 1 else 1, 1 if silu else 2 if act else 0, _stream())
+         real if real > 1 else 1, 1 if silu else {None: 0, "gelu_tanh": 2, "relu2": 3}[act], _stream())
     return partial if real > 1 else out
 
 
@@ -800,7 +865,7 @@ def pair_splits(M: int, N: int, K: int) -> int:
 
 
 def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | None" = None, scale: "RowScale | None" = None,
-              residual=None, next_gain=None, splits: int = 1, act: "str | None" = None):
+              residual=None, next_gain=None, splits: int = 1, act: "str | None" = None, token: "TokenColumns | None" = None):
     """The same product and epilogues as `gemm_tcgen05`, by pairs of CTAs on 256 x 256 tiles, on
     256 x 512 tiles (``wide=True``; by default where those fill the GPU at least as well; ``wide=448``, ``384`` or
     ``320``: tiles of that many columns, float32 result or residual epilogue, chosen by `pair_wide_cols` where
@@ -811,13 +876,17 @@ def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | 
     owed form and ``(xg, RowScale)`` comes back (the scale's eps left at 0 for the caller to set).
     ``splits`` > 1 (float32 result, no other epilogue): K in that many slices, the result a stack ``[splits', M, N]``
     of partial sums (bias in the first) for the consumer to add.  ``act="gelu_tanh"``: the gated epilogue
-    ``gelu_tanh(gate + bias) * (up + bias)`` in place of ``silu``'s (rows and bias interleaved in blocks of 8)."""
+    ``gelu_tanh(gate + bias) * (up + bias)`` in place of ``silu``'s (rows and bias interleaved in blocks of 8); ``"relu2"``:
+    bfloat16 ``max(v, 0)^2`` of the plain result; ``"token"``: bfloat16 ``gelu_tanh(v)`` times ``token``'s columns."""
     _chk(x, w, bias, residual, next_gain)
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_pair: bfloat16 operands only")
-    if act not in (None, "gelu_tanh") or (act and silu):
-        raise KernelError(f"gemm_pair: gated epilogue {act!r}")
-    gelu, silu = act is not None, silu or act is not None
+    if act not in (None, "gelu_tanh", "relu2", "token") or (act and silu):
+        raise KernelError(f"gemm_pair: epilogue {act!r}")
+    plain_act = act if act in ("relu2", "token") else None
+    gelu, silu = act == "gelu_tanh", silu or act == "gelu_tanh"
+    if plain_act and (residual is not None or bias is not None or out_dtype != torch.bfloat16 or (token is None) != (act == "relu2")):
+        raise KernelError(f"gemm_pair: the {act} epilogue takes neither bias nor residual and gives bfloat16")
     M, K = x.shape
     N = w.shape[0]
     if w.shape[1] != K:
@@ -827,7 +896,7 @@ def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | 
     plain_or_residual = not silu and (residual is not None or out_dtype == torch.float32)
     if wide is None:
         wide = False if splits > 1 else "slim" if pair_tiles_slim(M, N) else \
-            pair_wide_cols(M, N) if plain_or_residual else pair_tiles_wide(M, N)
+            False if act == "token" else pair_wide_cols(M, N) if plain_or_residual else pair_tiles_wide(M, N)
     code = 2 if wide == "slim" else 0 if wide is False else 1 if wide is True or wide == 512 else int(wide)
     if code > 2 and (code not in (448, 384, 320) or not plain_or_residual):
         raise KernelError(f"gemm_pair: tiles of {wide} columns (448, 384 or 320, and only with a float32 result or a residual)")
@@ -848,12 +917,13 @@ def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | 
         real = int(lib().sllm_gemm_pair_splits(K, int(splits))) if splits > 1 else 1
         epi, out = 0, torch.empty((real, M, N) if real > 1 else (M, N), dtype=torch.float32, device=x.device)
     else:
-        epi, out = 1, torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        epi, out = {None: 1, "relu2": 5, "token": 6}[plain_act], torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     if splits > 1 and (epi != 0 or scale is not None):
         raise KernelError("gemm_pair: slices of K leave float32 partial sums: no other epilogue, no owed norm")
     call("sllm_gemm_pair", _p(x), _p(w), _p(bias), _p(out), M, N, K, epi, code, int(splits),
          *(scale.args_with_stride() if scale is not None else (None, 0, 0, 0.0, 0)),
-         _p(residual), _p(next_gain), _p(xg), _p(ssq), stride, _p(_status_word(x.device)), _stream())
+         _p(residual), _p(next_gain), _p(xg), _p(ssq), stride, *(token.args() if token is not None else _NO_TOKEN),
+         _p(_status_word(x.device)), _stream())
     _tc_used["since_check"] += 1
     if residual is not None:
         return (xg, RowScale(ssq, pair_parts(N, code), 0.0, N)) if next_gain is not None else None
@@ -912,12 +982,14 @@ def _tc_splits(N: int, K: int) -> int:
     return max(1, min(num_sms() // tiles, (K // 64) // 8))
 
 
-def linear_tc(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False):
+def linear_tc(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False, act: "str | None" = None):
     """The weight-streaming product on the tcgen05 tensor cores for up to 128 tokens.  With
     ``splits`` > 1 the result is a float32 stack ``[splits', M, N]`` of partial sums (bias in the
     first) that the consumer adds; with ``silu`` the matrix is gate|up interleaved in blocks of 8
-    and the bfloat16 result is ``silu(gate) * up`` of width N/2."""
+    and the bfloat16 result is ``silu(gate) * up`` of width N/2; with ``act="relu2"`` the bfloat16 result is ``max(v, 0)^2``."""
     _chk(x, w, bias)
+    if act not in (None, "relu2") or (act and (silu or out_dtype != torch.bfloat16)):
+        raise KernelError(f"linear_tc: epilogue {act!r}")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("linear_tc: bfloat16 operands only")
     M, K = x.shape
@@ -932,7 +1004,7 @@ def linear_tc(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False):
         epi = 0
         out = torch.empty((real, M, N) if real > 1 else (M, N), dtype=torch.float32, device=x.device)
     else:
-        epi, out = 1, torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        epi, out = 3 if act else 1, torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     call("sllm_linear_tc", _p(x), _p(w), _p(bias), _p(out), M, N, K, real, epi, _p(_status_word(x.device)), _stream())
     _tc_used["since_check"] += 1
     return out
@@ -988,12 +1060,14 @@ _NO_SCALE = (None, 0, 0.0, 0)
 MAX_SCALE_PARTS = 608          # partial sums a consumer keeps in shared memory per row
 
 
-def linear_ws(x, w, bias, out_dtype, residual=None, scale: RowScale | None = None, next_gain=None):
+def linear_ws(x, w, bias, out_dtype, residual=None, scale: RowScale | None = None, next_gain=None, act: "str | None" = None,
+              token: "TokenColumns | None" = None):
     """The warp-split streaming kernel (at most 16 tokens): ``x @ w.T (+ bias)`` in ``out_dtype``,
     or, given ``residual`` (float32 ``[M, N]``), added into it in place (returns None).  ``scale``: a norm
     still owed on ``x`` (`RowScale`).  ``next_gain`` (with ``residual``): the gain of the norm that follows; the
     kernel then also writes that norm's input in the owed form and ``(xg, RowScale)`` is returned (the scale's
-    eps is left at 0 for the caller to set)."""
+    eps is left at 0 for the caller to set).  ``act`` (without ``residual``): ``"relu2"``, the result's ``max(v, 0)^2``, or
+    ``"token"``, ``gelu_tanh(v)`` times ``token``'s columns."""
     _chk(x, w, bias, residual, next_gain)
     M, K = x.shape
     N = w.shape[0]
@@ -1013,7 +1087,8 @@ def linear_ws(x, w, bias, out_dtype, residual=None, scale: RowScale | None = Non
         xg = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
         ssq = torch.empty((M, (parts + 3) & ~3), dtype=torch.float32, device=x.device)
     call("sllm_linear_ws", _p(x), _p(w), _p(bias), _p(out), _dtc(out_dtype), _p(residual), M, N, K,
-         *(scale.args() if scale is not None else _NO_SCALE), _p(next_gain), _p(xg), _p(ssq), _stream())
+         *(scale.args() if scale is not None else _NO_SCALE), _p(next_gain), _p(xg), _p(ssq),
+         PLAIN_ACTS[act], *(token.args() if token is not None else _NO_TOKEN), _stream())
     if next_gain is not None:
         return xg, RowScale(ssq, parts, 0.0, N)
     return out
@@ -1127,6 +1202,41 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias, out_dtype: torch.dtype, allow
     if bias is not None:
         out += bias.to(out.dtype)
     return out
+
+
+def plain_act(x, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
+    """``act`` of ``x [T, N]`` in ``out_dtype``: ``relu2`` is ``max(x, 0)^2``, ``token`` is ``gelu_tanh(x)`` times ``token``'s columns
+    (a table of ``out_dtype``)."""
+    _chk(x)
+    T, N = x.shape
+    if (act == "token") != (token is not None) or (token is not None and token.table.dtype != out_dtype):
+        raise KernelError("plain_act: the token activation needs its table, of the result's dtype")
+    out = torch.empty((T, N), dtype=out_dtype, device=x.device)
+    call("sllm_plain_act", _p(x), _dt(x), _p(out), _dtc(out_dtype), T, N, PLAIN_ACTS[act], *(token.args() if token is not None else _NO_TOKEN),
+         _stream())
+    return out
+
+
+_PLAIN_ACT_FUSED = os.environ.get("SLLM_PLAIN_ACT_FUSED", "1") != "0"      # 0: the product, then the activation kernel
+
+
+def linear_plain_act(x, w, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
+    """``act(x @ w.T)`` in ``out_dtype`` (see `plain_act`).  bfloat16: the activation leaves with the product's tile (the warp-split
+    streaming product, the CTA-pair product; ``relu2`` also in the streaming product and on tensor memory up to 128 tokens).
+    Otherwise the product in float32, then the activation kernel."""
+    if _PLAIN_ACT_FUSED and x.is_cuda and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and \
+            x.shape[1] == w.shape[1]:
+        M, K = x.shape
+        N = w.shape[0]
+        if ws_supports(M, N, K):
+            return linear_ws(x, w, None, out_dtype, act=act, token=token)
+        if act == "relu2" and stream_supports(M, N, K):
+            return linear_stream(x, w, None, out_dtype, act=act)
+        if act == "relu2" and N * K >= LINEAR_TC_LARGE and linear_tc_supports(M, N, K):
+            return linear_tc(x, w, None, out_dtype, act=act)
+        if _pair_rows(M) and pair_supports(M, N, K):
+            return gemm_pair(x, w, None, out_dtype, act=act, token=token)
+    return plain_act(linear(x, w, None, torch.float32), out_dtype, act, token)
 
 
 def silu_mul(gu: torch.Tensor, interleave: int, out_dtype: torch.dtype) -> torch.Tensor:
@@ -1253,9 +1363,21 @@ def rope_kv_write(qkv, bias, positions, table, rotary_dim, nq, nkv, hd, slot_map
     return q
 
 
-def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None):
+def _gate_args(gate):
+    """(pointer to the first token's logit of head 0, row length) of a per-head output gate given as (float32 product, column)."""
+    if gate is None:
+        return None, 0
+    t, off = gate
+    if t.dtype != torch.float32 or t.dim() != 2:
+        raise KernelError("attention: the heads' gates are columns of a float32 product")
+    return _p(t) + 4 * int(off), t.shape[1]
+
+
+def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None,
+                   softcap: float = 0.0, gate=None):
     """The CUDA-core attention kernel: any head size up to 640 (one instance to 256, one beyond), float32 arithmetic.  ``sink`` (float32 ``[nq]``): the
-    softmax's denominator also holds exp(sink_h), a term without key or value that the scale does not touch."""
+    softmax's denominator also holds exp(sink_h), a term without key or value that the scale does not touch.  ``softcap``, ``gate``:
+    see `paged_attention`."""
     _chk(q, k_cache, v_cache, block_tables, positions, seq_of_token)
     T = q.shape[0]
     if q.dtype != k_cache.dtype:
@@ -1264,7 +1386,7 @@ def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, n
     out = torch.empty_like(q)
     call("sllm_attention_simt", _p(q), _p(k_cache), _p(v_cache), _dt(q), _p(block_tables),
          block_tables.shape[1], _p(positions), _p(seq_of_token), T, nq, nkv, hd, page_size, float(scale),
-         int(window or 0), int(block or 0), _p(sink), _p(out), _stream())
+         int(window or 0), int(block or 0), _p(sink), float(softcap or 0.0), *_gate_args(gate), _p(out), _stream())
     return out
 
 
@@ -1338,7 +1460,7 @@ def choose_splits(num_small: int, nkv: int, max_ctx: int, ctas_per_sm: int = 2, 
 
 
 def attention_mma(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, decode: bool, num_splits: int,
-                  nq, nkv, hd, scale, window, out=None, block=None, sink=None):
+                  nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None):
     """The tensor-core attention kernel on one tile list (see `attention_tiles`); the merge of a split context
     touches the rows of that list's requests only."""
     _chk(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles[0], tiles[1])
@@ -1353,7 +1475,8 @@ def attention_mma(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, de
         part_lse = torch.empty((num_splits, T, nq), dtype=torch.float32, device=q.device)
     call("sllm_attention_mma", _p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_o), _p(part_lse), _p(block_tables),
          block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]), tiles[2], 1 if decode else 0,
-         num_splits, T, nq, nkv, hd, k_cache.shape[2], float(scale), int(window or 0), int(block or 0), _p(sink), _stream())
+         num_splits, T, nq, nkv, hd, k_cache.shape[2], float(scale), int(window or 0), int(block or 0), _p(sink),
+         float(softcap or 0.0), *_gate_args(gate), _stream())
     if num_splits > 1:
         launches["own"] += 1          # the combine kernel
     return out
@@ -1370,7 +1493,7 @@ def _tma_ctas_per_sm(hd: int) -> int:
 
 
 def attention_tma_decode(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, num_splits: int,
-                         nq, nkv, hd, scale, window, out=None, block=None, sink=None):
+                         nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None):
     """The decode form fed by TMA (16-row tiles only; see `attention_tiles`)."""
     _chk(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles[0], tiles[1])
     if q.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16:
@@ -1385,7 +1508,7 @@ def attention_tma_decode(q, k_cache, v_cache, block_tables, q_start, ctx_len, ti
     call("sllm_attention_tma_decode", _p(q), _p(k_cache), _p(v_cache), k_cache.shape[0], _p(out), _p(part_o),
          _p(part_lse), _p(block_tables), block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]),
          tiles[2], num_splits, T, nq, nkv, hd, k_cache.shape[2], float(scale), int(window or 0), int(block or 0),
-         _p(sink), _p(_status_word(q.device)), _stream())
+         _p(sink), float(softcap or 0.0), *_gate_args(gate), _p(_status_word(q.device)), _stream())
     _tc_used["since_check"] += 1
     if num_splits > 1:
         launches["own"] += 1
@@ -1421,7 +1544,7 @@ def choose_tc_splits(num_tiles: int, nkv: int, max_ctx: int) -> tuple[int, int]:
 
 
 def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq, nkv, hd, scale, out=None,
-                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, sink=None):
+                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, sink=None, softcap: float = 0.0, gate=None):
     """The prefill form on tcgen05 (tiles of 128 * row_tiles rows, row_tiles 1 or 2; no window; see
     `attention_tiles`).  ``splits`` = (ranges, 64-key tiles a range) cuts the context into ranges
     that run as CTAs of their own and are merged afterwards; ranges x tiles must cover the longest
@@ -1442,7 +1565,8 @@ def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq,
     call("sllm_attention_tc", _p(q), _p(k_cache), _p(v_cache), k_cache.shape[0], _p(out), _p(block_tables),
          block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]), tiles[2], int(row_tiles), nq, nkv,
          hd, k_cache.shape[2], float(scale), n_splits, max(per, 1), T, _p(part_o), _p(part_lse),
-         _p(parts[0]) if parts else None, _p(parts[1]) if parts else None, _p(sink), _p(_status_word(q.device)), _stream())
+         _p(parts[0]) if parts else None, _p(parts[1]) if parts else None, _p(sink), float(softcap or 0.0), *_gate_args(gate),
+         _p(_status_word(q.device)), _stream())
     if n_splits > 1:
         launches["own"] += 1               # the merge kernel
     _tc_used["since_check"] += 1
@@ -1488,9 +1612,11 @@ def mma_supports(hd: int) -> bool:
     return bool(lib().sllm_attention_mma_supports(int(hd)))
 
 
-def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, window, block=None, sink=None):
+def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, window, block=None, sink=None, softcap: float = 0.0,
+                    gate=None):
     """Causal attention of the step's tokens over their requests' pages.  ``sink`` (float32 ``[nq]``): exp(sink_h) joins
-    each head's softmax denominator (every form takes it).  ``window``: only the last ``window`` keys;
+    each head's softmax denominator (every form takes it).  ``softcap`` > 0: a score becomes softcap tanh(score / softcap) before
+    the softmax; ``gate`` = (float32 product, column): head h's output times sigmoid of column + h (every form takes both).  ``window``: only the last ``window`` keys;
     ``block``: only the keys of the query's own block of ``block`` positions, counted from the sequence's start (both
     run on the mma.sync and TMA-fed forms, not on tcgen05).  bfloat16 with a head size
     the tensor-core kernels take: requests of at most 16 (token, head-in-group) rows go to the decode
@@ -1500,7 +1626,7 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     g = step.groups[group]
     if q.dtype != torch.bfloat16 or not mma_supports(hd):
         return attention_simt(q, k_cache, v_cache, g.block_tables, step.positions, step.seq_of_token,
-                              nq, nkv, hd, scale, window, block, sink)
+                              nq, nkv, hd, scale, window, block, sink, softcap, gate)
     G = nq // nkv
     # blocks that start on page borders: the prefill form runs each block's part of a portion as a causal sequence of its own
     blocked_tc = bool(block) and block % k_cache.shape[2] == 0 and bool(step.ctx_lens)
@@ -1528,19 +1654,19 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     out = torch.empty_like(q)
     if small and tma_attention_supports(hd, k_cache.shape[2]):
         attention_tma_decode(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, small, splits,
-                             nq, nkv, hd, scale, window, out, block, sink)
+                             nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
     elif small:
         attention_mma(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, small, True, splits,
-                      nq, nkv, hd, scale, window, out, block, sink)
+                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
     if large and use_tc and parts is not None:
         attention_tc(q, k_cache, v_cache, g.block_tables, parts[0], parts[1], parts[3], nq, nkv, hd, scale, out,
-                     row_tiles=rows // 128, parts=parts[2], sink=sink)
+                     row_tiles=rows // 128, parts=parts[2], sink=sink, softcap=softcap, gate=gate)
     elif large and use_tc:
         attention_tc(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, nq, nkv, hd, scale, out,
-                     row_tiles=rows // 128, splits=tc_splits, sink=sink)
+                     row_tiles=rows // 128, splits=tc_splits, sink=sink, softcap=softcap, gate=gate)
     elif large:
         attention_mma(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, False, 1,
-                      nq, nkv, hd, scale, window, out, block, sink)
+                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
     return out
 
 

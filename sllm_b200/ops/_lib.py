@@ -75,7 +75,7 @@ def _declare(L):
                                c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "sllm_gemm_f32": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_attention_simt": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                                c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                                c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
         "sllm_sample_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "sllm_repetition_penalty": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "sllm_mark_seen": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
@@ -85,17 +85,18 @@ def _declare(L):
         "sllm_attention_tma_ctas_per_sm": [c_int],
         "sllm_attention_tma_decode": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                                       c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                      c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                                      c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
         "sllm_wait_probe": [c_void_p, ctypes.c_ulonglong, c_void_p, c_void_p],
         "sllm_attention_tc_supports": [c_int, c_int],
         "sllm_attention_tc": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
-                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
         "sllm_gemm_tcgen05_supports": [c_int, c_int, c_int],
         "sllm_gemm_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "sllm_gemm_pair_supports": [c_int, c_int, c_int],
         "sllm_gemm_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                           c_void_p, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+                           c_void_p, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                           c_int, c_int, c_void_p, c_void_p],
         "sllm_gemm_pair_parts": [c_int],
         "sllm_gemm_pair_parts_of": [c_int, c_int],
         "sllm_gemm_pair_splits": [c_int, c_int],
@@ -104,7 +105,7 @@ def _declare(L):
         "sllm_linear_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "sllm_linear_ws_supports": [c_int, c_int, c_int],
         "sllm_linear_ws": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                           c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+                           c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_linear_ws_parts": [c_int, c_int],
         "sllm_linear_stream_silu_scaled": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int,
                                            c_void_p],
@@ -118,7 +119,7 @@ def _declare(L):
                                c_int, c_void_p],
         "sllm_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                               c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p],
+                               c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p],
         "sllm_attention_mma_pooled": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
                                       c_int, c_int, c_int,
@@ -147,6 +148,10 @@ def _declare(L):
                             c_int, c_int, c_int, c_void_p],
         "sllm_decay_linear_attention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_retention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_softcap": [c_void_p, ctypes.c_longlong, c_float, c_void_p],
+        "sllm_plain_act": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_latent_rope_write": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_head_linear_strided": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,

@@ -199,6 +199,16 @@ class OwedNorm:
         return self.norm.add_norm(self.residual, None)
 
 
+@dataclass
+class StreamCopy:
+    """What a block whose readers take the stream as it is hands to the next one of its kind: the (complete) stream in the
+    compute dtype, written by the kernel that completed it."""
+    x: torch.Tensor
+
+
+COMPLETE = (OwedNorm, StreamCopy)           # hand-overs behind which nothing is left to add to the stream
+
+
 # ---- registries ---------------------------------------------------------------
 
 class Registry:

@@ -141,6 +141,74 @@ class DecayLinearAttention(Mixer):
         return self.inp.nbytes() + self.out.nbytes() + 4 * self.gain.numel() + 4 * self.heads
 
 
+@MIXERS.register("retention")
+class Retention(Mixer):
+    """Retention: linear attention with one fixed decay per head on rotated queries and keys,
+
+        S_t = decay_h S_(t-1) + k_t v_t^T,        o_t = S_t^T q_t
+
+    with q = W_q x and k = W_k x (heads x dim), both rotated by position over their first ``rotary_dim`` channels, k then times
+    dim^(-1/2), and v = W_v x (heads x vdim).  Each head's o over its root mean square (no gain), times silu(W_g x), then W_o.
+    Parameters: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``decay`` (one number per head), ``rotary`` (None, or ``theta``,
+    ``rotary_dim``, ``max_positions``), ``eps`` (of the heads' norm).  q, k, v and the gate are one matrix whose product stays
+    float32; rotation and scale happen in the recurrence kernel's loader."""
+
+    NAMES = ("q", "k", "v", "g")
+
+    def __init__(self, params, **kw):
+        super().__init__(params, **kw)
+        self.hidden = int(params["hidden_size"])
+        self.heads = int(params["heads"])
+        self.dim = int(params["dim"])
+        self.vdim = int(params["vdim"])
+        self.eps = float(params["eps"])
+        decay = [float(d) for d in params["decay"]]
+        if len(decay) != self.heads:
+            raise ValueError(f"retention: {len(decay)} decays for {self.heads} heads")
+        if not ops.delta_rule_supports(self.dim, self.vdim):
+            raise ValueError(f"retention: a head of {self.dim} key channels is outside what the recurrence kernel keeps in registers (1..256)")
+        rot = params.get("rotary")
+        self.rot_params = dict(rot) if rot else None
+        self.rot = int(rot["rotary_dim"]) if rot else 0
+        if self.rot % 2 or self.rot > self.dim:
+            raise ValueError(f"retention: {self.rot} rotated channels must be even and at most dim={self.dim}")
+        self.decay = torch.tensor(decay, dtype=torch.float32).to(self.device)
+        self.rotary = None
+
+    def cache_need(self):
+        return SlotState((self.heads, self.dim, self.vdim), "retention")
+
+    def tensor_specs(self):
+        H, W = self.heads, self.hidden
+        K, V = H * self.dim, H * self.vdim
+        return [TensorSpec("q", (K, W)), TensorSpec("k", (K, W)), TensorSpec("v", (V, W)), TensorSpec("g", (V, W)),
+                TensorSpec("o", (W, V))]
+
+    def bind(self, fetch):
+        K, V = self.heads * self.dim, self.heads * self.vdim
+        self.inp = Linear(self._matrix(torch.cat([fetch(n) for n in self.NAMES], dim=0)))
+        self.offs = (0, K, 2 * K)
+        self.off_g = 2 * K + V
+        self.out = Linear(self._matrix(fetch("o")))
+        if self.rot_params is not None:
+            from .side_by_side import rotary_for
+            self.rotary = rotary_for(self.rot_params, self.dtype, self.device)
+
+    accepts_residual = True
+
+    def mix(self, x, step: StepContext, cache: LayerCache, position=None, write_cache=True):
+        proj = self.inp(x, torch.float32)                                            # [T, 2K + 2V] float32
+        o = ops.retention(proj, self.offs, self.decay, self.rotary.table if self.rotary is not None else None, self.rot,
+                          self.dim ** -0.5, cache.states["retention"], step, self.heads, self.dim, self.vdim)
+        return ops.delta_out(o, None, proj, self.off_g, self.eps, self.heads, self.vdim, self.dtype, "silu")
+
+    def forward(self, x, step, cache, position, write_cache=True, residual=None):
+        return self.out.into(self.mix(x, step, cache, position, write_cache), residual)
+
+    def weight_bytes(self):
+        return self.inp.nbytes() + self.out.nbytes() + 4 * self.heads
+
+
 @MIXERS.register("forget_gate_attention")
 class ForgetGateAttention(Mixer):
     """Linear attention whose forget gate also decides what is written (HGRN2):

@@ -12,7 +12,7 @@ import numpy as np
 import torch
 
 from .. import ops
-from .base import (BLOCKS, FEED_FORWARDS, NORMS, POSITIONS, SHIFTS, FeedForward, Norm, OwedNorm, Part,
+from .base import (BLOCKS, COMPLETE, FEED_FORWARDS, NORMS, POSITIONS, SHIFTS, FeedForward, Norm, Part,
                    PositionEncoding, SlotState, TensorSpec, flatten_needs)
 from .standard import Linear
 
@@ -66,8 +66,8 @@ class GroupRMSNorm(Norm):
 
 def pending_terms(delta) -> list:
     """The terms a block before has left to be added: nothing, one tensor (possibly a stack of partial sums), a
-    sequence of such, or a norm still owed (whose stream is complete: nothing to add)."""
-    if delta is None or isinstance(delta, OwedNorm):
+    sequence of such, or a hand-over whose stream is complete (a norm still owed, a copy of the stream: nothing to add)."""
+    if delta is None or isinstance(delta, COMPLETE):
         return []
     if isinstance(delta, (tuple, list)):
         return [d for d in delta if d is not None]
@@ -152,6 +152,41 @@ class GatedDense(FeedForward):
 
     def weight_bytes(self):
         return self.gate_up.nbytes() + self.down.nbytes()
+
+
+@FEED_FORWARDS.register("plain_dense")
+class PlainDense(FeedForward):
+    """down(act(up(x))): two matrices without biases and an activation between them, ``relu2`` (max(z, 0)^2).  The activation
+    leaves with the first product's tile where that product's kernel has it (`ops.linear_plain_act`)."""
+
+    ACTIVATIONS = ("relu2",)
+
+    def __init__(self, params, **kw):
+        super().__init__(params, **kw)
+        self.hidden = int(params["hidden_size"])
+        self.inter = int(params["intermediate_size"])
+        self.act = str(params.get("activation", "relu2"))
+        self.names = params.get("names", ("up", "down"))
+        if self.act not in self.ACTIVATIONS:
+            raise ValueError(f"plain_dense: activation {self.act!r}; known: {list(self.ACTIVATIONS)}")
+        self.up = None
+        self.down = None
+
+    def tensor_specs(self):
+        u, d = self.names
+        return [TensorSpec(u, (self.inter, self.hidden)), TensorSpec(d, (self.hidden, self.inter))]
+
+    def bind(self, fetch):
+        u, d = self.names
+        self.up, self.down = Linear(self._matrix(fetch(u))), Linear(self._matrix(fetch(d)))
+
+    accepts_residual = True
+
+    def forward(self, x, step, residual=None):
+        return self.down.into(ops.linear_plain_act(x, self.up.weight, self.dtype, self.act), residual)
+
+    def weight_bytes(self):
+        return self.up.nbytes() + self.down.nbytes()
 
 
 @BLOCKS.register("parallel_shift")

@@ -20,7 +20,7 @@ from dataclasses import dataclass
 import torch
 
 from .. import ops
-from .base import BLOCKS, NORMS, SHIFTS, Norm, OwedNorm, Part, SlotState, TensorSpec, flatten_needs
+from .base import BLOCKS, COMPLETE, NORMS, SHIFTS, Norm, Part, SlotState, TensorSpec, flatten_needs
 
 
 @NORMS.register("scalar_rmsnorm")
@@ -44,7 +44,7 @@ class ScalarRMSNorm(Norm):
     def add_norm(self, residual, delta):
         if isinstance(delta, Pending):        # (made for another reader: the term joins the stream here)
             return ops.post_add_norm(residual, delta.term, delta.post.weight, delta.post.eps, self.weight, self.eps, self.dtype)
-        if delta is not None and not isinstance(delta, OwedNorm):
+        if delta is not None and not isinstance(delta, COMPLETE):
             ops.add_group_ssq(residual, [delta], 1, self.eps, want_rinv=False)
         return ops.post_add_norm(residual, None, None, 0.0, self.weight, self.eps, self.dtype)
 
@@ -154,7 +154,7 @@ class SandwichBlock:
         term = post = None
         if isinstance(delta, Pending):
             term, post = delta.term, delta.post
-        elif delta is not None and not isinstance(delta, OwedNorm):
+        elif delta is not None and not isinstance(delta, COMPLETE):
             ops.add_group_ssq(residual, [delta], 1, norm.eps, want_rinv=False)
         h = self._read(residual, term, post, norm, self.mixer_conv, cache, "conv_mixer", step)
         term = self.mixer.forward(h, step, cache, position, write_cache)

@@ -1,9 +1,10 @@
 """Two mixers side by side on one input, and the attention one of them usually is.
 
 `NormedAttention`: grouped-query softmax attention over the paged cache whose query and key heads are RMS-normed (one
-gain of the head's size, shared by the heads) before they are rotated; it owns its rotary table (each layer may have
+gain of the head's size, shared by the heads, or none) before they are rotated; it owns its rotary table (each layer may have
 other frequencies, and a two-regime frequency scaling); a query may be restricted to the keys of its own block of
-positions; the value size may differ from the key size.
+positions; the value size may differ from the key size; scores may be capped, a head's output gated, and the keys and values
+another layer's.
 
 `SideBySide`: both mixers read the same input; the layer's term is the mean of their outputs, each first RMS-normed over
 the model width with a gain of its own.
@@ -41,7 +42,11 @@ class NormedAttention(Mixer):
     """Parameters: ``hidden_size``, ``heads``, ``kv_heads``, ``dim`` (query/key size of a head), ``vdim`` (value size),
     ``scale`` (of the scores), ``eps`` (of the head norms), ``rotary`` (None, or ``theta``, ``rotary_dim``, optional
     ``scaling``: see `parts.standard.Rotary`), ``block`` (None, or the size of the blocks of positions, counted from 0,
-    inside which a query sees the keys at or before it), ``max_positions``.
+    inside which a query sees the keys at or before it), ``max_positions``.  Optional: ``head_gain`` (default true; false: the head
+    norms have no gain, so that norming before or after the rotation is the same), ``softcap`` (scores become softcap
+    tanh(score / softcap)), ``head_gate`` (true: a matrix ``g`` with a row per query head, whose output is multiplied by
+    sigmoid(g x)_h), ``shared_kv`` (true: the layer has no keys and values of its own and reads the cache another run wrote).
+    All of the layer's input matrices are one product.
 
     The cache's head holds max(dim, vdim) channels (rounded up to a size the tensor-core kernels take, in bfloat16):
     keys and values are stored with zeros beyond their own size, which neither scores nor sums see; the output
@@ -59,6 +64,10 @@ class NormedAttention(Mixer):
         self.eps = float(p["eps"])
         self.block = int(p["block"]) if p.get("block") else None
         self.max_positions = int(p["max_positions"])
+        self.head_gain = bool(p.get("head_gain", True))
+        self.softcap = float(p.get("softcap") or 0.0)
+        self.head_gate = bool(p.get("head_gate", False))
+        self.shared_kv = bool(p.get("shared_kv", False))
         rot = p.get("rotary")
         self.rot_params = dict(rot, max_positions=self.max_positions) if rot else None
         self.rot = int(rot["rotary_dim"]) if rot else 0
@@ -79,13 +88,26 @@ class NormedAttention(Mixer):
 
     def tensor_specs(self):
         W = self.hidden
-        return [TensorSpec("q", (self.nq * self.dim, W)), TensorSpec("k", (self.nkv * self.dim, W)),
-                TensorSpec("v", (self.nkv * self.vdim, W)), TensorSpec("q.norm", (self.dim,), role="gain"),
-                TensorSpec("k.norm", (self.dim,), role="gain"), TensorSpec("o", (W, self.nq * self.vdim))]
+        specs = [TensorSpec("q", (self.nq * self.dim, W))]
+        if not self.shared_kv:
+            specs += [TensorSpec("k", (self.nkv * self.dim, W)), TensorSpec("v", (self.nkv * self.vdim, W))]
+        if self.head_gain:
+            specs.append(TensorSpec("q.norm", (self.dim,), role="gain"))
+            if not self.shared_kv:
+                specs.append(TensorSpec("k.norm", (self.dim,), role="gain"))
+        if self.head_gate:
+            specs.append(TensorSpec("g", (self.nq, W)))
+        return specs + [TensorSpec("o", (W, self.nq * self.vdim))]
 
     def bind(self, fetch):
-        self.qkv = Linear(self._matrix(torch.cat([fetch(n) for n in ("q", "k", "v")], dim=0)))
-        self.q_gain, self.k_gain = self._f32(fetch("q.norm")), self._f32(fetch("k.norm"))
+        names = ["q"] + ([] if self.shared_kv else ["k", "v"]) + (["g"] if self.head_gate else [])
+        self.qkv = Linear(self._matrix(torch.cat([fetch(n) for n in names], dim=0)))
+        self.off_g = self.nq * self.dim + (0 if self.shared_kv else self.nkv * (self.dim + self.vdim))
+        if self.head_gain:
+            self.q_gain = self._f32(fetch("q.norm"))
+            self.k_gain = self._f32(fetch("k.norm")) if not self.shared_kv else self.q_gain
+        else:
+            self.q_gain = self.k_gain = torch.ones(self.dim, dtype=torch.float32).to(self.device)
         o = fetch("o")
         if self.D != self.vdim:
             wide = torch.zeros((self.hidden, self.nq, self.D), dtype=o.dtype)
@@ -99,11 +121,13 @@ class NormedAttention(Mixer):
 
     def mix(self, x, step: StepContext, cache: LayerCache, position=None, write_cache=True):
         g = step.groups[cache.group]
-        qkv = self.qkv(x, torch.float32)                                             # [T, (nq+nkv) dim + nkv vdim] float32
+        qkv = self.qkv(x, torch.float32)                                             # [T, (nq+nkv) dim + nkv vdim (+ nq)] float32
+        write_cache = write_cache and not self.shared_kv
         q = ops.qk_norm_rope_kv_write(qkv, self.q_gain, self.k_gain, self.eps, step.positions,
                                       self.rotary.table if self.rotary is not None else None, self.rot, self.nq, self.nkv,
                                       self.dim, self.vdim, g.slot_mapping if write_cache else None, cache.k, cache.v, self.dtype)
-        return ops.paged_attention(q, cache.k, cache.v, step, cache.group, self.nq, self.nkv, self.D, self.scale, None, self.block)
+        return ops.paged_attention(q, cache.k, cache.v, step, cache.group, self.nq, self.nkv, self.D, self.scale, None, self.block,
+                                   softcap=self.softcap, gate=(qkv, self.off_g) if self.head_gate else None)
 
     def forward(self, x, step, cache, position, write_cache=True, residual=None):
         return self.out.into(self.mix(x, step, cache, position, write_cache), residual)

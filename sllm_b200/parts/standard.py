@@ -13,7 +13,7 @@ import torch
 from .. import ops
 from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, FeedForward,
                    LayerCache, Mixer, Norm, OwedNorm, PagedKV, Part, PositionEncoding,
-                   StepContext, TensorSpec)
+                   StepContext, StreamCopy, TensorSpec)
 
 
 class Linear:
@@ -320,6 +320,8 @@ class PreNormBlock:
         that cannot take it asks for the plain form itself), anything else through the norm's kernel."""
         if isinstance(delta, OwedNorm):
             return delta if delta.norm is norm else norm.add_norm(residual, None)
+        if isinstance(delta, StreamCopy):
+            delta = None
         return norm.add_norm(residual, delta)
 
     def forward(self, residual, delta, step, cache, position, write_cache=True, next_norm=None):

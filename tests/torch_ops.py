@@ -105,7 +105,7 @@ def delta_out(o, gain, proj, off_g, eps, heads, dv, out_dtype, gate_act="sigmoid
     else:
         g = proj[:, off_g:off_g + heads * dv]
         gate = torch.sigmoid(g) if gate_act == "sigmoid" else g * torch.sigmoid(g)
-    y = x.reshape(T, heads * dv) * gain * gate
+    y = x.reshape(T, heads * dv) * (1.0 if gain is None else gain) * gate
     if out is None:
         return y.to(out_dtype)
     out[:, out_off:out_off + heads * dv] = y.to(out.dtype)
@@ -194,6 +194,8 @@ def qk_norm_rope_kv_write(qkv, q_gain, k_gain, eps, positions, table, rotary_dim
     qkv = qkv[:, col_off:]
     T = qkv.shape[0]
     D = k_cache.shape[3]
+    if slot_mapping is None:           # queries alone: the product may hold no keys and values
+        nkv = 0
     qk = qkv[:, :(nq + nkv) * dim].float().reshape(T, nq + nkv, dim)
     v = qkv[:, (nq + nkv) * dim:(nq + nkv) * dim + nkv * vdim].float().reshape(T, nkv, vdim)
     if q_gain is not None:
@@ -381,6 +383,28 @@ def post_add_norm(stream, term, post_gain, post_eps, pre_gain, pre_eps, out_dtyp
     return (stream * (stream.pow(2).mean(-1, keepdim=True) + pre_eps).rsqrt() * pre_gain).to(out_dtype)
 
 
+def post_add_copy(stream, term, post_gain, post_eps, out_dtype=None):
+    post_add_norm(stream, term, post_gain, post_eps, None, 0.0)
+    if out_dtype is None:
+        return None
+    return stream if out_dtype == torch.float32 else stream.to(out_dtype)
+
+
+def softcap_(x, cap):
+    return x.copy_(cap * torch.tanh(x / cap))
+
+
+def plain_act(x, out_dtype, act, token=None):
+    if act == "relu2":
+        return torch.relu(x.float()).square().to(out_dtype)
+    e = token.table[token.ids.long(), token.off:token.off + x.shape[1]].float()
+    return (torch.nn.functional.gelu(x.float(), approximate="tanh") * e).to(out_dtype)
+
+
+def linear_plain_act(x, w, out_dtype, act, token=None):
+    return plain_act(linear(x, w, None, torch.float32), out_dtype, act, token)
+
+
 def post_add_norm_conv(stream, term, post_gain, post_eps, pre_gain, pre_eps, weight, state, step, out_dtype):
     assert stream.shape[0] == step.num_seqs, "one token a request"
     h = post_add_norm(stream, term, post_gain, post_eps, pre_gain, pre_eps, torch.float32)
@@ -409,6 +433,22 @@ def decay_linear_attention(proj, offs, decay, state, step, heads, dk, dv):
     q = act(proj[:, off_q:off_q + heads * dk]).reshape(T, heads, dk)
     k = act(proj[:, off_k:off_k + heads * dk]).reshape(T, heads, dk)
     v = act(proj[:, off_v:off_v + heads * dv]).reshape(T, heads, dv)
+    out = torch.empty((T, heads, dv), dtype=torch.float32, device=proj.device)
+
+    def token(t, S):
+        S = decay[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        return S, torch.einsum("hij,hi->hj", S, q[t])
+    _walk(step, state, out, token)
+    return out.reshape(T, heads * dv)
+
+
+def retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv):
+    T = proj.shape[0]
+    off_q, off_k, off_v = offs
+    rot = rotary_dim if table is not None else 0
+    q = _rotate(proj[:, off_q:off_q + heads * dk].reshape(T, heads, dk), step.positions, table, rot)
+    k = _rotate(proj[:, off_k:off_k + heads * dk].reshape(T, heads, dk), step.positions, table, rot) * k_scale
+    v = proj[:, off_v:off_v + heads * dv].reshape(T, heads, dv)
     out = torch.empty((T, heads, dv), dtype=torch.float32, device=proj.device)
 
     def token(t, S):
@@ -480,7 +520,8 @@ def rope_kv_write(qkv, bias, positions, table, rotary_dim, nq, nkv, hd, slot_map
     return q
 
 
-def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None):
+def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None,
+                   softcap=0.0, gate=None):
     T = q.shape[0]
     ps = k_cache.shape[2]
     out = torch.empty((T, nq, hd), dtype=torch.float32, device=q.device)
@@ -498,18 +539,22 @@ def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, n
         k = k.repeat_interleave(rep, dim=1)
         v = v.repeat_interleave(rep, dim=1)
         s = torch.einsum("hd,nhd->hn", qf[t], k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         if sink is not None:                               # one more term of the denominator: no key, no value, not scaled
             p = torch.softmax(torch.cat([s, sink.float()[:, None]], dim=-1), dim=-1)[:, :-1]
         else:
             p = torch.softmax(s, dim=-1)
         out[t] = torch.einsum("hn,nhd->hd", p, v)
+        if gate is not None:
+            out[t] *= torch.sigmoid(gate[0][t, gate[1]:gate[1] + nq])[:, None]
     return out.reshape(T, nq * hd).to(q.dtype)
 
 
-def paged_attention(q, k_cache, v_cache, step, group, nq, nkv, hd, scale, window, block=None, sink=None):
+def paged_attention(q, k_cache, v_cache, step, group, nq, nkv, hd, scale, window, block=None, sink=None, softcap=0.0, gate=None):
     g = step.groups[group]
     return attention_simt(q, k_cache, v_cache, g.block_tables, step.positions, step.seq_of_token,
-                          nq, nkv, hd, scale, window, block, sink)
+                          nq, nkv, hd, scale, window, block, sink, softcap, gate)
 
 
 def pool_kv_write(k_cache, v_cache, step, group, pk_cache, pv_cache, pool_group, pool):
@@ -607,7 +652,7 @@ def penalty_from_seen_(logits, seen, step, penalty):
     return logits
 
 
-ALL = ["forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
+ALL = ["retention", "post_add_copy", "softcap_", "plain_act", "linear_plain_act", "forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
        "decay_linear_attention", "gated_delta_rule", "gated_linear_attention", "qk_norm_rope_kv_write", "short_conv_silu", "norm_mean_add_", "moe_route", "moe_act",
        "add_sinusoid_", "add_group_ssq", "group_norm_shift", "act_mul", "linear_act_mul", "tanh_cols", "delta_rule", "delta_out", "latent_write",
        "head_linear", "embed_gather", "add_rmsnorm", "linear", "can_accumulate", "linear_accumulate", "silu_mul", "linear_silu_mul", "rope_kv_write",
