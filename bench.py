@@ -473,6 +473,27 @@ def gerupel_config(sz: dict) -> dict:
             "layers": [layer for _ in range(n if sz["layers"] >= 4 else sz["layers"])]}
 
 
+def sezopel_config(sz: dict) -> dict:
+    """Sezopel at one size: the same width, depth and vocabulary; layers go round attention with keys and values of its own
+    (an eighth of the heads as kv heads, half the head rotated, scores capped), retention (heads of 64 x 64, the state of
+    Kidolorn's fixed-decay heads), attention that reads the first one's cache, retention; the two-matrix feed-forward is half as
+    wide again as the gated one of the other designs (as many weights); 256 channels of the token's own vector per layer."""
+    W, H, D = sz["width"], sz["heads"], sz["dim"]
+    mlp = {"kind": "dense", "ff": sz["ff"] * 3 // 2 // 64 * 64}
+    heads = W // 64
+    decay = [1.0 - 2.0 ** (-5.0 - 5.0 * h / max(heads - 1, 1)) for h in range(heads)]
+    attention = {"heads": H, "kv_heads": max(1, H // 8), "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 30.0,
+                 "rot": {"base": 10000.0, "dims": D // 2}}
+    retention = {"type": "retention", "mlp": mlp, "mixer": {"heads": heads, "dim": 64, "vdim": 64, "decay": decay,
+                                                            "rot": {"base": 10000.0, "dims": 64}}}
+    layers = []
+    for i in range(sz["layers"]):
+        m = dict(attention, kv_from=i - 2) if i % 4 == 2 else attention
+        layers.append(retention if i % 2 else {"type": "attention", "mixer": m, "mlp": mlp})
+    return {"architecture": "Sezopel", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "token_side": {"dim": 256}, "logit_softcap": 30.0, "layers": layers}
+
+
 def design_run(args) -> dict:
     global PREFILL_TOKENS
     import torch
@@ -493,6 +514,9 @@ def design_run(args) -> dict:
         if args.workload == "gerupel":
             # beside Nutopel (attention next to a matrix-state recurrence, experts) and Qwen2 (grouped-query attention)
             designs = [("gerupel", gerupel_config(sz)), ("nutopel", nutopel_config(sz)), designs[-1]]
+        if args.workload == "sezopel":
+            # beside Kidolorn (fixed-decay linear attention, norms behind the sublayers) and Qwen2 (grouped-query attention)
+            designs = [("sezopel", sezopel_config(sz)), ("kidolorn", kidolorn_config(sz)), designs[-1]]
         for which, config in designs:
             model, _ = build_random_model(config, seed=0, dtype="bfloat16", device="cuda:0", std=0.02)
             cfg = {"vocab_size": sz["vocab"]}
@@ -767,7 +791,7 @@ def base_config(cfg, args, prompt_len) -> dict:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", choices=("decode", "rososun", "nutopel", "kidolorn", "gerupel") + tuple(SERVING), default="decode",
+    ap.add_argument("--workload", choices=("decode", "rososun", "nutopel", "kidolorn", "gerupel", "sezopel") + tuple(SERVING), default="decode",
                     help="decode: the default run; serve-*: the baseline's serving workloads through LLM.generate")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=32)
@@ -806,7 +830,7 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         print(json.dumps({"error": "no CUDA device"}))
         return 1
-    if args.workload in ("rososun", "nutopel", "kidolorn", "gerupel"):
+    if args.workload in ("rososun", "nutopel", "kidolorn", "gerupel", "sezopel"):
         print(json.dumps(design_run(args)))
         return 0
     if args.workload != "decode":

@@ -72,6 +72,7 @@ struct DeltaParams {
   const float* table = nullptr;        // [max_pos][2][rot / 2], cos then sin
   int rot = 0, max_pos = 0;
   float k_scale = 1.f;
+  int max_len = 0;                     // > 0: requests that bring more tokens are another kernel's (retention.cu)
 };
 
 // RPT: rows of a column per lane (dk <= 8 * RPT = DKP, the padded key size).
@@ -87,6 +88,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
   pdl_wait();
   const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS;
   const int t_begin = p.q_start[seq], t_end = p.q_start[seq + 1];
+  if (p.max_len > 0 && t_end - t_begin > p.max_len) return;
   const int tid = threadIdx.x, lane = tid & 31;
   const bool loader = tid >= DR_COMPUTE;
   const int nchunks = (t_end - t_begin + chunk - 1) / chunk;
@@ -446,13 +448,17 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
 template <typename TO>
 __global__ void delta_out_kernel(const float* __restrict__ o, const float* __restrict__ gain, const float* __restrict__ proj,
                                  int ld, int off_g, float eps, TO* __restrict__ out, int rows, int H, int dv, int gate_act,
-                                 int out_ld, int out_off) {
+                                 int out_ld, int out_off, const int* __restrict__ seq_of_token, const int* __restrict__ q_start, int max_len) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);     // (t, h)
   if (row >= rows) return;
   const int t = row / H, h = row % H;
+  if (max_len > 0) {                    // rows of requests with longer portions are another kernel's
+    const int seq = seq_of_token[t];
+    if (q_start[seq + 1] - q_start[seq] > max_len) return;
+  }
   const float* x = o + (size_t)row * dv;
   float ss = 0.f;
   for (int j = lane; j < dv; j += 32) ss = fmaf(x[j], x[j], ss);
@@ -469,12 +475,17 @@ __global__ void delta_out_kernel(const float* __restrict__ o, const float* __res
 template <typename TO>
 __global__ void __launch_bounds__(256)
 delta_out_wide_kernel(const float* __restrict__ o, const float* __restrict__ gain, const float* __restrict__ proj, int ld, int off_g,
-                      float eps, TO* __restrict__ out, int H, int dv, int gate_act, int out_ld, int out_off) {
+                      float eps, TO* __restrict__ out, int H, int dv, int gate_act, int out_ld, int out_off, const int* __restrict__ seq_of_token,
+                      const int* __restrict__ q_start, int max_len) {
   __shared__ float red[33];
   pdl_launch_dependents();
   pdl_wait();
   const size_t row = blockIdx.x;
   const int t = (int)(row / H), h = (int)(row % H);
+  if (max_len > 0) {
+    const int seq = seq_of_token[t];
+    if (q_start[seq + 1] - q_start[seq] > max_len) return;
+  }
   const float* x = o + row * dv;
   float ss = 0.f;
   for (int j = threadIdx.x; j < dv; j += blockDim.x) ss = fmaf(x[j], x[j], ss);
@@ -627,10 +638,11 @@ SLLM_EXPORT int sllm_forget_gate_attention(const float* proj, int ld, int off_q,
 }
 
 // Retention (a fixed decay per head, `decay` [H]; q and k rotated by position, k times k_scale) over q | k | v columns of
-// `proj` [T, ld]; rot == 0: no rotation, positions and table unused.
+// `proj` [T, ld]; rot == 0: no rotation, positions and table unused.  max_len > 0: requests that bring more tokens are left alone.
 SLLM_EXPORT int sllm_retention(const float* proj, int ld, int off_q, int off_k, int off_v, const float* decay, const int* positions,
                                const float* table, int rot, int max_pos, float k_scale, float* state, const int* q_start,
-                               const int* state_slots, float* out, int S, int H, int dk, int dv, int max_q, cudaStream_t stream) {
+                               const int* state_slots, float* out, int S, int H, int dk, int dv, int max_q, int max_len,
+                               cudaStream_t stream) {
   SLLM_REQUIRE(S >= 0 && H > 0 && H <= 65535, "retention: bad sizes S=%d H=%d", S, H);
   SLLM_REQUIRE(sllm_delta_rule_supports(dk, dv), "retention: a head of %d key and %d value channels is outside 1..256 keys", dk, dv);
   SLLM_REQUIRE(off_q >= 0 && off_k >= 0 && off_v >= 0 && off_q + H * dk <= ld && off_k + H * dk <= ld && off_v + H * dv <= ld,
@@ -645,31 +657,35 @@ SLLM_EXPORT int sllm_retention(const float* proj, int ld, int off_q, int off_k, 
   p.mode = DR_RETENTION; p.hdiv = 1; p.gates = nullptr; p.ldg = p.off_b = p.off_dt = 0; p.a_log = decay; p.dt_bias = nullptr;
   p.r_scale = 1.f; p.inv_tau = 1.f;
   p.positions = positions; p.table = table; p.rot = rot; p.max_pos = max_pos > 0 ? max_pos : 1; p.k_scale = k_scale;
+  p.max_len = max_len;
+  if (max_len > 0 && (p.max_q <= 0 || p.max_q > max_len)) p.max_q = max_len;
   return dispatch_delta_rule(p, S, stream);
 }
 
 SLLM_EXPORT int sllm_delta_out(const float* o, const float* gain, const float* proj, int ld, int off_g, float eps, void* out,
-                               int out_dtype, int T, int H, int dv, int gate_act, int out_ld, int out_off, cudaStream_t stream) {
+                               int out_dtype, int T, int H, int dv, int gate_act, int out_ld, int out_off, const int* seq_of_token, const int* q_start,
+                               int max_len, cudaStream_t stream) {
+  SLLM_REQUIRE(max_len == 0 || (seq_of_token && q_start), "delta_out: leaving rows out needs the batch's description");
   SLLM_REQUIRE(out_off >= 0 && out_off + H * dv <= out_ld, "delta_out: the output's columns lie outside its %d", out_ld);
   SLLM_REQUIRE(T >= 0 && H > 0 && dv > 0 && (gate_act == 2 || (off_g >= 0 && off_g + H * dv <= ld)), "delta_out: bad sizes T=%d H=%d dv=%d", T, H, dv);
   if (T == 0) return SLLM_OK;
   const long rows = (long)T * H;
   if (dv >= 512) {                      // a warp would walk such a row sixteen times and more
     if (out_dtype == SLLM_F32)
-      launch_kernel(delta_out_wide_kernel<float>, (unsigned)rows, 256, 0, stream, o, gain, proj, ld, off_g, eps, (float*)out, H, dv, gate_act, out_ld, out_off);
+      launch_kernel(delta_out_wide_kernel<float>, (unsigned)rows, 256, 0, stream, o, gain, proj, ld, off_g, eps, (float*)out, H, dv, gate_act, out_ld, out_off, seq_of_token, q_start, max_len);
     else if (out_dtype == SLLM_BF16)
       launch_kernel(delta_out_wide_kernel<__nv_bfloat16>, (unsigned)rows, 256, 0, stream, o, gain, proj, ld, off_g, eps,
-                    (__nv_bfloat16*)out, H, dv, gate_act, out_ld, out_off);
+                    (__nv_bfloat16*)out, H, dv, gate_act, out_ld, out_off, seq_of_token, q_start, max_len);
     else
       SLLM_REQUIRE(false, "delta_out: unknown dtype %d", out_dtype);
     return launch_status("delta_out");
   }
   const int blocks = (int)((rows + 7) / 8);
   if (out_dtype == SLLM_F32)
-    launch_kernel(delta_out_kernel<float>, blocks, 256, 0, stream, o, gain, proj, ld, off_g, eps, (float*)out, (int)rows, H, dv, gate_act, out_ld, out_off);
+    launch_kernel(delta_out_kernel<float>, blocks, 256, 0, stream, o, gain, proj, ld, off_g, eps, (float*)out, (int)rows, H, dv, gate_act, out_ld, out_off, seq_of_token, q_start, max_len);
   else if (out_dtype == SLLM_BF16)
     launch_kernel(delta_out_kernel<__nv_bfloat16>, blocks, 256, 0, stream, o, gain, proj, ld, off_g, eps, (__nv_bfloat16*)out,
-                  (int)rows, H, dv, gate_act, out_ld, out_off);
+                  (int)rows, H, dv, gate_act, out_ld, out_off, seq_of_token, q_start, max_len);
   else
     SLLM_REQUIRE(false, "delta_out: unknown dtype %d", out_dtype);
   return launch_status("delta_out");

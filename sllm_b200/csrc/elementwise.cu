@@ -386,16 +386,18 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, siz
 }
 
 // ---------------------------------------------------------------------------
-// out[t, n] = max(x, 0)^2, or gelu_tanh(x) * table[ids[t], off + n]: behind products whose kernel has no such epilogue
+// out[t, n] = max(x, 0)^2, or gelu_tanh(x) * table[ids[t], off + n]: behind products whose kernel has no such epilogue; x may
+// be a stack of k-split partial sums
 // ---------------------------------------------------------------------------
 template <typename TI, typename TT, typename TO>
 __global__ void __launch_bounds__(256)
-plain_act_kernel(const TI* __restrict__ x, TO* __restrict__ out, int T, int N, int act, const TokenTable token) {
+plain_act_kernel(const TI* __restrict__ x, int parts, size_t part_stride, TO* __restrict__ out, int T, int N, int act, const TokenTable token) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t total = (size_t)T * N;
   for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
-    const float v = to_f32(x[e]);
+    float v = to_f32(x[e]);
+    for (int p = 1; p < parts; ++p) v += to_f32(x[p * part_stride + e]);
     float y;
     if (act == SLLM_ACT_RELU2) {
       y = relu2_f32(v);
@@ -546,9 +548,9 @@ SLLM_EXPORT int sllm_softcap(float* x, long long n, float cap, cudaStream_t stre
 }
 
 // act: SLLM_ACT_RELU2, or SLLM_ACT_TOKEN with a table of the output's dtype
-SLLM_EXPORT int sllm_plain_act(const void* x, int in_dtype, void* out, int out_dtype, int T, int N, int act, const void* token_table,
+SLLM_EXPORT int sllm_plain_act(const void* x, int in_dtype, int parts, size_t part_stride, void* out, int out_dtype, int T, int N, int act, const void* token_table,
                                const int* token_ids, int token_off, int token_ld, int token_rows, cudaStream_t stream) {
-  SLLM_REQUIRE(T >= 0 && N > 0 && (act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN), "plain_act: bad sizes T=%d N=%d act=%d", T, N, act);
+  SLLM_REQUIRE(T >= 0 && N > 0 && parts >= 1 && (act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN), "plain_act: bad sizes T=%d N=%d act=%d", T, N, act);
   SLLM_REQUIRE(act != SLLM_ACT_TOKEN || (token_table && token_ids && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld),
                "plain_act: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
   if (T == 0) return SLLM_OK;
@@ -556,7 +558,7 @@ SLLM_EXPORT int sllm_plain_act(const void* x, int in_dtype, void* out, int out_d
   tt.table = token_table; tt.ids = token_ids; tt.off = token_off; tt.ld = token_ld; tt.V = token_rows;
   const size_t total = (size_t)T * N;
   const unsigned blocks = (unsigned)((total + 255) / 256 > 8192 ? 8192 : (total + 255) / 256);
-#define PA(TI_, TO_) launch_kernel(plain_act_kernel<TI_, TO_, TO_>, blocks, 256, 0, stream, (const TI_*)x, (TO_*)out, T, N, act, tt)
+#define PA(TI_, TO_) launch_kernel(plain_act_kernel<TI_, TO_, TO_>, blocks, 256, 0, stream, (const TI_*)x, parts, part_stride, (TO_*)out, T, N, act, tt)
   if (in_dtype == SLLM_F32 && out_dtype == SLLM_F32) PA(float, float);
   else if (in_dtype == SLLM_F32 && out_dtype == SLLM_BF16) PA(float, __nv_bfloat16);
   else if (in_dtype == SLLM_BF16 && out_dtype == SLLM_BF16) PA(__nv_bfloat16, __nv_bfloat16);

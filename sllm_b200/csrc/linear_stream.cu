@@ -32,7 +32,6 @@ constexpr int LS_XSTRIDE = LS_KC + 32;     // bf16 elements: 320 bytes, = 64 mod
 
 #define EPI_STORE 0
 #define EPI_SILU 1
-#define EPI_RELU2 3     // a plain result (+bias) through max(v, 0)^2
 #define EPI_GELU 2      // the tanh form of GELU in place of SiLU, gate and up each with its bias
 
 constexpr int LS_SSQ_MAX = 608;            // partial sums of squares per token a scaled launch takes (as in linear_ws.cu)
@@ -222,10 +221,7 @@ linear_stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* _
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int tok = 8 * j + 2 * t4 + (c & 1), row = (c & 2) ? row_b : row_a;
-        if (tok < M && row < N) {
-          const float v = acc[j][c] + (bias ? bias[row] : 0.f);
-          out[(size_t)tok * N + row] = from_f32<OUT>(EPI == EPI_RELU2 ? relu2_f32(v) : v);
-        }
+        if (tok < M && row < N) out[(size_t)tok * N + row] = from_f32<OUT>(acc[j][c] + (bias ? bias[row] : 0.f));
       }
   }
 }
@@ -268,24 +264,22 @@ SLLM_EXPORT int sllm_linear_stream_supports(int M, int N, int K) {
 
 // epilogue 0: out[M, N] (+bias) in out_dtype, or with splits > 1 float32 partial[splits, M, N];
 // epilogue 1: out[M, N/2] = silu(gate) * up for rows interleaved in blocks of 8 (splits must be 1);
-// epilogue 2: the same with gelu_tanh(gate + bias) * (up + bias), the bias interleaved like the rows;
-// epilogue 3: out[M, N] = max(x W^T (+bias), 0)^2, bfloat16 (splits must be 1).
+// epilogue 2: the same with gelu_tanh(gate + bias) * (up + bias), the bias interleaved like the rows.
 SLLM_EXPORT int sllm_linear_stream(const void* x, const void* W, const float* bias, void* out, int out_dtype,
                                    float* partial, int M, int N, int K, int splits, int epilogue,
                                    cudaStream_t stream) {
   SLLM_REQUIRE(sllm_linear_stream_supports(M, N, K), "linear_stream: sizes M=%d N=%d K=%d (needs M<=64, K%%128==0)", M, N, K);
   SLLM_REQUIRE(splits >= 1, "linear_stream: splits=%d", splits);
   SLLM_REQUIRE(splits == 1 || partial != nullptr, "linear_stream: k-splits need scratch");
-  SLLM_REQUIRE(epilogue == EPI_STORE || (splits == 1 && (N % 16 == 0 || epilogue == EPI_RELU2) && out_dtype == SLLM_BF16),
+  SLLM_REQUIRE(epilogue == EPI_STORE || (splits == 1 && N % 16 == 0 && out_dtype == SLLM_BF16),
                "linear_stream: the gated epilogues need splits=1, N%%16==0 and a bfloat16 result");
-  SLLM_REQUIRE(epilogue >= EPI_STORE && epilogue <= EPI_RELU2, "linear_stream: unknown epilogue %d", epilogue);
+  SLLM_REQUIRE(epilogue >= EPI_STORE && epilogue <= EPI_GELU, "linear_stream: unknown epilogue %d", epilogue);
   const __nv_bfloat16* xb = (const __nv_bfloat16*)x;
   const __nv_bfloat16* wb = (const __nv_bfloat16*)W;
   const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : (M <= 32 ? 4 : 8));
 #define GO(NT_)                                                                                              \
   if (epilogue == EPI_SILU) return launch_ls<NT_, EPI_SILU, __nv_bfloat16>(xb, wb, bias, out, partial, M, N, K, splits, stream); \
   if (epilogue == EPI_GELU) return launch_ls<NT_, EPI_GELU, __nv_bfloat16>(xb, wb, bias, out, partial, M, N, K, splits, stream); \
-  if (epilogue == EPI_RELU2) return launch_ls<NT_, EPI_RELU2, __nv_bfloat16>(xb, wb, bias, out, partial, M, N, K, splits, stream); \
   if (out_dtype == SLLM_BF16) return launch_ls<NT_, EPI_STORE, __nv_bfloat16>(xb, wb, bias, out, partial, M, N, K, splits, stream); \
   return launch_ls<NT_, EPI_STORE, float>(xb, wb, bias, out, partial, M, N, K, splits, stream);
   switch (nt) {

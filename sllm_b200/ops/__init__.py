@@ -207,10 +207,11 @@ GATE_ACTS = {"sigmoid": 0, "silu": 1, "none": 2}
 
 
 def delta_out(o, gain, proj, off_g: int, eps: float, heads: int, dv: int, out_dtype, gate_act: str = "sigmoid", out=None,
-              out_off: int = 0) -> torch.Tensor:
+              out_off: int = 0, step=None, max_len: int = 0) -> torch.Tensor:
     """Each head's ``o`` over its root mean square, times ``gain`` (``[heads*dv]``; None: ones), times ``sigmoid`` (or ``silu``) of
     the gate logits (columns ``off_g`` of ``proj``), in ``out_dtype``; with ``gate_act`` ``none`` there is no gate and
-    ``proj`` may be None.  ``out``: a wider tensor whose columns ``out_off ..`` receive the result."""
+    ``proj`` may be None.  ``out``: a wider tensor whose columns ``out_off ..`` receive the result.  ``max_len`` > 0 (with ``step``):
+    rows of requests that bring more tokens are left alone."""
     if gate_act == "none":
         proj, off_g = o, 0
     _chk(o, gain, proj, out)
@@ -218,7 +219,8 @@ def delta_out(o, gain, proj, off_g: int, eps: float, heads: int, dv: int, out_dt
     if out is None:
         out = torch.empty((T, heads * dv), dtype=out_dtype, device=o.device)
     call("sllm_delta_out", _p(o), _p(gain), _p(proj), proj.shape[1], int(off_g), float(eps), _p(out), _dtc(out.dtype), T, heads, dv,
-         GATE_ACTS[gate_act], out.shape[1], int(out_off), _stream())
+         GATE_ACTS[gate_act], out.shape[1], int(out_off), _p(step.seq_of_token) if max_len else None, _p(step.q_start) if max_len else None,
+         int(max_len), _stream())
     return out
 
 
@@ -529,11 +531,13 @@ def decay_linear_attention(proj, offs, decay, state, step, heads: int, dk: int, 
     return out
 
 
-def retention(proj, offs, decay, table, rotary_dim: int, k_scale: float, state, step, heads: int, dk: int, dv: int) -> torch.Tensor:
+def retention(proj, offs, decay, table, rotary_dim: int, k_scale: float, state, step, heads: int, dk: int, dv: int,
+              max_len: int = 0) -> torch.Tensor:
     """S <- decay_h S + k v^T; o = S^T q over the step's tokens from and into ``state`` (float32 ``[slots, heads, dk, dv]``), with
     q and k rotated by position over their first ``rotary_dim`` channels (channel i with i + rotary_dim/2; ``table`` float32
     ``[positions, 2, rotary_dim/2]``, None: no rotation) and k then times ``k_scale``.  ``proj`` float32 ``[T, ld]`` holds q, k, v
-    at columns ``offs``; ``decay`` float32 ``[heads]``.  Returns ``o`` float32 ``[T, heads*dv]``."""
+    at columns ``offs``; ``decay`` float32 ``[heads]``.  Returns ``o`` float32 ``[T, heads*dv]``.  ``max_len`` > 0: requests that bring
+    more tokens are left alone (neither their states nor their rows are touched)."""
     _chk(proj, decay, table, state)
     T, ld = proj.shape
     if proj.dtype != torch.float32 or decay.dtype != torch.float32 or state.dtype != torch.float32:
@@ -547,7 +551,85 @@ def retention(proj, offs, decay, table, rotary_dim: int, k_scale: float, state, 
     off_q, off_k, off_v = (int(o) for o in offs)
     call("sllm_retention", _p(proj), ld, off_q, off_k, off_v, _p(decay), _p(step.positions), _p(table), rot, table.shape[0] if rot else 0,
          float(k_scale), _p(state), _p(step.q_start), _p(step.state_slots), _p(out), step.num_seqs, heads, dk, dv, int(step.max_q_len),
-         _stream())
+         int(max_len), _stream())
+    return out
+
+
+RETENTION_CHUNK = 64           # tokens per chunk of the chunked form (its kernels')
+# Portions of at least so many tokens take it (0: none does).  In a graph, one portion at 32 heads of 64 x 64, us: 64 tokens 19 token by
+# token and 25 in chunks, 128 tokens 31 and 26, 2,048 tokens 525 and 81.
+RETENTION_CHUNKED_FROM = int(os.environ.get("SLLM_RETENTION_CHUNKED_FROM", "96"))
+
+
+@functools.lru_cache(maxsize=4096)
+def retention_chunked_supports(dk: int, dv: int) -> bool:
+    return bool(lib().sllm_retention_chunked_supports(int(dk), int(dv)))
+
+
+def retention_chunks(q_lens, ctx_lens, min_len: int, device):
+    """The step's long portions cut into chunks of `RETENTION_CHUNK` tokens: (first tokens, their positions, lengths, chunks; requests,
+    their first chunk, how many, requests) on the device, or None where no portion has ``min_len`` tokens."""
+    t0, pos, n, seq, first, count = [], [], [], [], [], []
+    start = 0
+    for s, (q, ctx) in enumerate(zip(q_lens, ctx_lens)):
+        if q >= min_len:
+            seq.append(s)
+            first.append(len(t0))
+            for a in range(0, q, RETENTION_CHUNK):
+                t0.append(start + a)
+                pos.append(ctx - q + a)
+                n.append(min(RETENTION_CHUNK, q - a))
+            count.append(len(t0) - first[-1])
+        start += q
+    if not seq:
+        return None
+    t = torch.tensor(t0 + pos + n + seq + first + count, dtype=torch.int32).to(device, non_blocking=True)
+    C, R = len(t0), len(seq)
+    o = 3 * C
+    return t[:C], t[C:2 * C], t[2 * C:o], C, t[o:o + R], t[o + R:o + 2 * R], t[o + 2 * R:], R
+
+
+def retention_chunked(proj, offs, off_g: int, decay, table, rotary_dim: int, k_scale: float, eps: float, state, step, chunks, heads: int,
+                      dk: int, dv: int, out) -> None:
+    """Retention, the heads' norm and the silu gate (columns ``off_g`` of ``proj``) for the requests that ``chunks`` (see
+    `retention_chunks`) cuts, a chunk of tokens at a time; their rows of ``out`` ``[T, heads*dv]`` and their states are written, others
+    left alone."""
+    _chk(proj, decay, table, state, out)
+    if proj.dtype != torch.float32 or decay.dtype != torch.float32 or state.dtype != torch.float32:
+        raise KernelError("retention_chunked: everything that enters the recurrence is float32")
+    if tuple(decay.shape) != (heads,) or tuple(state.shape[1:]) != (heads, dk, dv) or tuple(out.shape) != (proj.shape[0], heads * dv):
+        raise KernelError(f"retention_chunked: decay {tuple(decay.shape)}, state {tuple(state.shape)} or output {tuple(out.shape)} does not fit "
+                          f"{heads} heads of {dk}x{dv}")
+    rot = int(rotary_dim) if table is not None else 0
+    if rot and (table.dtype != torch.float32 or tuple(table.shape[1:]) != (2, rot // 2)):
+        raise KernelError("retention_chunked: rotary table must be float32 [positions, 2, rotary_dim/2]")
+    t0, pos, n, C, seq, first, count, R = chunks
+    scratch = torch.empty((C, heads, dk, dv), dtype=torch.float32, device=proj.device)
+    off_q, off_k, off_v = (int(o) for o in offs)
+    call("sllm_retention_chunked", _p(proj), proj.shape[1], off_q, off_k, off_v, int(off_g), _p(decay), _p(table), rot,
+         table.shape[0] if rot else 0, float(k_scale), float(eps), _p(state), _p(step.state_slots), _p(t0), _p(pos), _p(n), C, _p(seq), _p(first),
+         _p(count), R, _p(scratch), _p(out), _dtc(out.dtype), out.shape[1], heads, dk, dv, _stream())
+    launches["own"] += 2           # the three kernels of the entry point
+
+
+def retention_gated(proj, offs, off_g: int, decay, table, rotary_dim: int, k_scale: float, eps: float, state, step, heads: int, dk: int,
+                    dv: int, out_dtype) -> torch.Tensor:
+    """`retention` and what follows it in a layer: each head's output over its root mean square, times silu of columns ``off_g`` of
+    ``proj``, ``[T, heads*dv]`` in ``out_dtype``.  Long prompt portions run in chunks (heads of up to 128 x 128), single tokens and short
+    portions token by token; a step may hold both."""
+    chunks, longest = None, 0
+    if RETENTION_CHUNKED_FROM > 0 and step.max_q_len >= RETENTION_CHUNKED_FROM and step.q_lens and retention_chunked_supports(dk, dv):
+        if "retention" not in step.attn_tiles:
+            step.attn_tiles["retention"] = retention_chunks(step.q_lens, step.ctx_lens, RETENTION_CHUNKED_FROM, proj.device)
+        chunks, longest = step.attn_tiles["retention"], RETENTION_CHUNKED_FROM - 1
+    if chunks is None:
+        o = retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv)
+        return delta_out(o, None, proj, off_g, eps, heads, dv, out_dtype, "silu")
+    out = torch.empty((proj.shape[0], heads * dv), dtype=out_dtype, device=proj.device)
+    retention_chunked(proj, offs, off_g, decay, table, rotary_dim, k_scale, eps, state, step, chunks, heads, dk, dv, out)
+    if chunks[7] < step.num_seqs:
+        o = retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv, max_len=longest)
+        delta_out(o, None, proj, off_g, eps, heads, dv, out_dtype, "silu", out=out, step=step, max_len=longest)
     return out
 
 
@@ -679,10 +761,10 @@ def linear_stream(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False,
     a float32 stack ``[splits', M, N]`` of partial sums (bias in the first) that the consumer
     adds; with ``silu`` the matrix is gate|up interleaved in blocks of 8 and the result is
     ``silu(gate) * up`` of width N/2; with ``act="gelu_tanh"`` it is ``gelu_tanh(gate + bias) * (up + bias)``
-    (the bias interleaved like the rows); with ``act="relu2"`` the plain result's ``max(v, 0)^2`` (bfloat16)."""
-    if act not in (None, "gelu_tanh", "relu2") or (act and silu):
-        raise KernelError(f"linear_stream: epilogue {act!r}")
-    gated = silu or act == "gelu_tanh"
+    (the bias interleaved like the rows)."""
+    if act not in (None, "gelu_tanh") or (act and silu):
+        raise KernelError(f"linear_stream: gated epilogue {act!r}")
+    gated = silu or act is not None
     _chk(x, w, bias)
     M, K = x.shape
     N = w.shape[0]
@@ -697,7 +779,7 @@ def linear_stream(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False,
     else:
         out = torch.empty((M, N // 2 if gated else N), dtype=out_dtype, device=x.device)
     call("sllm_linear_stream", _p(x), _p(w), _p(bias), _p(out), _dtc(out_dtype), _p(partial), M, N, K,
-         real if real > 1 else 1, 1 if silu else {None: 0, "gelu_tanh": 2, "relu2": 3}[act], _stream())
+         real if real > 1 else 1, 1 if silu else 2 if act else 0, _stream())
     return partial if real > 1 else out
 
 
@@ -968,10 +1050,14 @@ def _tc_from_rows(N: int, K: int) -> int:
 
 
 @functools.lru_cache(maxsize=4096)
+def linear_tc_takes(M: int, N: int, K: int) -> bool:
+    """Whether the kernel runs these sizes at all."""
+    return _LINEAR_TC and M <= LINEAR_TC_MAX_ROWS and bool(lib().sllm_linear_tc_supports(int(M), int(N), int(K)))
+
+
+@functools.lru_cache(maxsize=4096)
 def linear_tc_supports(M: int, N: int, K: int) -> bool:
-    if not (_LINEAR_TC and M <= LINEAR_TC_MAX_ROWS and bool(lib().sllm_linear_tc_supports(int(M), int(N), int(K)))):
-        return False
-    return M >= _tc_from_rows(N, K)
+    return linear_tc_takes(M, N, K) and M >= _tc_from_rows(N, K)
 
 
 @functools.lru_cache(maxsize=4096)
@@ -1026,9 +1112,13 @@ def ws_supports(M: int, N: int, K: int) -> bool:
     """Whether the warp-split kernel is the one for this product.  With two token tiles (9..16 tokens) only where
     its 16-row CTAs fit the GPU at once: at N = 5120 (320 to 592 CTAs for 296 places) it falls behind the k-split
     kernel by more than the fused epilogues save (16 tokens, K = 27648: 64.3 against 49.2 us)."""
-    if not (M <= WS_MAX_ROWS and N <= WS_MAX_COLS and bool(lib().sllm_linear_ws_supports(int(M), int(N), int(K)))):
-        return False
-    return _ws_tokens_ok(M, N, K)
+    return N <= WS_MAX_COLS and ws_takes(M, N, K) and _ws_tokens_ok(M, N, K)
+
+
+@functools.lru_cache(maxsize=4096)
+def ws_takes(M: int, N: int, K: int) -> bool:
+    """Whether the kernel runs these sizes at all."""
+    return M <= WS_MAX_ROWS and bool(lib().sllm_linear_ws_supports(int(M), int(N), int(K)))
 
 
 def _ws_tokens_ok(M: int, N: int, K: int) -> bool:
@@ -1205,14 +1295,15 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias, out_dtype: torch.dtype, allow
 
 
 def plain_act(x, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
-    """``act`` of ``x [T, N]`` in ``out_dtype``: ``relu2`` is ``max(x, 0)^2``, ``token`` is ``gelu_tanh(x)`` times ``token``'s columns
+    """``act`` of ``x [T, N]`` (or of the sum of a stack of partial sums ``[parts, T, N]``) in ``out_dtype``: ``relu2`` is ``max(x, 0)^2``, ``token`` is ``gelu_tanh(x)`` times ``token``'s columns
     (a table of ``out_dtype``)."""
     _chk(x)
-    T, N = x.shape
+    T, N = x.shape[-2:]
+    parts, stride = (x.shape[0], T * N) if x.dim() == 3 else (1, 0)
     if (act == "token") != (token is not None) or (token is not None and token.table.dtype != out_dtype):
         raise KernelError("plain_act: the token activation needs its table, of the result's dtype")
     out = torch.empty((T, N), dtype=out_dtype, device=x.device)
-    call("sllm_plain_act", _p(x), _dt(x), _p(out), _dtc(out_dtype), T, N, PLAIN_ACTS[act], *(token.args() if token is not None else _NO_TOKEN),
+    call("sllm_plain_act", _p(x), _dt(x), parts, stride, _p(out), _dtc(out_dtype), T, N, PLAIN_ACTS[act], *(token.args() if token is not None else _NO_TOKEN),
          _stream())
     return out
 
@@ -1222,21 +1313,23 @@ _PLAIN_ACT_FUSED = os.environ.get("SLLM_PLAIN_ACT_FUSED", "1") != "0"      # 0: 
 
 def linear_plain_act(x, w, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
     """``act(x @ w.T)`` in ``out_dtype`` (see `plain_act`).  bfloat16: the activation leaves with the product's tile (the warp-split
-    streaming product, the CTA-pair product; ``relu2`` also in the streaming product and on tensor memory up to 128 tokens).
-    Otherwise the product in float32, then the activation kernel."""
+    streaming product up to 16 tokens, the CTA-pair product of prompt portions; ``relu2`` of large matrices also on tensor memory).
+    Otherwise the product in float32, cut along K where that is faster, then the activation kernel, which adds the slices.
+    (In a graph, us: 8,448 x 2,048 and 8 tokens 8.3 in the warp-split form, 8.7 in four slices and a kernel, 17.5 in the streaming
+    form unsliced; 16,512 x 4,096 and 8 tokens 29.3 / 26.6 / 36.8, on tensor memory 28.0; 32 tokens of the former 13.0 / 11.5 / 20.6,
+    of the latter 27.6 on tensor memory and 35 in slices.)"""
     if _PLAIN_ACT_FUSED and x.is_cuda and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and \
             x.shape[1] == w.shape[1]:
         M, K = x.shape
         N = w.shape[0]
-        if ws_supports(M, N, K):
+        large = N * K >= LINEAR_TC_LARGE
+        if ws_supports(M, N, K) or (M <= 16 and not large and ws_takes(M, N, K)):
             return linear_ws(x, w, None, out_dtype, act=act, token=token)
-        if act == "relu2" and stream_supports(M, N, K):
-            return linear_stream(x, w, None, out_dtype, act=act)
-        if act == "relu2" and N * K >= LINEAR_TC_LARGE and linear_tc_supports(M, N, K):
+        if act == "relu2" and large and M >= LINEAR_TC_WIDE_FROM_ROWS and linear_tc_takes(M, N, K):
             return linear_tc(x, w, None, out_dtype, act=act)
         if _pair_rows(M) and pair_supports(M, N, K):
             return gemm_pair(x, w, None, out_dtype, act=act, token=token)
-    return plain_act(linear(x, w, None, torch.float32), out_dtype, act, token)
+    return plain_act(linear(x, w, None, torch.float32, True), out_dtype, act, token)
 
 
 def silu_mul(gu: torch.Tensor, interleave: int, out_dtype: torch.dtype) -> torch.Tensor:

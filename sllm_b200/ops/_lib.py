@@ -51,7 +51,7 @@ def _declare(L):
         "sllm_delta_rule": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_delta_out": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                           c_int, c_void_p],
+                           c_int, c_void_p, c_void_p, c_int, c_void_p],
         "sllm_gated_delta_rule": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                   c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
         "sllm_gated_linear_attention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -149,9 +149,13 @@ def _declare(L):
         "sllm_decay_linear_attention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_retention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_retention_chunked_supports": [c_int, c_int],
+        "sllm_retention_chunked": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float,
+                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                   c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_softcap": [c_void_p, ctypes.c_longlong, c_float, c_void_p],
-        "sllm_plain_act": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "sllm_plain_act": [c_void_p, c_int, c_int, c_size_t, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_latent_rope_write": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_head_linear_strided": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,

@@ -151,7 +151,7 @@ class Retention(Mixer):
     dim^(-1/2), and v = W_v x (heads x vdim).  Each head's o over its root mean square (no gain), times silu(W_g x), then W_o.
     Parameters: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``decay`` (one number per head), ``rotary`` (None, or ``theta``,
     ``rotary_dim``, ``max_positions``), ``eps`` (of the heads' norm).  q, k, v and the gate are one matrix whose product stays
-    float32; rotation and scale happen in the recurrence kernel's loader."""
+    float32; rotation and scale happen as the recurrence's kernels load it (`ops.retention_gated`)."""
 
     NAMES = ("q", "k", "v", "g")
 
@@ -198,9 +198,8 @@ class Retention(Mixer):
 
     def mix(self, x, step: StepContext, cache: LayerCache, position=None, write_cache=True):
         proj = self.inp(x, torch.float32)                                            # [T, 2K + 2V] float32
-        o = ops.retention(proj, self.offs, self.decay, self.rotary.table if self.rotary is not None else None, self.rot,
-                          self.dim ** -0.5, cache.states["retention"], step, self.heads, self.dim, self.vdim)
-        return ops.delta_out(o, None, proj, self.off_g, self.eps, self.heads, self.vdim, self.dtype, "silu")
+        return ops.retention_gated(proj, self.offs, self.off_g, self.decay, self.rotary.table if self.rotary is not None else None, self.rot,
+                                   self.dim ** -0.5, self.eps, cache.states["retention"], step, self.heads, self.dim, self.vdim, self.dtype)
 
     def forward(self, x, step, cache, position, write_cache=True, residual=None):
         return self.out.into(self.mix(x, step, cache, position, write_cache), residual)

@@ -395,6 +395,7 @@ def softcap_(x, cap):
 
 
 def plain_act(x, out_dtype, act, token=None):
+    x = x.float().sum(0) if x.dim() == 3 else x
     if act == "relu2":
         return torch.relu(x.float()).square().to(out_dtype)
     e = token.table[token.ids.long(), token.off:token.off + x.shape[1]].float()
@@ -440,6 +441,11 @@ def decay_linear_attention(proj, offs, decay, state, step, heads, dk, dv):
         return S, torch.einsum("hij,hi->hj", S, q[t])
     _walk(step, state, out, token)
     return out.reshape(T, heads * dv)
+
+
+def retention_gated(proj, offs, off_g, decay, table, rotary_dim, k_scale, eps, state, step, heads, dk, dv, out_dtype):
+    o = retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv)
+    return delta_out(o, None, proj, off_g, eps, heads, dv, out_dtype, "silu")
 
 
 def retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv):
@@ -652,7 +658,7 @@ def penalty_from_seen_(logits, seen, step, penalty):
     return logits
 
 
-ALL = ["retention", "post_add_copy", "softcap_", "plain_act", "linear_plain_act", "forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
+ALL = ["retention", "retention_gated", "post_add_copy", "softcap_", "plain_act", "linear_plain_act", "forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
        "decay_linear_attention", "gated_delta_rule", "gated_linear_attention", "qk_norm_rope_kv_write", "short_conv_silu", "norm_mean_add_", "moe_route", "moe_act",
        "add_sinusoid_", "add_group_ssq", "group_norm_shift", "act_mul", "linear_act_mul", "tanh_cols", "delta_rule", "delta_out", "latent_write",
        "head_linear", "embed_gather", "add_rmsnorm", "linear", "can_accumulate", "linear_accumulate", "silu_mul", "linear_silu_mul", "rope_kv_write",
