@@ -79,6 +79,16 @@ class RunEntry:
 
 
 @dataclass(frozen=True)
+class TokenPairs:
+    """A table of rows by the pair (token before, token), added to the embedding: row ``(before * mul_prev + token * mul_cur)
+    mod buckets`` of the tensor ``name`` ``[buckets + 1, hidden]``; a sequence's first token has the last row."""
+    name: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class ModelPlan:
     architecture: str
     hidden_size: int
@@ -101,11 +111,20 @@ class ModelPlan:
     token_table_name: str | None = None      # tensor [vocab, token_table_width]: vectors that belong to a token, for parts that ask for it
     token_table_width: int = 0
     logit_softcap: float | None = None       # logits become softcap tanh(logits / softcap)
+    token_pairs: TokenPairs | None = None    # rows by pairs of tokens that the embedding takes in
+    streams: int | None = None               # the residual stream is so many copies [T, streams, hidden] (None: one, [T, hidden]); every
+                                             # block of the plan must be a kind that arranges them
 
     def validate(self) -> None:
         from .errors import ConfigError
         if not self.layers:
             raise ConfigError("a model needs at least one layer")
+        if self.streams is not None and (self.streams < 1 or self.embedding_norm is not None or self.position is not None or
+                                         any(e.reentry is not None for e in self.run_list)):
+            raise ConfigError(f"a stream of {self.streams} copies goes with no norm on the embedding, no position encoding added to it and "
+                              f"no pass vectors")
+        if self.token_pairs is not None and self.vocab_size > 1 << 24:
+            raise ConfigError(f"pairs of tokens: the token before is kept in float32 state, exact for ids below 2^24; vocab={self.vocab_size}")
         for i, layer in enumerate(self.layers):
             for role, e in layer.parts.items():
                 if e.family not in ("mixer", "feed_forward", "norm", "shift"):

@@ -48,6 +48,8 @@ struct AttnParams {
   const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
   int gate_ld;
   const float* sink;             // [nq] or null: exp(sink_h) joins the softmax's denominator (no key, no value, not scaled)
+  const float* rel;              // [nkv, rel_n, nq / nkv] or null: added to the score (after the cap) by the distance from key to query
+  int rel_n;                     // (distances from rel_n - 1 on: the last row)
   // pooled blocks beside a window (pool > 0; needs window > 0 and num_splits == 1): a query at position i also sees entry b
   // of the pooled cache (same page geometry) for every b < (i - window + 1) / pool; these entries are walked as key tiles
   // of their own before the window's
@@ -224,6 +226,14 @@ __global__ void __launch_bounds__(AttThreads<DECODE>::value) attention_mma_kerne
       lo_r[i] = 1;                                // empty
     }
   }
+  const float* rel_h[2];                          // the bias table at the row's head (rows of G)
+  int rel_pos[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int row = row0 + wrow + g + 8 * i;
+    rel_h[i] = p.rel != nullptr ? p.rel + (size_t)kvh * p.rel_n * G + row % G : nullptr;
+    rel_pos[i] = pos0 + row / G;
+  }
   float m_r[2] = {-INFINITY, -INFINITY}, l_r[2] = {0.f, 0.f};
   float o[DT][4];
 #pragma unroll
@@ -275,7 +285,8 @@ __global__ void __launch_bounds__(AttThreads<DECODE>::value) attention_mma_kerne
         const int key = kbase + n * 8 + 2 * t4 + (c & 1);
         const int i = c >> 1;
         const bool seen = pooled_tile ? key < nb_r[i] : (key < hi_r[i] && key >= lo_r[i]);
-        const float sl = p.cap_log2 > 0.f ? softcap_log2(s[n][c], p.cap_slope, p.cap_log2) : s[n][c] * p.scale_log2;
+        float sl = p.cap_log2 > 0.f ? softcap_log2(s[n][c], p.cap_slope, p.cap_log2) : s[n][c] * p.scale_log2;
+        if (p.rel != nullptr) sl = fmaf(rel_h[i][(size_t)min(max(rel_pos[i] - key, 0), p.rel_n - 1) * G], 1.4426950408889634f, sl);
         const float v = seen ? sl : -INFINITY;
         s[n][c] = v;
         mx[i] = fmaxf(mx[i], v);
@@ -499,7 +510,8 @@ SLLM_EXPORT int sllm_attention_mma(const void* q, const void* k_cache, const voi
                                    const int* ctx_len, const int* tile_seq, const int* tile_row0, int tiles,
                                    int decode, int num_splits, int total_tokens, int nq, int nkv, int hd,
                                    int page_size, float scale, int window, int block, const float* sink, float softcap, const float* gate,
-                                   int gate_ld, cudaStream_t stream) {
+                                   int gate_ld, const float* rel, int rel_n, cudaStream_t stream) {
+  SLLM_REQUIRE(rel == nullptr || rel_n >= 1, "attention_mma: a bias by distance needs its table");
   SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_mma: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_mma: bad head counts nq=%d nkv=%d", nq, nkv);
   SLLM_REQUIRE(sllm_attention_mma_supports(hd), "attention_mma: head_dim=%d is not one of 16, 32, 64, 128", hd);
@@ -516,7 +528,7 @@ SLLM_EXPORT int sllm_attention_mma(const void* q, const void* k_cache, const voi
   p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
   p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
-  p.gate = gate; p.gate_ld = gate_ld;
+  p.gate = gate; p.gate_ld = gate_ld; p.rel = rel; p.rel_n = rel_n;
   p.pk_cache = p.pv_cache = nullptr; p.pool_tables = nullptr; p.pool_max_pages = p.pool = 0;
   p.out_ld = p.out_off = p.vdim = 0; p.out_scale = 1.f;
 #define DISPATCH(HD_)                                                             \
@@ -559,7 +571,7 @@ SLLM_EXPORT int sllm_attention_mma_pooled(const void* q, const void* k_cache, co
   p.num_splits = num_splits; p.total_tokens = total_tokens;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
-  p.cap_log2 = p.cap_slope = 0.f; p.gate = nullptr; p.gate_ld = 0;
+  p.cap_log2 = p.cap_slope = 0.f; p.gate = nullptr; p.gate_ld = 0; p.rel = nullptr; p.rel_n = 0;
   p.pk_cache = (const __nv_bfloat16*)pk_cache; p.pv_cache = (const __nv_bfloat16*)pv_cache; p.pool_tables = pool_tables;
   p.pool_max_pages = pool_max_pages; p.pool = pool;
   p.out_ld = out_ld; p.out_off = out_off; p.vdim = vdim; p.out_scale = out_scale;

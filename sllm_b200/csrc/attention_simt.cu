@@ -11,7 +11,8 @@
 //   Query head h reads kv head h / (nq / nkv) (ref/standard.py:65-68).
 //   With `sink` (one number per query head) the softmax's denominator also holds exp(sink_h).
 //   With `softcap` > 0 a score becomes softcap tanh(score / softcap) before the softmax; with `gate` (logits, one per token
-//   and query head) the head's output is multiplied by the gate's sigmoid.
+//   and query head) the head's output is multiplied by the gate's sigmoid.  With `rel` [nkv, rel_n, nq / nkv] the score then takes in
+//   a bias by the distance from key to query (distances beyond the table: its last row) and the query head.
 //
 // Each of the block's warps takes keys w, w+W, w+2W, ... in ascending order with an
 // online softmax; the warps' partial results are merged in warp order.  The order
@@ -33,13 +34,13 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_cache, 
                       const int* __restrict__ block_tables, int max_pages, const int* __restrict__ positions,
                       const int* __restrict__ seq_of_token, int nq, int nkv, int hd, int page_size, float scale,
                       int window, int chunk, const float* __restrict__ sink, float softcap, const float* __restrict__ gate, int gate_ld,
-                      TQ* __restrict__ out) {
+                      const float* __restrict__ rel, int rel_n, TQ* __restrict__ out) {
   __shared__ float qs[ATT_MAX_HD];
   __shared__ float acc_s[ATT_WARPS][ATT_MAX_HD];
   __shared__ float m_s[ATT_WARPS], l_s[ATT_WARPS];
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
-  const int kvh = h / (nq / nkv);
+  const int G = nq / nkv, kvh = h / G;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int pos = positions[t];
   const int* bt = block_tables + (size_t)seq_of_token[t] * max_pages;
@@ -61,7 +62,8 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_cache, 
     float dot = 0.f;
     for (int d = lane; d < hd; d += 32) dot = fmaf(qs[d], to_f32(k_cache[row + d]), dot);
     dot = warp_sum(dot);
-    const float s = softcap > 0.f ? softcap * tanhf(dot * scale / softcap) : dot * scale;
+    float s = softcap > 0.f ? softcap * tanhf(dot * scale / softcap) : dot * scale;
+    if (rel != nullptr) s += rel[((size_t)kvh * rel_n + min(pos - j, rel_n - 1)) * G + h % G];
     const float m_new = fmaxf(m, s);
     const float corr = expf(m - m_new);              // exp(-inf) = 0 on the first key
     const float p = expf(s - m_new);
@@ -109,30 +111,31 @@ SLLM_EXPORT int sllm_attention_simt(const void* q, const void* k_cache, const vo
                                     const int* block_tables, int max_pages, const int* positions,
                                     const int* seq_of_token, int T, int nq, int nkv, int hd, int page_size,
                                     float scale, int window, int chunk, const float* sink, float softcap, const float* gate, int gate_ld,
-                                    void* out, cudaStream_t stream) {
+                                    const float* rel, int rel_n, void* out, cudaStream_t stream) {
   SLLM_REQUIRE(T >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention: bad head counts nq=%d nkv=%d", nq, nkv);
   SLLM_REQUIRE(hd > 0 && hd <= ATT_WIDE_HD, "attention: head_dim=%d is outside 1..%d", hd, ATT_WIDE_HD);
   SLLM_REQUIRE(page_size > 0 && max_pages > 0, "attention: bad page_size=%d max_pages=%d", page_size, max_pages);
   SLLM_REQUIRE(nq <= 65535, "attention: %d query heads exceed one launch", nq);
+  SLLM_REQUIRE(rel == nullptr || rel_n >= 1, "attention: a bias by distance needs its table");
   if (T == 0) return SLLM_OK;
   dim3 grid(T, nq);
   if (dtype == SLLM_F32) {
     if (hd <= ATT_MAX_HD) launch_kernel(attention_simt_kernel<float, float, ATT_MAX_HD>, grid, ATT_WARPS * 32, 0, stream,
         (const float*)q, (const float*)k_cache, (const float*)v_cache, block_tables, max_pages, positions,
-        seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, (float*)out);
+        seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, rel, rel_n, (float*)out);
     else
       launch_kernel(attention_simt_kernel<float, float, ATT_WIDE_HD>, grid, ATT_WARPS * 32, 0, stream,
           (const float*)q, (const float*)k_cache, (const float*)v_cache, block_tables, max_pages, positions,
-          seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, (float*)out);
+          seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, rel, rel_n, (float*)out);
   }
   else if (dtype == SLLM_BF16) {
     if (hd <= ATT_MAX_HD) launch_kernel(attention_simt_kernel<__nv_bfloat16, __nv_bfloat16, ATT_MAX_HD>, grid, ATT_WARPS * 32, 0, stream,
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_tables,
-        max_pages, positions, seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, (__nv_bfloat16*)out);
+        max_pages, positions, seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, rel, rel_n, (__nv_bfloat16*)out);
     else
       launch_kernel(attention_simt_kernel<__nv_bfloat16, __nv_bfloat16, ATT_WIDE_HD>, grid, ATT_WARPS * 32, 0, stream,
           (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_tables,
-          max_pages, positions, seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, (__nv_bfloat16*)out);
+          max_pages, positions, seq_of_token, nq, nkv, hd, page_size, scale, window, chunk, sink, softcap, gate, gate_ld, rel, rel_n, (__nv_bfloat16*)out);
   } else
     SLLM_REQUIRE(false, "attention: unknown dtype %d", dtype);
   return launch_status("attention_simt");

@@ -81,6 +81,9 @@ struct AttnTcParams {
   float cap_log2, cap_slope;     // CAP: capped scores, cap * log2(e) and 2 scale log2(e) / cap (see softcap_log2)
   const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
   int gate_ld;
+  const float* rel;              // REL: [nkv, rel_n, nq / nkv], added to the score (after the cap) by the distance from key to query
+  int rel_n;                     // (distances from rel_n - 1 on: the last row)
+  const float* rel_top;          // [nq] each head's largest bias
 };
 
 constexpr int TC_BM = 128, TC_BN = 64;
@@ -135,8 +138,10 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
   return d;
 }
 
-// CAP: a score becomes cap * tanh(score / cap) before the softmax
-template <int HD, int RT, bool CAP>
+// CAP: a score becomes cap * tanh(score / cap) before the softmax.  REL: a bias by distance is added then; a tile whose keys all lie
+// rel_n - 1 positions and more before the warp's rows adds one number a row, which joins the exponent's constant; in the tiles nearer by, a
+// row's maximum is bounded by its largest score plus its head's largest bias (any number near the maximum will do: it cancels).
+template <int HD, int RT, bool CAP, bool REL>
 __global__ void __launch_bounds__(TcLayout<HD, RT>::THREADS, RT == 1 ? 2 : 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                     const __grid_constant__ CUtensorMap run_k, const __grid_constant__ CUtensorMap run_v,
@@ -420,6 +425,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(&q_full[t]);
     }
+    // REL: the row's place in the bias table (rows of G; neighbouring rows of a tile read neighbouring numbers), its last and largest bias
+    const float* rel_h = nullptr;
+    const int rel_pos = pos0 + row / G;
+    float rel_far = 0.f, rel_top = 0.f;
+    if constexpr (REL) {
+      rel_h = p.rel + (size_t)kvh * p.rel_n * G + row % G;
+      rel_far = __ldg(rel_h + (size_t)(p.rel_n - 1) * G) * 1.4426950408889634f;
+      rel_top = __ldg(p.rel_top + kvh * G + row % G) * 1.4426950408889634f;
+    }
     float m_used = -INFINITY, l = 0.f;                                 // the maximum in scaled (log2) units
     bool ok = !*failed;
     for (int j = 0; j < my_tiles && ok; ++j) {
@@ -448,6 +462,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       // (the cap's curve rises, so the maximum of the capped scores is the capped maximum; no key: -inf stays)
       if constexpr (CAP) mx = mx == -INFINITY ? mx : softcap_log2(mx, p.cap_slope, p.cap_log2);
       else mx *= p.scale_log2;
+      const bool far = REL && __all_sync(0xffffffffu, rel_pos - (kbase + TC_BN - 1) >= p.rel_n - 1);
+      if constexpr (REL) mx += far ? rel_far : rel_top;
       const bool grow = mx > m_used + TC_RESCALE_STEP;      // also the first tile with a key (m_used = -inf)
       // Only a rescale of O waits for the product of the tile before it (O must not change under it).
       // The barrier is the one behind that product, s_free of its buffer: its phases go by every
@@ -475,7 +491,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
+      const float neg_m = (m_used == -INFINITY ? 0.f : -m_used) + (far ? rel_far : 0.f);
+      auto near_bias = [&](int key) { return __ldg(rel_h + (size_t)min(max(rel_pos - key, 0), p.rel_n - 1) * G) * 1.4426950408889634f; };
       uint32_t pk[32];                                      // column i: keys 2i (low half) and 2i+1
       float2 sums = make_float2(0.f, 0.f);                  // of the even and of the odd keys
       if constexpr (CAP) {
@@ -487,7 +504,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           // (beyond 2^60 the quotient is nothing; the bound keeps the product of the two finite)
           const float2 d = add_x2(make_float2(ex2(fminf(z.x, 60.f)), ex2(fminf(z.y, 60.f))), make_float2(1.f, 1.f));
           const float rr = __fdividef(1.0f, d.x * d.y);
-          const float2 x = fma_x2(d.y * rr, d.x * rr, two_cap, top);
+          float2 x = fma_x2(d.y * rr, d.x * rr, two_cap, top);
+          if (REL && !far) x = add_x2(x, make_float2(near_bias(key), near_bias(key + 1)));
           return make_float2(edge && key >= hi ? 0.f : ex2(x.x), edge && key + 1 >= hi ? 0.f : ex2(x.y));
         };
 #pragma unroll
@@ -500,8 +518,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       } else {
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        const float2 x01 = fma_x2(__uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]), p.scale_log2, neg_m);
-        const float2 x23 = fma_x2(__uint_as_float(s1[2 * i]), __uint_as_float(s1[2 * i + 1]), p.scale_log2, neg_m);
+        float2 x01 = fma_x2(__uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]), p.scale_log2, neg_m);
+        float2 x23 = fma_x2(__uint_as_float(s1[2 * i]), __uint_as_float(s1[2 * i + 1]), p.scale_log2, neg_m);
+        if (REL && !far) {
+          const int key = kbase + 2 * i;
+          x01 = add_x2(x01, make_float2(near_bias(key), near_bias(key + 1)));
+          x23 = add_x2(x23, make_float2(near_bias(key + 32), near_bias(key + 33)));
+        }
         const float2 e01 = make_float2(ex2(x01.x), ex2(x01.y)), e23 = make_float2(ex2(x23.x), ex2(x23.y));
         sums = add_x2(sums, add_x2(e01, e23));
         pk[i] = pack2(e01.x, e01.y);
@@ -627,20 +650,20 @@ static bool tc_cache_map(const void* base, long long rows, int ps, int hd, CUten
   return true;
 }
 
-template <int HD, int RT, bool CAP>
+template <int HD, int RT, bool CAP, bool REL>
 static int launch_tc(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& rk, const CUtensorMap& rv,
                      const AttnTcParams& p, int tiles, cudaStream_t stream) {
   constexpr int smem = TcLayout<HD, RT>::SMEM;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tc_kernel<HD, RT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attention_tc_kernel<HD, RT, CAP, REL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
       set_error("attention_tc: cannot raise the shared memory limit");
       return SLLM_ERR_LAUNCH;
     }
     configured = true;
   }
   dim3 grid((unsigned)tiles * p.nkv, 1, p.num_splits);
-  launch_kernel(attention_tc_kernel<HD, RT, CAP>, grid, TcLayout<HD, RT>::THREADS, (size_t)smem, stream, mk, mv, rk, rv, p);
+  launch_kernel(attention_tc_kernel<HD, RT, CAP, REL>, grid, TcLayout<HD, RT>::THREADS, (size_t)smem, stream, mk, mv, rk, rv, p);
   int rc = launch_status("attention_tc");
   if (rc != SLLM_OK || p.num_splits == 1) return rc;
   launch_kernel(attention_tc_combine_kernel<HD>, p.total_tokens * p.nq, HD >= 128 ? 128 : 64, 0, stream,
@@ -670,7 +693,9 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
                                   const int* tile_seq, const int* tile_row0, int tiles, int row_tiles, int nq, int nkv,
                                   int hd, int page_size, float scale, int num_splits, int tiles_per_split, int total_tokens,
                                   float* part_o, float* part_lse, const int* seq_row, const int* page_shift, const float* sink,
-                                  float softcap, const float* gate, int gate_ld, int* status, cudaStream_t stream) {
+                                  float softcap, const float* gate, int gate_ld, const float* rel, int rel_n, const float* rel_top,
+                                  int* status, cudaStream_t stream) {
+  SLLM_REQUIRE(rel == nullptr || (rel_n >= 1 && rel_top && seq_row == nullptr), "attention_tc: a bias by distance needs its table, and whole requests");
   SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_tc: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE((seq_row == nullptr) == (page_shift == nullptr), "attention_tc: parts of requests need both their row and their first page");
   SLLM_REQUIRE(row_tiles == 1 || row_tiles == 2, "attention_tc: row_tiles=%d must be 1 or 2", row_tiles);
@@ -703,11 +728,14 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
   p.total_tokens = total_tokens; p.part_o = part_o; p.part_lse = part_lse; p.seq_row = seq_row; p.page_shift = page_shift;
   p.sink = sink;
   p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
-  p.gate = gate; p.gate_ld = gate_ld;
-  SLLM_REQUIRE(softcap == 0.f || row_tiles == 1, "attention_tc: capped scores run in the form of one row tile a CTA");
-  if (softcap > 0.f)
-    return hd == 128 ? launch_tc<128, 1, true>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 1, true>(mk, mv, rk, rv, p, tiles, stream);
-  if (row_tiles == 2)
-    return hd == 128 ? launch_tc<128, 2, false>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 2, false>(mk, mv, rk, rv, p, tiles, stream);
-  return hd == 128 ? launch_tc<128, 1, false>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, 1, false>(mk, mv, rk, rv, p, tiles, stream);
+  p.gate = gate; p.gate_ld = gate_ld; p.rel = rel; p.rel_n = rel_n; p.rel_top = rel_top;
+  SLLM_REQUIRE((softcap == 0.f && rel == nullptr) || row_tiles == 1, "attention_tc: capped or biased scores run in the form of one row tile a CTA");
+#define TC_GO(RT_, CAP_, REL_) \
+  return hd == 128 ? launch_tc<128, RT_, CAP_, REL_>(mk, mv, rk, rv, p, tiles, stream) : launch_tc<64, RT_, CAP_, REL_>(mk, mv, rk, rv, p, tiles, stream)
+  if (softcap > 0.f && rel != nullptr) TC_GO(1, true, true);
+  if (softcap > 0.f) TC_GO(1, true, false);
+  if (rel != nullptr) TC_GO(1, false, true);
+  if (row_tiles == 2) TC_GO(2, false, false);
+  TC_GO(1, false, false);
+#undef TC_GO
 }

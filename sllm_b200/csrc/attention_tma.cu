@@ -54,6 +54,8 @@ struct AttnTmaParams {
   float cap_log2, cap_slope;     // CAP: capped scores, cap * log2(e) and 2 scale log2(e) / cap (see softcap_log2)
   const float* gate;             // or null: logits [T, gate_ld], one per query head; the head's output times their sigmoid
   int gate_ld;
+  const float* rel;              // REL: [nkv, rel_n, nq / nkv], added to the score (after the cap) by the distance from key to query
+  int rel_n;                     // (distances from rel_n - 1 on: the last row)
 };
 
 // Byte offset of the 16-byte chunk `chunk` (of the head's HD/8) of key row `row` within a stage's K or V.
@@ -65,8 +67,8 @@ __device__ __forceinline__ int swz(int row, int chunk) {
   return unit * 128 + (((chunk & 7) ^ (unit & 7)) << 4);
 }
 
-// CAP: a score becomes cap * tanh(score / cap) before the softmax
-template <int HD, bool CAP>
+// CAP: a score becomes cap * tanh(score / cap) before the softmax (with REL, where there is a cap); REL: then a bias by distance is added
+template <int HD, bool CAP, bool REL>
 __global__ void __launch_bounds__(TA_THREADS)
 attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const __grid_constant__ CUtensorMap run_k, const __grid_constant__ CUtensorMap run_v,
@@ -228,6 +230,19 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         lo_r[i] = 1;
       }
     }
+    const float* rel_h[2];                                // REL: the bias table at the row's head (rows of G), and its last entry
+    int rel_pos[2];
+    float rel_far[2];
+    if constexpr (REL) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int row = min(row0 + g + 8 * i, rows_total - 1);
+        rel_h[i] = p.rel + (size_t)kvh * p.rel_n * G + row % G;
+        rel_pos[i] = pos0 + row / G;
+        rel_far[i] = __ldg(rel_h[i] + (size_t)(p.rel_n - 1) * G) * 1.4426950408889634f;
+      }
+    }
+    auto scored = [&](float raw) { return (CAP && (!REL || p.cap_log2 > 0.f)) ? softcap_log2(raw, p.cap_slope, p.cap_log2) : raw * p.scale_log2; };
     float m_r[2] = {-INFINITY, -INFINITY}, l_r[2] = {0.f, 0.f};
     float o[DT][4];
 #pragma unroll
@@ -281,14 +296,28 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       float mx[2] = {-INFINITY, -INFINITY};
       // Only a tile at an edge of some row's key range needs the mask; the warp decides once.
       const bool edge = kbase < lo_r[0] || kbase < lo_r[1] || kbase + 16 > hi_r[0] || kbase + 16 > hi_r[1];
-      if (__any_sync(0xffffffffu, edge)) {
+      // keys so near that they have distances of their own take their bias from the table, the others all the last one
+      const bool near = REL && (rel_pos[0] - (kbase + 15) < p.rel_n - 1 || rel_pos[1] - (kbase + 15) < p.rel_n - 1);
+      if (REL && __any_sync(0xffffffffu, near)) {
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
             const int key = kbase + n * 8 + 2 * t4 + (c & 1);
             const int i = c >> 1;
-            const float sl = CAP ? softcap_log2(sc[n][c], p.cap_slope, p.cap_log2) : sc[n][c] * p.scale_log2;
+            const float b = __ldg(rel_h[i] + (size_t)min(max(rel_pos[i] - key, 0), p.rel_n - 1) * G);
+            const float v = (key < hi_r[i] && key >= lo_r[i]) ? fmaf(b, 1.4426950408889634f, scored(sc[n][c])) : -INFINITY;
+            sc[n][c] = v;
+            mx[i] = fmaxf(mx[i], v);
+          }
+      } else if (__any_sync(0xffffffffu, edge)) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const int key = kbase + n * 8 + 2 * t4 + (c & 1);
+            const int i = c >> 1;
+            const float sl = REL ? scored(sc[n][c]) + rel_far[i] : scored(sc[n][c]);
             const float v = (key < hi_r[i] && key >= lo_r[i]) ? sl : -INFINITY;
             sc[n][c] = v;
             mx[i] = fmaxf(mx[i], v);
@@ -298,7 +327,7 @@ attention_tma_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
-            sc[n][c] = CAP ? softcap_log2(sc[n][c], p.cap_slope, p.cap_log2) : sc[n][c] * p.scale_log2;
+            sc[n][c] = REL ? scored(sc[n][c]) + rel_far[c >> 1] : scored(sc[n][c]);
             mx[c >> 1] = fmaxf(mx[c >> 1], sc[n][c]);
           }
       }
@@ -531,20 +560,20 @@ constexpr size_t ta_smem(int hd) {
   return (size_t)TA_STAGES * 2 * TA_BN * hd * 2 + 16 * (hd + 8) * 2 + 2 * TA_STAGES * 8 + 16 + TA_BT_CACHE * 4 + 1024;
 }
 
-template <int HD, bool CAP>
+template <int HD, bool CAP, bool REL>
 static int launch_ta(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& rk, const CUtensorMap& rv,
                      const AttnTmaParams& p, int tiles, cudaStream_t stream) {
   constexpr size_t smem = ta_smem(HD);
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tma_decode_kernel<HD, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attention_tma_decode_kernel<HD, CAP, REL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       set_error("attention_tma: cannot raise the shared memory limit");
       return SLLM_ERR_LAUNCH;
     }
     configured = true;
   }
   dim3 grid((unsigned)tiles * p.nkv, 1, p.num_splits);
-  launch_kernel(attention_tma_decode_kernel<HD, CAP>, grid, TA_THREADS, smem, stream, mk, mv, rk, rv, p);
+  launch_kernel(attention_tma_decode_kernel<HD, CAP, REL>, grid, TA_THREADS, smem, stream, mk, mv, rk, rv, p);
   int rc = launch_status("attention_tma");
   if (rc != SLLM_OK) return rc;
   if (p.num_splits > 1) {
@@ -583,7 +612,8 @@ SLLM_EXPORT int sllm_attention_tma_decode(const void* q, const void* k_cache, co
                                           int max_pages, const int* q_start, const int* ctx_len, const int* tile_seq,
                                           const int* tile_row0, int tiles, int num_splits, int total_tokens, int nq,
                                           int nkv, int hd, int page_size, float scale, int window, int block, const float* sink,
-                                          float softcap, const float* gate, int gate_ld, int* status, cudaStream_t stream) {
+                                          float softcap, const float* gate, int gate_ld, const float* rel, int rel_n, int* status, cudaStream_t stream) {
+  SLLM_REQUIRE(rel == nullptr || rel_n >= 1, "attention_tma: a bias by distance needs its table");
   SLLM_REQUIRE(softcap >= 0.f && (gate == nullptr || gate_ld >= nq), "attention_tma: softcap=%f, gates in rows of %d", softcap, gate_ld);
   SLLM_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_tma: bad head counts nq=%d nkv=%d", nq, nkv);
   SLLM_REQUIRE(sllm_attention_tma_supports(hd, page_size), "attention_tma: head_dim=%d page_size=%d not taken", hd, page_size);
@@ -612,7 +642,8 @@ SLLM_EXPORT int sllm_attention_tma_decode(const void* q, const void* k_cache, co
   p.num_splits = num_splits; p.total_tokens = total_tokens; p.scale_log2 = scale * 1.4426950408889634f;
   p.sink = sink;
   p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
-  p.gate = gate; p.gate_ld = gate_ld;
-  if (softcap > 0.f) return hd == 128 ? launch_ta<128, true>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, true>(mk, mv, rk, rv, p, tiles, stream);
-  return hd == 128 ? launch_ta<128, false>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, false>(mk, mv, rk, rv, p, tiles, stream);
+  p.gate = gate; p.gate_ld = gate_ld; p.rel = rel; p.rel_n = rel_n;
+  if (rel != nullptr) return hd == 128 ? launch_ta<128, true, true>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, true, true>(mk, mv, rk, rv, p, tiles, stream);
+  if (softcap > 0.f) return hd == 128 ? launch_ta<128, true, false>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, true, false>(mk, mv, rk, rv, p, tiles, stream);
+  return hd == 128 ? launch_ta<128, false, false>(mk, mv, rk, rv, p, tiles, stream) : launch_ta<64, false, false>(mk, mv, rk, rv, p, tiles, stream);
 }

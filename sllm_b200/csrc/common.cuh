@@ -69,6 +69,7 @@ __device__ __forceinline__ float block_sum(float v, float* red /* >= 33 floats *
 #define SLLM_ACT_NONE 0
 #define SLLM_ACT_RELU2 1       // max(v, 0)^2
 #define SLLM_ACT_TOKEN 2       // gelu_tanh(v) times the token's own entry of a table
+#define SLLM_ACT_GELU 3        // the exact gelu, v (1 + erf(v / sqrt 2)) / 2
 
 // For SLLM_ACT_TOKEN: column n of row m is multiplied by table[ids[m]][off + n] (rows of `ld`, V of them; ids outside are
 // clamped, the host validates them).
@@ -80,6 +81,7 @@ struct TokenTable {
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+__device__ __forceinline__ float gelu_f32(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
 __device__ __forceinline__ float relu2_f32(float v) { v = fmaxf(v, 0.f); return v * v; }
 __device__ __forceinline__ size_t token_row(const TokenTable& t, int m) {
   int id = t.ids[m];

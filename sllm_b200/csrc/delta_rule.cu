@@ -37,6 +37,9 @@
 //   retention (an instance of its own, ROT):  S <- decay_h S + k v^T;  o = S^T q  with q and k rotated by position over their
 //       first `rot` channels (channel i with i + rot/2, cos and sin from a table) and k then times k_scale: the loader warps
 //       rotate, the walk reads one decay for the whole head.
+//   a state-space recurrence (an instance of its own, SSM):  S <- a S + dt B x^T;  o = S^T C + D x  with dt = softplus(z + dt_bias) and
+//       a = exp(-exp(A_log) dt) one number per token and head; heads share B and C in groups: k = dt B, v = x, r = C, and the walk
+//       reads the token's one decay from the row that holds u in the general form.
 //
 // A second kernel finishes the mixer's output: each head's o over its root mean square, times a gain,
 // times sigmoid(gate logit), in the compute dtype.
@@ -47,7 +50,8 @@ namespace sllm {
 constexpr int DR_COMPUTE = 128;   // threads that walk the tokens (as many again prepare the next chunk)
 constexpr int DR_THREADS = 2 * DR_COMPUTE;
 constexpr int DR_MAX_CHUNK = 16;
-constexpr int DR_RETENTION = 5;
+constexpr int DR_RETENTION = 5, DR_STATE_SPACE = 6;
+constexpr int DR_GENERAL = 0, DR_ROT = 1, DR_SSM = 2;      // the kernel's instances: by `mode`, retention, state space
 
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
 
@@ -72,14 +76,16 @@ struct DeltaParams {
   const float* table = nullptr;        // [max_pos][2][rot / 2], cos then sin
   int rot = 0, max_pos = 0;
   float k_scale = 1.f;
+  const float* skip = nullptr;         // state space: [H] D; dt logits in `gates` at off_dt + h
   int max_len = 0;                     // > 0: requests that bring more tokens are another kernel's (retention.cu)
 };
 
 // RPT: rows of a column per lane (dk <= 8 * RPT = DKP, the padded key size).
 constexpr int DR_SPLIT = 8;
 
-template <int RPT, int CB, bool ROT>
+template <int RPT, int CB, int KIND>
 __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParams p) {
+  constexpr bool ROT = KIND == DR_ROT, SSM = KIND == DR_SSM;
   constexpr int SPLIT = DR_SPLIT, COLS = DR_COMPUTE / SPLIT * CB, DKP = RPT * SPLIT, PER_LANE = (DKP + 31) / 32;
   constexpr int VPL = (COLS + 31) / 32;       // values of v a loader lane brings
   extern __shared__ __align__(16) float sm[];
@@ -93,6 +99,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
   const bool loader = tid >= DR_COMPUTE;
   const int nchunks = (t_end - t_begin + chunk - 1) / chunk;
   const float head_decay = ROT ? __ldg(p.a_log + h) : 0.f;
+  const float head_skip = SSM ? __ldg(p.skip + h) : 0.f;
 
   // a loader warp prepares token after token of chunk c: rows of u, d, a*u, k, r (zeros beyond dk) and v's slice
   auto prepare = [&](int c) {
@@ -146,6 +153,50 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
             s_r[tt * DKP + i] = fmaf(r[q][m], cs[q][m], rp[q][m] * sn[q][m]);
           }
         }
+#pragma unroll
+        for (int m = 0; m < VPL; ++m)
+          if (lane + 32 * m < COLS) s_v[tt * COLS + lane + 32 * m] = v[q][m];
+      }
+      return;
+    }
+    if constexpr (SSM) {
+      float z[TPW];
+      const int kh = h / p.hdiv;
+#pragma unroll
+      for (int q = 0; q < TPW; ++q) {
+        const int tt = lw + q * (DR_COMPUTE / 32);
+        const bool tok = tt < nt;
+        const int t = t0 + (tok ? tt : 0);
+        const float* row = p.proj + (size_t)t * p.ld;
+        z[q] = __ldg(p.gates + (size_t)t * p.ldg + p.off_dt + h);
+#pragma unroll
+        for (int m = 0; m < PER_LANE; ++m) {
+          const int i = lane + 32 * m;
+          const bool in = tok && i < dk;
+          k[q][m] = in ? __ldg(row + p.off_k + kh * dk + i) : 0.f;
+          r[q][m] = in ? __ldg(row + p.off_r + kh * dk + i) : 0.f;
+        }
+#pragma unroll
+        for (int m = 0; m < VPL; ++m) {
+          const int j = c0 + lane + 32 * m;
+          v[q][m] = (tok && lane + 32 * m < COLS && j < dv) ? __ldg(row + p.off_v + h * dv + j) : 0.f;
+        }
+      }
+      const float rate = -expf(__ldg(p.a_log + h)), bias = __ldg(p.dt_bias + h);
+#pragma unroll
+      for (int q = 0; q < TPW; ++q) {
+        const int tt = lw + q * (DR_COMPUTE / 32);
+        if (tt >= nt) break;
+        const float x = z[q] + bias, dt = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+#pragma unroll
+        for (int m = 0; m < PER_LANE; ++m) {
+          const int i = lane + 32 * m;
+          if (i < DKP) {
+            s_k[tt * DKP + i] = k[q][m] * dt;
+            s_r[tt * DKP + i] = r[q][m];
+          }
+        }
+        if (lane == 0) s_u[tt * DKP] = expf(rate * dt);
 #pragma unroll
         for (int m = 0; m < VPL; ++m)
           if (lane + 32 * m < COLS) s_v[tt * COLS + lane + 32 * m] = v[q][m];
@@ -312,14 +363,15 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
         }
 #pragma unroll
         for (int cc = 0; cc < CB; ++cc) us[cc] = ut[cc] = o[cc] = o2[cc] = 0.f;
-        if constexpr (ROT) {
+        if constexpr (ROT || SSM) {
+          const float decay = SSM ? b[tt * DKP] : head_decay;
 #pragma unroll
           for (int n = 0; n < RPT; n += 2) {
             const float ka = k[n * SPLIT], kb = k[(n + 1) * SPLIT], ra = r[n * SPLIT], rb = r[(n + 1) * SPLIT];
 #pragma unroll
             for (int cc = 0; cc < CB; ++cc) {
-              s[n][cc] = fmaf(ka, vv[cc], head_decay * s[n][cc]);
-              s[n + 1][cc] = fmaf(kb, vv[cc], head_decay * s[n + 1][cc]);
+              s[n][cc] = fmaf(ka, vv[cc], decay * s[n][cc]);
+              s[n + 1][cc] = fmaf(kb, vv[cc], decay * s[n + 1][cc]);
               o[cc] = fmaf(s[n][cc], ra, o[cc]);
               o2[cc] = fmaf(s[n + 1][cc], rb, o2[cc]);
             }
@@ -410,6 +462,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
           float tot = (hi ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi ? a0 : a1, 2);
           tot += __shfl_xor_sync(0xffffffffu, tot, 4);
           const int mine = col + 2 * (rs & 1) + ((rs >> 1) & 1);
+          if constexpr (SSM) tot = fmaf(head_skip, b[5 * chunk * DKP + tt * COLS + mine - c0], tot);
           if (rs < 4 && mine < dv) p.out[(size_t)(t0 + tt) * p.H * dv + h * dv + mine] = tot;
         } else {
 #pragma unroll
@@ -417,6 +470,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaParam
             float tot = o[cc] + o2[cc];
 #pragma unroll
             for (int w = 1; w < SPLIT; w <<= 1) tot += __shfl_xor_sync(0xffffffffu, tot, w);
+            if constexpr (SSM) tot = fmaf(head_skip, vv[cc], tot);
             if (rs == 0 && col + cc < dv) p.out[(size_t)(t0 + tt) * p.H * dv + h * dv + col + cc] = tot;
           }
         }
@@ -504,7 +558,7 @@ using namespace sllm;
 
 SLLM_EXPORT int sllm_delta_rule_supports(int dk, int dv) { return dk >= 1 && dk <= 256 && dv >= 1 && dv <= 65535 * 16; }
 
-template <int RPT, int CB, bool ROT>
+template <int RPT, int CB, int KIND>
 static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   constexpr int DKP = RPT * DR_SPLIT, DR_COLS = DR_COMPUTE / DR_SPLIT * CB;
   const size_t per_token = (size_t)(5 * DKP + DR_COLS) * sizeof(float);
@@ -515,7 +569,7 @@ static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   const size_t smem = 2 * per_token * chunk;
   static size_t allowed = 48 * 1024;          // (per instantiation: what the kernel has been told it may use)
   if (smem > allowed) {
-    if (cudaFuncSetAttribute(delta_rule_kernel<RPT, CB, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(delta_rule_kernel<RPT, CB, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       cudaGetLastError();
       set_error("delta_rule: the kernel's shared memory could not be raised");
       return SLLM_ERR_LAUNCH;
@@ -523,7 +577,7 @@ static int launch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
     allowed = smem;
   }
   const dim3 grid((unsigned)S, (unsigned)p.H, (unsigned)((p.dv + DR_COLS - 1) / DR_COLS));
-  launch_kernel(delta_rule_kernel<RPT, CB, ROT>, grid, DR_THREADS, smem, stream, p);
+  launch_kernel(delta_rule_kernel<RPT, CB, KIND>, grid, DR_THREADS, smem, stream, p);
   return launch_status("delta_rule");
 }
 
@@ -552,8 +606,9 @@ static int dispatch_delta_rule(DeltaParams p, int S, cudaStream_t stream) {
   // enough (request, head, 64 columns) for every SM: four columns a lane; else one, in four times the CTAs
   const bool wide = (long)S * p.H * ((dv + 63) / 64) >= (long)num_sms();
 #define SLLM_DR(RPT_)                                                                                                         \
-  return p.mode == DR_RETENTION ? (wide ? launch_delta_rule<RPT_, 4, true>(p, S, stream) : launch_delta_rule<RPT_, 1, true>(p, S, stream)) \
-                                : (wide ? launch_delta_rule<RPT_, 4, false>(p, S, stream) : launch_delta_rule<RPT_, 1, false>(p, S, stream))
+  return p.mode == DR_RETENTION ? (wide ? launch_delta_rule<RPT_, 4, DR_ROT>(p, S, stream) : launch_delta_rule<RPT_, 1, DR_ROT>(p, S, stream)) \
+         : p.mode == DR_STATE_SPACE ? (wide ? launch_delta_rule<RPT_, 4, DR_SSM>(p, S, stream) : launch_delta_rule<RPT_, 1, DR_SSM>(p, S, stream)) \
+                                    : (wide ? launch_delta_rule<RPT_, 4, DR_GENERAL>(p, S, stream) : launch_delta_rule<RPT_, 1, DR_GENERAL>(p, S, stream))
   if (dk <= 16) SLLM_DR(2);
   if (dk <= 32) SLLM_DR(4);
   if (dk <= 64) SLLM_DR(8);
@@ -657,6 +712,26 @@ SLLM_EXPORT int sllm_retention(const float* proj, int ld, int off_q, int off_k, 
   p.mode = DR_RETENTION; p.hdiv = 1; p.gates = nullptr; p.ldg = p.off_b = p.off_dt = 0; p.a_log = decay; p.dt_bias = nullptr;
   p.r_scale = 1.f; p.inv_tau = 1.f;
   p.positions = positions; p.table = table; p.rot = rot; p.max_pos = max_pos > 0 ? max_pos : 1; p.k_scale = k_scale;
+  p.max_len = max_len;
+  if (max_len > 0 && (p.max_q <= 0 || p.max_q > max_len)) p.max_q = max_len;
+  return dispatch_delta_rule(p, S, stream);
+}
+
+// A state-space recurrence over x | B | C columns of `xbc` [T, ldx] (x head by head, B and C group by group: head h uses group h / (H / groups)) with step
+// logits at columns off_dt + h of `dtp` [T, ldd].  max_len > 0: requests that bring more tokens are left alone.
+SLLM_EXPORT int sllm_state_space(const float* xbc, int ldx, const float* dtp, int ldd, int off_dt, const float* dt_bias, const float* a_log,
+                                 const float* skip, float* state, const int* q_start, const int* state_slots, float* out, int S, int H, int groups,
+                                 int N, int dv, int max_q, int max_len, cudaStream_t stream) {
+  SLLM_REQUIRE(S >= 0 && H > 0 && H <= 65535 && groups > 0 && H % groups == 0, "state_space: bad sizes S=%d H=%d groups=%d", S, H, groups);
+  SLLM_REQUIRE(sllm_delta_rule_supports(N, dv), "state_space: a state of %d rows and %d columns is outside 1..256 rows", N, dv);
+  SLLM_REQUIRE(ldx >= H * dv + 2 * groups * N && off_dt >= 0 && off_dt + H <= ldd, "state_space: columns outside the inputs' %d and %d", ldx, ldd);
+  if (S == 0) return SLLM_OK;
+  DeltaParams p;
+  p.proj = xbc; p.decay = xbc; p.a_bias = nullptr; p.state = state; p.q_start = q_start; p.state_slots = state_slots;
+  p.out = out; p.ld = ldx; p.off_v = 0; p.off_k = H * dv; p.off_r = H * dv + groups * N; p.off_a = 0; p.H = H; p.dk = N; p.dv = dv;
+  p.chunk = 1; p.max_q = max_q;
+  p.mode = DR_STATE_SPACE; p.hdiv = H / groups; p.gates = dtp; p.ldg = ldd; p.off_b = 0; p.off_dt = off_dt; p.a_log = a_log; p.dt_bias = dt_bias;
+  p.r_scale = 1.f; p.inv_tau = 1.f; p.skip = skip;
   p.max_len = max_len;
   if (max_len > 0 && (p.max_q <= 0 || p.max_q > max_len)) p.max_q = max_len;
   return dispatch_delta_rule(p, S, stream);

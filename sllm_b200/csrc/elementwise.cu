@@ -386,7 +386,7 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, siz
 }
 
 // ---------------------------------------------------------------------------
-// out[t, n] = max(x, 0)^2, or gelu_tanh(x) * table[ids[t], off + n]: behind products whose kernel has no such epilogue; x may
+// out[t, n] = max(x, 0)^2, the exact gelu of x, or gelu_tanh(x) * table[ids[t], off + n]: behind products whose kernel has no such epilogue; x may
 // be a stack of k-split partial sums
 // ---------------------------------------------------------------------------
 template <typename TI, typename TT, typename TO>
@@ -401,6 +401,8 @@ plain_act_kernel(const TI* __restrict__ x, int parts, size_t part_stride, TO* __
     float y;
     if (act == SLLM_ACT_RELU2) {
       y = relu2_f32(v);
+    } else if (act == SLLM_ACT_GELU) {
+      y = gelu_f32(v);
     } else {
       const int t = (int)(e / N), n = (int)(e % N);
       y = gelu_tanh_f32(v) * to_f32(reinterpret_cast<const TT*>(token.table)[token_row(token, t) + n]);
@@ -547,10 +549,10 @@ SLLM_EXPORT int sllm_softcap(float* x, long long n, float cap, cudaStream_t stre
   return launch_status("softcap");
 }
 
-// act: SLLM_ACT_RELU2, or SLLM_ACT_TOKEN with a table of the output's dtype
+// act: SLLM_ACT_RELU2, SLLM_ACT_GELU, or SLLM_ACT_TOKEN with a table of the output's dtype
 SLLM_EXPORT int sllm_plain_act(const void* x, int in_dtype, int parts, size_t part_stride, void* out, int out_dtype, int T, int N, int act, const void* token_table,
                                const int* token_ids, int token_off, int token_ld, int token_rows, cudaStream_t stream) {
-  SLLM_REQUIRE(T >= 0 && N > 0 && parts >= 1 && (act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN), "plain_act: bad sizes T=%d N=%d act=%d", T, N, act);
+  SLLM_REQUIRE(T >= 0 && N > 0 && parts >= 1 && (act == SLLM_ACT_RELU2 || act == SLLM_ACT_GELU || act == SLLM_ACT_TOKEN), "plain_act: bad sizes T=%d N=%d act=%d", T, N, act);
   SLLM_REQUIRE(act != SLLM_ACT_TOKEN || (token_table && token_ids && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld),
                "plain_act: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
   if (T == 0) return SLLM_OK;

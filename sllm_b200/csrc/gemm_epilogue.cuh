@@ -13,6 +13,7 @@ namespace sllm {
 #define TG_EPI_GELU 4      // like TG_EPI_SILU with gelu_tanh(gate + bias) * (up + bias), the bias interleaved like the columns
 #define TG_EPI_RELU2 5     // bfloat16 out[M, N] = max(product, 0)^2 (no bias)
 #define TG_EPI_TOKEN 6     // bfloat16 out[M, N] = gelu_tanh(product) * the token's entry of a table (no bias); see TgExtra::token
+#define TG_EPI_GELU_ERF 7  // bfloat16 out[M, N] = the exact gelu of the product (no bias)
 #define TG_EPI_RESID 3     // residual[M, N] (float32) += the product (+ bias), in place; see TgExtra
 
 // What an epilogue may do beyond its store, for the RMSNorm that a prompt portion's products take apart
@@ -48,12 +49,15 @@ __device__ __forceinline__ void tg_scale(uint32_t (&r)[32], float s) {
   for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * s);
 }
 
-// what TG_EPI_RELU2 and TG_EPI_TOKEN do to the columns n .. n + 31 of row m before the bfloat16 store
+// what TG_EPI_RELU2, TG_EPI_GELU_ERF and TG_EPI_TOKEN do to the columns n .. n + 31 of row m before the bfloat16 store
 template <int EPI>
 __device__ __forceinline__ void tg_activate(uint32_t (&r)[32], int m, int n, int M, int N, const TgExtra& e) {
   if constexpr (EPI == TG_EPI_RELU2) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(relu2_f32(__uint_as_float(r[i])));
+  } else if constexpr (EPI == TG_EPI_GELU_ERF) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(gelu_f32(__uint_as_float(r[i])));
   } else if constexpr (EPI == TG_EPI_TOKEN) {
     if (m >= M) return;
     const __nv_bfloat16* row = reinterpret_cast<const __nv_bfloat16*>(e.token.table) + token_row(e.token, m) + n;

@@ -641,7 +641,7 @@ SLLM_EXPORT int sllm_gemm_pair(const void* A, const void* W, const float* bias, 
   SLLM_REQUIRE(status != nullptr, "gemm_pair: a status word is required");
   SLLM_REQUIRE(!tg_gated(epilogue) || N % 16 == 0, "gemm_pair: the gated epilogues need N %% 16 == 0");
   TgExtra extra;
-  SLLM_REQUIRE((epilogue != TG_EPI_RELU2 && epilogue != TG_EPI_TOKEN) || bias == nullptr, "gemm_pair: epilogue %d takes no bias", epilogue);
+  SLLM_REQUIRE((epilogue != TG_EPI_RELU2 && epilogue != TG_EPI_TOKEN && epilogue != TG_EPI_GELU_ERF) || bias == nullptr, "gemm_pair: epilogue %d takes no bias", epilogue);
   if (epilogue == TG_EPI_TOKEN) {
     SLLM_REQUIRE(token_table != nullptr && token_ids != nullptr && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld,
                  "gemm_pair: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);
@@ -698,6 +698,7 @@ SLLM_EXPORT int sllm_gemm_pair(const void* A, const void* W, const float* bias, 
     case TG_EPI_SILU: GO(TG_EPI_SILU)
     case TG_EPI_GELU: GO(TG_EPI_GELU)
     case TG_EPI_RELU2: GO(TG_EPI_RELU2)
+    case TG_EPI_GELU_ERF: GO(TG_EPI_GELU_ERF)
     case TG_EPI_TOKEN:
       return wide == 2 ? launch_tp<TG_EPI_TOKEN, 128>(ma, mw, bias, out, M, N, K, status, stream, extra, ksplits, kb_per_split)
                        : launch_tp<TG_EPI_TOKEN, 256>(ma, mw, bias, out, M, N, K, status, stream, extra, ksplits, kb_per_split);

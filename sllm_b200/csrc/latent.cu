@@ -200,9 +200,34 @@ head_linear_mma_kernel(const TX* __restrict__ x, int ldx, int xoff, const __nv_b
   }
 }
 
+// out[t, i] = x[t, off + i] / rms * gain[i]: a CTA per token (the latent queries go through)
+template <typename TO>
+__global__ void norm_cols_kernel(const float* __restrict__ x, int ld, int off, int n, const float* __restrict__ gain, float eps, TO* __restrict__ out) {
+  __shared__ float red[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* row = x + (size_t)blockIdx.x * ld + off;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+  TO* dst = out + (size_t)blockIdx.x * n;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f32<TO>(row[i] * inv * gain[i]);
+}
+
 }  // namespace sllm
 
 using namespace sllm;
+
+SLLM_EXPORT int sllm_norm_cols(const float* x, int ld, int off, int n, const float* gain, float eps, void* out, int out_dtype, int T, cudaStream_t stream) {
+  SLLM_REQUIRE(T >= 0 && n > 0 && off >= 0 && off + n <= ld && gain != nullptr, "norm_cols: columns %d..%d of %d", off, off + n, ld);
+  if (T == 0) return SLLM_OK;
+  const int threads = n >= 512 ? 256 : 128;
+  if (out_dtype == SLLM_F32) launch_kernel(norm_cols_kernel<float>, (unsigned)T, threads, 0, stream, x, ld, off, n, gain, eps, (float*)out);
+  else if (out_dtype == SLLM_BF16) launch_kernel(norm_cols_kernel<__nv_bfloat16>, (unsigned)T, threads, 0, stream, x, ld, off, n, gain, eps, (__nv_bfloat16*)out);
+  else SLLM_REQUIRE(false, "norm_cols: unknown dtype %d", out_dtype);
+  return launch_status("norm_cols");
+}
 
 SLLM_EXPORT int sllm_latent_rope_write(const float* proj, int ld, int off, int rank, int tail, int rot, const float* gain, float eps,
                                        const int* positions, const float* table, int max_pos, const int* slot_mapping, void* cache,

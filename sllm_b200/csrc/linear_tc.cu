@@ -47,6 +47,7 @@ struct LtCfg {
 #define LT_EPI_BF16 1
 #define LT_EPI_SILU 2
 #define LT_EPI_RELU2 3     // bfloat16 max(product, 0)^2
+#define LT_EPI_GELU_ERF 4  // bfloat16 exact gelu of the product
 
 template <int BN, int EPI>
 __global__ void __launch_bounds__(192, 1)
@@ -216,7 +217,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
               for (int j = 0; j < 32; ++j)
                 if (c0 + j < M) {
                   const float v = __uint_as_float(r[j]) + bv;
-                  o[(size_t)(c0 + j) * N] = __float2bfloat16_rn(EPI == LT_EPI_RELU2 ? relu2_f32(v) : v);
+                  o[(size_t)(c0 + j) * N] = __float2bfloat16_rn(EPI == LT_EPI_RELU2 ? relu2_f32(v) : EPI == LT_EPI_GELU_ERF ? gelu_f32(v) : v);
                 }
             }
           }
@@ -307,6 +308,7 @@ SLLM_EXPORT int sllm_linear_tc(const void* x, const void* W, const float* bias, 
       case LT_EPI_BF16: LT_LAUNCH(64, LT_EPI_BF16);
       case LT_EPI_SILU: LT_LAUNCH(64, LT_EPI_SILU);
       case LT_EPI_RELU2: LT_LAUNCH(64, LT_EPI_RELU2);
+      case LT_EPI_GELU_ERF: LT_LAUNCH(64, LT_EPI_GELU_ERF);
     }
   } else {
     switch (epilogue) {
@@ -314,6 +316,7 @@ SLLM_EXPORT int sllm_linear_tc(const void* x, const void* W, const float* bias, 
       case LT_EPI_BF16: LT_LAUNCH(128, LT_EPI_BF16);
       case LT_EPI_SILU: LT_LAUNCH(128, LT_EPI_SILU);
       case LT_EPI_RELU2: LT_LAUNCH(128, LT_EPI_RELU2);
+      case LT_EPI_GELU_ERF: LT_LAUNCH(128, LT_EPI_GELU_ERF);
     }
   }
 #undef LT_LAUNCH

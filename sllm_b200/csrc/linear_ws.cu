@@ -280,6 +280,7 @@ linear_ws_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __res
       }
     } else if (valid) {
       if (act == SLLM_ACT_RELU2) v = relu2_f32(v);
+      else if (act == SLLM_ACT_GELU) v = gelu_f32(v);
       else if (act == SLLM_ACT_TOKEN) v = gelu_tanh_f32(v) * __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(token.table)[token_row(token, tok) + n]);
       out[(size_t)tok * N + n] = from_f32<OUT>(v);
     }
@@ -342,7 +343,7 @@ SLLM_EXPORT int sllm_linear_ws(const void* x, const void* W, const float* bias, 
                                int M, int N, int K, const float* ssq_in, int parts_in, float eps_in, int width_in,
                                const float* gain, void* xg_out, float* ssq_out, int act, const void* token_table, const int* token_ids,
                                int token_off, int token_ld, int token_rows, cudaStream_t stream) {
-  SLLM_REQUIRE(act == SLLM_ACT_NONE || ((act == SLLM_ACT_RELU2 || act == SLLM_ACT_TOKEN) && residual == nullptr),
+  SLLM_REQUIRE(act == SLLM_ACT_NONE || ((act == SLLM_ACT_RELU2 || act == SLLM_ACT_GELU || act == SLLM_ACT_TOKEN) && residual == nullptr),
                "linear_ws: activation %d (0 none, 1 relu squared, 2 gelu times the tokens' table), not with a residual", act);
   SLLM_REQUIRE(act != SLLM_ACT_TOKEN || (token_table && token_ids && token_rows > 0 && token_off >= 0 && token_off + N <= token_ld),
                "linear_ws: the tokens' table has rows of %d, columns %d..%d are wanted", token_ld, token_off, token_off + N);

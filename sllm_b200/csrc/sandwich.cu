@@ -14,8 +14,10 @@
 //     request's slot in a short serial pass, then every warp walks its run again from its entry state and writes.
 //   * gated_clamp_act: y = g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit), gate and
 //     up columns alternating in blocks; optionally times a routing weight per (token, expert) that a mixture of
-//     experts carries on its activation rows (zero: not chosen, and the columns are not read).
-//   * moe_route_top_softmax: the `top` largest router logits win; their weights are the softmax over the winners alone.
+//     experts carries on its activation rows (zero: not chosen, and the columns are not read); the last `tail` columns may belong to an
+//     expert of another size, with the last weight.
+//   * moe_route_top_softmax: the `top` largest router logits win; their weights are the softmax over the winners alone.  A column behind
+//     the experts' logits may gate an expert every token uses: its sigmoid is the last of the dense weights.
 //   * rope_cols: per head, a few columns of a float32 product rotated by position (rotate-half layout) and written
 //     into a slice of wider per-head rows (the rotated part of a query that otherwise lives in a latent space).
 #include <math.h>
@@ -276,12 +278,12 @@ mingru_scan_kernel(const float* __restrict__ proj, int ld, int off_z, int off_x,
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256)
 gated_clamp_act_kernel(const TI* __restrict__ gu, const float* __restrict__ dense, TO* __restrict__ out, int N, int E, int ff,
-                       int il, float limit, float alpha, int act) {
+                       int tail, int il, float limit, float alpha, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < N; c += gridDim.y * blockDim.x) {
-    const float w = dense != nullptr ? dense[t * E + c / ff] : 1.f;
+    const float w = dense != nullptr ? dense[t * E + (c < N - tail ? c / ff : E - 1)] : 1.f;
     float y = 0.f;
     if (w != 0.f) {
       const TI* p = gu + t * 2 * N + (size_t)(c / il) * 2 * il + c % il;
@@ -300,12 +302,12 @@ gated_clamp_act_kernel(const TI* __restrict__ gu, const float* __restrict__ dens
 // bfloat16 in and out, blocks of 8 (or a multiple): eight columns a thread, one 16-byte load each of gate and up
 __global__ void __launch_bounds__(256)
 gated_clamp_act_vec_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ dense, __nv_bfloat16* __restrict__ out,
-                           int N, int E, int ff, int il, float limit, float alpha, int act) {
+                           int N, int E, int ff, int tail, int il, float limit, float alpha, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
   for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < N; c += gridDim.y * blockDim.x * 8) {
-    const float w = dense != nullptr ? dense[t * E + c / ff] : 1.f;
+    const float w = dense != nullptr ? dense[t * E + (c < N - tail ? c / ff : E - 1)] : 1.f;
     uint4 res = make_uint4(0u, 0u, 0u, 0u);
     if (w != 0.f) {
       const __nv_bfloat16* p = gu + t * 2 * N + (size_t)(c / il) * 2 * il + c % il;
@@ -333,7 +335,7 @@ constexpr int RS_WARPS = 4;
 
 // a warp per token
 __global__ void __launch_bounds__(RS_WARPS * 32)
-moe_route_top_softmax_kernel(const float* __restrict__ logits, int T, int E, int top, float scale, float* __restrict__ dense,
+moe_route_top_softmax_kernel(const float* __restrict__ logits, int ld, int T, int E, int gated, int top, float scale, float* __restrict__ dense,
                              int* __restrict__ idx, float* __restrict__ wts) {
   extern __shared__ float sm[];
   pdl_launch_dependents();
@@ -342,11 +344,13 @@ moe_route_top_softmax_kernel(const float* __restrict__ logits, int T, int E, int
   const int t = blockIdx.x * RS_WARPS + warp;
   if (t >= T) return;
   float* choice = sm + (size_t)warp * E;
-  const float* z = logits + (size_t)t * E;
+  const float* z = logits + (size_t)t * ld;
+  dense += (size_t)t * (E + gated);
   for (int e = lane; e < E; e += 32) {
     choice[e] = z[e];
-    dense[(size_t)t * E + e] = 0.f;
+    dense[e] = 0.f;
   }
+  if (gated && lane == 0) dense[E] = sw_sigmoid(z[E]);
   __syncwarp();
   float zmax = 0.f, sum = 0.f;
   for (int n = 0; n < top; ++n) {
@@ -378,7 +382,7 @@ moe_route_top_softmax_kernel(const float* __restrict__ logits, int T, int E, int
     for (int n = 0; n < top; ++n) {
       const float w = wts[(size_t)t * top + n] * inv;
       wts[(size_t)t * top + n] = w;
-      dense[(size_t)t * E + idx[(size_t)t * top + n]] = w;
+      dense[idx[(size_t)t * top + n]] = w;
     }
 }
 
@@ -497,25 +501,26 @@ SLLM_EXPORT int sllm_mingru_scan(const float* proj, int ld, int off_z, int off_x
 }
 
 SLLM_EXPORT int sllm_gated_clamp_act(const void* gu, int in_dtype, const float* dense, void* out, int out_dtype, int T, int N, int E,
-                                     int ff, int interleave, float limit, float alpha, int act, cudaStream_t stream) {
+                                     int ff, int tail, int interleave, float limit, float alpha, int act, cudaStream_t stream) {
   SLLM_REQUIRE(T >= 0 && N >= 1 && ff >= 1 && interleave >= 1 && N % interleave == 0, "gated_clamp_act: bad sizes T=%d N=%d ff=%d blocks of %d",
                T, N, ff, interleave);
-  SLLM_REQUIRE(dense == nullptr || (E >= 1 && (long)E * ff == N && ff % interleave == 0),
-               "gated_clamp_act: %d experts of %d columns in blocks of %d do not make %d", E, ff, interleave, N);
+  SLLM_REQUIRE(tail >= 0 && (tail == 0 || (dense != nullptr && tail % interleave == 0)), "gated_clamp_act: %d columns of an expert of its own in blocks of %d", tail, interleave);
+  SLLM_REQUIRE(dense == nullptr || (E >= 1 && (long)(E - (tail > 0)) * ff + tail == N && ff % interleave == 0),
+               "gated_clamp_act: %d experts of %d columns (and %d) in blocks of %d do not make %d", E, ff, tail, interleave, N);
   if (T == 0) return SLLM_OK;
-  if (in_dtype == SLLM_BF16 && out_dtype == SLLM_BF16 && interleave % 8 == 0 && (dense == nullptr || ff % 8 == 0) &&
+  if (in_dtype == SLLM_BF16 && out_dtype == SLLM_BF16 && interleave % 8 == 0 && (dense == nullptr || (ff % 8 == 0 && tail % 8 == 0)) &&
       (uintptr_t)gu % 16 == 0 && (uintptr_t)out % 16 == 0) {
     int by = (N / 8 + 255) / 256;
     if (by > 64) by = 64;
     launch_kernel(gated_clamp_act_vec_kernel, dim3((unsigned)T, (unsigned)by), 256, 0, stream, (const __nv_bfloat16*)gu, dense,
-                  (__nv_bfloat16*)out, N, E, ff, interleave, limit, alpha, act);
+                  (__nv_bfloat16*)out, N, E, ff, tail, interleave, limit, alpha, act);
     return launch_status("gated_clamp_act");
   }
   int by = (N + 255) / 256;
   if (by > 64) by = 64;
   const dim3 grid((unsigned)T, (unsigned)by);
 #define LAUNCH(TI, TO) \
-  launch_kernel(gated_clamp_act_kernel<TI, TO>, grid, 256, 0, stream, (const TI*)gu, dense, (TO*)out, N, E, ff, interleave, limit, alpha, act)
+  launch_kernel(gated_clamp_act_kernel<TI, TO>, grid, 256, 0, stream, (const TI*)gu, dense, (TO*)out, N, E, ff, tail, interleave, limit, alpha, act)
   if (in_dtype == SLLM_F32 && out_dtype == SLLM_F32) LAUNCH(float, float);
   else if (in_dtype == SLLM_F32 && out_dtype == SLLM_BF16) LAUNCH(float, __nv_bfloat16);
   else if (in_dtype == SLLM_BF16 && out_dtype == SLLM_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
@@ -524,14 +529,15 @@ SLLM_EXPORT int sllm_gated_clamp_act(const void* gu, int in_dtype, const float* 
   return launch_status("gated_clamp_act");
 }
 
-SLLM_EXPORT int sllm_moe_route_top_softmax(const float* logits, int T, int E, int top, float scale, float* dense, int* idx, float* wts,
+SLLM_EXPORT int sllm_moe_route_top_softmax(const float* logits, int ld, int T, int E, int gated, int top, float scale, float* dense, int* idx, float* wts,
                                            cudaStream_t stream) {
+  SLLM_REQUIRE((gated == 0 || gated == 1) && E + gated <= ld, "moe_route_top_softmax: %d experts and %d gates in rows of %d", E, gated, ld);
   SLLM_REQUIRE(T >= 0 && E >= 1 && top >= 1 && top <= E, "moe_route_top_softmax: bad sizes T=%d E=%d top=%d", T, E, top);
   const size_t smem = (size_t)RS_WARPS * E * sizeof(float);
   SLLM_REQUIRE(smem <= 48 * 1024, "moe_route_top_softmax: %d experts are more than the kernel keeps in shared memory", E);
   if (T == 0) return SLLM_OK;
-  launch_kernel(moe_route_top_softmax_kernel, (unsigned)((T + RS_WARPS - 1) / RS_WARPS), RS_WARPS * 32, smem, stream, logits, T, E,
-                top, scale, dense, idx, wts);
+  launch_kernel(moe_route_top_softmax_kernel, (unsigned)((T + RS_WARPS - 1) / RS_WARPS), RS_WARPS * 32, smem, stream, logits, ld, T, E,
+                gated, top, scale, dense, idx, wts);
   return launch_status("moe_route_top_softmax");
 }
 

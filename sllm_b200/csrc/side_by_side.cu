@@ -8,7 +8,9 @@
 //                           Without gains the heads are not normed; `q_mul` (one number per query head) multiplies the
 //                           query head (a factor on its scores).
 //                           Key and value sizes may differ: the cache's head is D >= both, the rest is zeros.
-//   short_conv_silu         y[t, c] = silu(sum_j w[c, taps-1-j] x[t-j, c]) over a request's own tokens; the taps-1 inputs
+//   whole_norm_kv_write     the same job where the norms run over all query rows and all key rows at once: biases, both norms, a factor
+//                           on the query that grows with the position, the cache write; a CTA per token, no rotation.
+//   short_conv_silu         y[t, c] = silu(sum_j w[c, taps-1-j] x[t-j, c] + bias[c]) over a request's own tokens; the taps-1 inputs
 //                           before a portion come from the request's state row, zeros before the sequence starts.
 //   short_conv_state        the state row receives the portion's last taps-1 inputs (older ones move up).
 //   norm_mean_add           stream += (a / rms(a) * ga + b / rms(b) * gb) / 2.
@@ -77,11 +79,62 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ qkv, int ld, const float*
   for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<TC>(d < dim ? x[d] * inv * (gain ? gain[d] : 1.f) : 0.f);
 }
 
+// A CTA per token; the token's queries and keys (sums of `parts` partial products, plus their biases) wait in shared memory for the
+// root mean squares.  q_every >= 1: the query's factor 1 + q_coef ln(floor((p + 1) / q_every) + 1).
+template <typename TC>
+__global__ void __launch_bounds__(256)
+whole_norm_kv_write_kernel(const float* __restrict__ qkv, int parts, size_t part_stride, int ld, const float* __restrict__ bias,
+                           const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, const int* __restrict__ positions,
+                           float q_coef, int q_every, int nq, int nkv, int dim, int vdim, int D, const int* __restrict__ slot_mapping,
+                           int page_size, int num_pages, TC* __restrict__ k_cache, TC* __restrict__ v_cache, TC* __restrict__ q_out) {
+  extern __shared__ float wn_x[];                                    // [(nq + nkv) * dim]
+  __shared__ float red[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const float* row = qkv + (size_t)t * ld;
+  auto value = [&](int c) {
+    float v = row[c];
+    for (int p = 1; p < parts; ++p) v += row[p * part_stride + c];
+    return bias != nullptr ? v + bias[c] : v;
+  };
+  int slot = -1;
+  if (slot_mapping != nullptr) {
+    slot = slot_mapping[t];
+    if (slot >= 0 && slot / page_size >= num_pages) slot = -1;
+  }
+  const int Q = nq * dim, K = slot >= 0 ? nkv * dim : 0;
+  float sq = 0.f, sk = 0.f;
+  for (int c = tid; c < Q + K; c += blockDim.x) {
+    const float v = value(c);
+    wn_x[c] = v;
+    if (c < Q) sq = fmaf(v, v, sq);
+    else sk = fmaf(v, v, sk);
+  }
+  sq = block_sum(sq, red);
+  float qi = 1.0f / sqrtf(sq / (float)Q + eps);
+  if (q_coef != 0.f) qi *= 1.0f + q_coef * logf((float)((positions[t] + 1) / q_every) + 1.0f);
+  TC* q = q_out + (size_t)t * nq * D;
+  for (int e = tid; e < nq * D; e += blockDim.x) {
+    const int h = e / D, d = e - h * D, c = h * dim + d;
+    q[e] = from_f32<TC>(d < dim ? wn_x[c] * qi * q_gain[c] : 0.f);
+  }
+  if (slot < 0) return;                                              // (the whole CTA: no place to write to)
+  sk = block_sum(sk, red);
+  const float ki = 1.0f / sqrtf(sk / (float)(nkv * dim) + eps);
+  const size_t head = (size_t)page_size * D, base = (size_t)(slot / page_size) * nkv * head + (size_t)(slot % page_size) * D;
+  for (int e = tid; e < nkv * D; e += blockDim.x) {
+    const int h = e / D, d = e - h * D, c = h * dim + d;
+    k_cache[base + h * head + d] = from_f32<TC>(d < dim ? wn_x[Q + c] * ki * k_gain[c] : 0.f);
+    v_cache[base + h * head + d] = from_f32<TC>(d < vdim ? value(Q + nkv * dim + h * vdim + d) : 0.f);
+  }
+}
+
 // grid (T, ceil(C / 256)): a thread per (token, channel).  MODE 0: silu of the convolution; MODE 1: the input plus its
 // convolution (a convolution in front of a sublayer that keeps the sublayer's input as it was beside it).
 template <int MODE, typename TO>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, int taps,
+short_conv_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, const float* __restrict__ bias, int taps,
                   const float* __restrict__ state, const int* __restrict__ seq_of_token, const int* __restrict__ q_start,
                   const int* __restrict__ state_slots, TO* __restrict__ out, int C, int own_state) {
   pdl_launch_dependents();
@@ -99,6 +152,7 @@ short_conv_kernel(const float* __restrict__ x, int ld, int off, const float* __r
     acc = fmaf(wc[taps - 1 - j], v, acc);
     now = v;
   }
+  if (bias != nullptr) acc += bias[c];
   out[(size_t)t * C + c] = from_f32<TO>(MODE == 0 ? sbs_silu(acc) : now + acc);
   if (own_state) {                                      // every request brings one token: its thread is the state's only reader
     for (int i = 0; i + 1 < taps; ++i) st[i] = i + 2 < taps ? st[i + 1] : now;
@@ -109,7 +163,7 @@ short_conv_kernel(const float* __restrict__ x, int ld, int off, const float* __r
 // weights and of the state.  The sums run in the scalar kernel's order, so both give the same bits.
 template <int MODE, int TAPS, typename TO>
 __global__ void __launch_bounds__(128)
-short_conv_vec4_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, float* __restrict__ state,
+short_conv_vec4_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                        const int* __restrict__ seq_of_token, const int* __restrict__ q_start, const int* __restrict__ state_slots,
                        TO* __restrict__ out, int C, int own_state) {
   constexpr int KEEP = TAPS - 1;
@@ -154,6 +208,10 @@ short_conv_vec4_kernel(const float* __restrict__ x, int ld, int off, const float
 #pragma unroll
     for (int i = 0; i < 4; ++i) acc[i] = fmaf(wl[i * TAPS + j], now[i], acc[i]);
   }
+  if (bias != nullptr) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[i] += bias[c + i];
+  }
   float y[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) y[i] = MODE == 0 ? sbs_silu(acc[i]) : now[i] + acc[i];
@@ -184,7 +242,7 @@ short_conv_vec4_kernel(const float* __restrict__ x, int ld, int off, const float
 // kernels above: the same bits.  grid (ceil(T / RUN), ceil(C / 512)).
 template <int MODE, int TAPS, typename TO, int RUN>
 __global__ void __launch_bounds__(128)
-short_conv_run_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, const float* __restrict__ state,
+short_conv_run_kernel(const float* __restrict__ x, int ld, int off, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ state,
                       const int* __restrict__ seq_of_token, const int* __restrict__ q_start, const int* __restrict__ state_slots,
                       TO* __restrict__ out, int C, int T) {
   constexpr int KEEP = TAPS - 1;
@@ -197,6 +255,11 @@ short_conv_run_kernel(const float* __restrict__ x, int ld, int off, const float*
   for (int k = 0; k < TAPS; ++k) {
     const float4 q = __ldg(reinterpret_cast<const float4*>(w + (size_t)c * TAPS) + k);
     wl[4 * k] = q.x; wl[4 * k + 1] = q.y; wl[4 * k + 2] = q.z; wl[4 * k + 3] = q.w;
+  }
+  float bl[4] = {0.f, 0.f, 0.f, 0.f};
+  if (bias != nullptr) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) bl[i] = __ldg(bias + c + i);
   }
   float win[KEEP + 1][4];                               // [older input, oldest first][channel]
   float now[4] = {0.f, 0.f, 0.f, 0.f};
@@ -239,7 +302,7 @@ short_conv_run_kernel(const float* __restrict__ x, int ld, int off, const float*
       float acc = 0.f;
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) acc = fmaf(wl[i * TAPS + k], win[k][i], acc);
-      acc = fmaf(wl[i * TAPS + KEEP], now[i], acc);
+      acc = fmaf(wl[i * TAPS + KEEP], now[i], acc) + bl[i];
       y[i] = MODE == 0 ? sbs_silu(acc) : now[i] + acc;
     }
     if constexpr (sizeof(TO) == 4) {
@@ -320,9 +383,42 @@ SLLM_EXPORT int sllm_qk_norm_rope_kv_write(const float* qkv, int ld, const float
   return launch_status("qk_norm_rope_kv_write");
 }
 
+SLLM_EXPORT int sllm_whole_norm_kv_write(const float* qkv, int parts, size_t part_stride, int ld, const float* bias, const float* q_gain,
+                                         const float* k_gain, float eps, const int* positions, float q_coef, int q_every, int nq, int nkv,
+                                         int dim, int vdim, int D, const int* slot_mapping, int page_size, int num_pages, void* k_cache,
+                                         void* v_cache, void* q_out, int cache_dtype, int T, cudaStream_t stream) {
+  SLLM_REQUIRE(T >= 0 && nq > 0 && nkv > 0 && dim > 0 && vdim > 0 && parts >= 1, "whole_norm: bad sizes T=%d nq=%d nkv=%d dim=%d vdim=%d", T, nq, nkv, dim, vdim);
+  SLLM_REQUIRE(D >= dim && D >= vdim, "whole_norm: the cache's head of %d is smaller than a key of %d or a value of %d", D, dim, vdim);
+  SLLM_REQUIRE(ld >= nq * dim + (slot_mapping != nullptr ? nkv * (dim + vdim) : 0), "whole_norm: the product's %d columns are fewer than q|k|v", ld);
+  SLLM_REQUIRE(q_gain != nullptr && (q_coef == 0.f || (q_every >= 1 && positions != nullptr)), "whole_norm: gain, or the factor's positions, missing");
+  SLLM_REQUIRE(slot_mapping == nullptr || (k_gain && page_size > 0 && num_pages > 0 && k_cache && v_cache), "whole_norm: cache arguments missing");
+  const size_t smem = (size_t)(nq + nkv) * dim * sizeof(float);
+  SLLM_REQUIRE(smem <= 200 * 1024, "whole_norm: %d channels of queries and keys do not fit the shared memory", (nq + nkv) * dim);
+  if (T == 0) return SLLM_OK;
+#define LAUNCH(TC)                                                                                                                         \
+  do {                                                                                                                                     \
+    static size_t allowed = 48 * 1024;                                                                                                     \
+    if (smem > allowed) {                                                                                                                  \
+      if (cudaFuncSetAttribute(whole_norm_kv_write_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {   \
+        cudaGetLastError();                                                                                                                \
+        set_error("whole_norm: the kernel's shared memory could not be raised");                                                           \
+        return SLLM_ERR_LAUNCH;                                                                                                            \
+      }                                                                                                                                    \
+      allowed = smem;                                                                                                                      \
+    }                                                                                                                                      \
+    launch_kernel(whole_norm_kv_write_kernel<TC>, (unsigned)T, 256, smem, stream, qkv, parts, part_stride, ld, bias, q_gain, k_gain, eps,    \
+                  positions, q_coef, q_every, nq, nkv, dim, vdim, D, slot_mapping, page_size, num_pages, (TC*)k_cache, (TC*)v_cache, (TC*)q_out); \
+  } while (0)
+  if (cache_dtype == SLLM_F32) LAUNCH(float);
+  else if (cache_dtype == SLLM_BF16) LAUNCH(__nv_bfloat16);
+  else SLLM_REQUIRE(false, "whole_norm: unknown dtype %d", cache_dtype);
+#undef LAUNCH
+  return launch_status("whole_norm_kv_write");
+}
+
 // mode 0: silu(conv(x)), float32 out; mode 1: x + conv(x) in `out_dtype`.  The state rows are rewritten by a second launch,
 // or, where every request brings one token, by the threads that read them.
-SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w, int taps, float* state, const int* seq_of_token,
+SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w, const float* bias, int taps, float* state, const int* seq_of_token,
                                 const int* q_start, const int* state_slots, void* out, int out_dtype, int mode, int T, int S, int C,
                                 cudaStream_t stream) {
   SLLM_REQUIRE(T >= 0 && S >= 0 && C > 0 && taps >= 1 && off >= 0 && off + C <= ld, "short_conv: bad sizes T=%d C=%d taps=%d", T, C, taps);
@@ -340,7 +436,7 @@ SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w,
   if (vec && !own_state && T >= CONV_RUN * S) {         // portions of eight tokens and more on average
     const dim3 rgrid((unsigned)((T + CONV_RUN - 1) / CONV_RUN), (unsigned)((C / 4 + 127) / 128));
 #define RUNK(MODE_, TAPS_, TO_)                                                                                            \
-  launch_kernel(short_conv_run_kernel<MODE_, TAPS_, TO_, CONV_RUN>, rgrid, 128, 0, stream, x, ld, off, w, (const float*)state, \
+  launch_kernel(short_conv_run_kernel<MODE_, TAPS_, TO_, CONV_RUN>, rgrid, 128, 0, stream, x, ld, off, w, bias, (const float*)state, \
                 seq_of_token, q_start, state_slots, (TO_*)out, C, T)
 #define RUN_TAPS(MODE_, TO_)                          \
   if (taps == 2) RUNK(MODE_, 2, TO_);                 \
@@ -354,7 +450,7 @@ SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w,
   } else if (vec) {
     const dim3 vgrid((unsigned)T, (unsigned)((C / 4 + 127) / 128));
 #define VEC(MODE_, TAPS_, TO_)                                                                                              \
-  launch_kernel(short_conv_vec4_kernel<MODE_, TAPS_, TO_>, vgrid, 128, 0, stream, x, ld, off, w, state, seq_of_token, q_start, \
+  launch_kernel(short_conv_vec4_kernel<MODE_, TAPS_, TO_>, vgrid, 128, 0, stream, x, ld, off, w, bias, state, seq_of_token, q_start, \
                 state_slots, (TO_*)out, C, own_state)
 #define VEC_TAPS(MODE_, TO_)                          \
   if (taps == 2) VEC(MODE_, 2, TO_);                  \
@@ -366,13 +462,13 @@ SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w,
 #undef VEC_TAPS
 #undef VEC
   } else if (mode == 0)
-    launch_kernel(short_conv_kernel<0, float>, grid, 256, 0, stream, x, ld, off, w, taps, (const float*)state, seq_of_token, q_start,
+    launch_kernel(short_conv_kernel<0, float>, grid, 256, 0, stream, x, ld, off, w, bias, taps, (const float*)state, seq_of_token, q_start,
                   state_slots, (float*)out, C, own_state);
   else if (out_dtype == SLLM_F32)
-    launch_kernel(short_conv_kernel<1, float>, grid, 256, 0, stream, x, ld, off, w, taps, (const float*)state, seq_of_token, q_start,
+    launch_kernel(short_conv_kernel<1, float>, grid, 256, 0, stream, x, ld, off, w, bias, taps, (const float*)state, seq_of_token, q_start,
                   state_slots, (float*)out, C, own_state);
   else
-    launch_kernel(short_conv_kernel<1, __nv_bfloat16>, grid, 256, 0, stream, x, ld, off, w, taps, (const float*)state, seq_of_token,
+    launch_kernel(short_conv_kernel<1, __nv_bfloat16>, grid, 256, 0, stream, x, ld, off, w, bias, taps, (const float*)state, seq_of_token,
                   q_start, state_slots, (__nv_bfloat16*)out, C, own_state);
   int rc = launch_status("short_conv");
   if (rc != SLLM_OK || taps == 1 || S == 0 || own_state) return rc;
@@ -380,10 +476,10 @@ SLLM_EXPORT int sllm_short_conv(const float* x, int ld, int off, const float* w,
   return launch_status("short_conv_state");
 }
 
-SLLM_EXPORT int sllm_short_conv_silu(const float* x, int ld, int off, const float* w, int taps, float* state,
+SLLM_EXPORT int sllm_short_conv_silu(const float* x, int ld, int off, const float* w, const float* bias, int taps, float* state,
                                      const int* seq_of_token, const int* q_start, const int* state_slots, float* out, int T,
                                      int S, int C, cudaStream_t stream) {
-  return sllm_short_conv(x, ld, off, w, taps, state, seq_of_token, q_start, state_slots, out, SLLM_F32, 0, T, S, C, stream);
+  return sllm_short_conv(x, ld, off, w, bias, taps, state, seq_of_token, q_start, state_slots, out, SLLM_F32, 0, T, S, C, stream);
 }
 
 SLLM_EXPORT int sllm_norm_mean_add(float* stream_, const float* a, const float* ga, const float* b, const float* gb, float eps,

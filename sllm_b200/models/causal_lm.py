@@ -12,11 +12,13 @@ from ..config.plan import ModelPlan
 from ..parts import delta_rule as _delta_rule, experts as _experts, latent_attention as _latent  # noqa: F401
 from ..parts import linear_attention as _linear_attention, parallel as _parallel, side_by_side as _side_by_side  # noqa: F401
 from ..parts import gated_recurrence as _gated_recurrence, output_norm as _output_norm, sandwich as _sandwich  # noqa: F401
+from ..parts import hyper_connections as _hyper_connections, state_space as _state_space  # noqa: F401
 from ..parts import standard as _standard  # noqa: F401  (each import registers its parts)
 from ..parts.base import (BLOCKS, COMPLETE, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, SHIFTS,
                           LayerCache, SlotState, StepContext, TensorSpec, flatten_needs, join_name)
 
 
+PREVIOUS_TOKEN = "previous_token"        # the model's own per-request state (see `CausalLM.cache_needs`)
 FAMILIES = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "norm": NORMS, "shift": SHIFTS}
 
 
@@ -55,6 +57,8 @@ class CausalLM:
         self.embedding_norm = NORMS.build(plan.embedding_norm, **kw) if plan.embedding_norm is not None else None
         self.pass_vectors = None   # [passes, H] float32
         self.token_table = None    # [V, width] compute dtype: vectors that belong to a token
+        self.pair_table = None     # [buckets + 1, H] compute dtype: rows by pairs of tokens
+        self.stream_sum = torch.ones(plan.streams, dtype=torch.float32, device=self.device) if plan.streams is not None else None
         self.position = POSITIONS.build(plan.position, **kw) if plan.position is not None else None
         self.embedding = None      # [V, H] compute dtype
         self.head = None           # [V, H] compute dtype (the embedding itself when tied)
@@ -82,6 +86,8 @@ class CausalLM:
             specs.append(TensorSpec(p.pass_vectors_name, (p.passes, p.hidden_size), role="bias"))
         if p.token_table_name is not None:
             specs.append(TensorSpec(p.token_table_name, (p.vocab_size, p.token_table_width), role="embedding"))
+        if p.token_pairs is not None:
+            specs.append(TensorSpec(p.token_pairs.name, (p.token_pairs.buckets + 1, p.hidden_size), role="embedding"))
         return specs
 
     def ignored_tensor_names(self):
@@ -100,6 +106,8 @@ class CausalLM:
             for _, part in self._named_parts():
                 if hasattr(part, "adopt_token_table"):
                     part.adopt_token_table(self.token_table)
+        if p.token_pairs is not None:
+            self.pair_table = fetch(p.token_pairs.name).to(device=self.device, dtype=self.dtype).contiguous()
         if p.head_name is None:
             self.head = self.embedding
         else:
@@ -125,7 +133,8 @@ class CausalLM:
     # ---- cache needs ----------------------------------------------------------------
     def cache_needs(self):
         """One entry per run of the run list: the mixer's need, or the index of
-        the run whose cache it borrows."""
+        the run whose cache it borrows.  What the model itself keeps per request (the token before, where the
+        embedding takes in pairs) rides with the first run."""
         out = []
         for e in self.plan.run_list:
             if e.cache_from is not None:
@@ -134,13 +143,20 @@ class CausalLM:
                 out.append(("borrow", e.cache_from, own) if own else ("borrow", e.cache_from))
             else:
                 out.append(("own", self.layers[e.layer].cache_need()))
+        if self.plan.token_pairs is not None:
+            out[0] = ("own", tuple(flatten_needs(out[0][1])) + (SlotState((1,), PREVIOUS_TOKEN),))
         return out
 
     # ---- forward ------------------------------------------------------------------
     def forward(self, step: StepContext, caches: list[LayerCache]) -> torch.Tensor:
         """Run the batch's tokens through every entry of the run list and return
         float32 logits ``[R, V]`` at ``step.logit_rows``."""
-        residual = ops.embed_gather(self.embedding, step.token_ids, self.plan.embedding_scale)       # [T, H] float32
+        p = self.plan
+        if p.token_pairs is None and p.streams is None:
+            residual = ops.embed_gather(self.embedding, step.token_ids, p.embedding_scale)           # [T, H] float32
+        else:
+            before = caches[0].states[PREVIOUS_TOKEN] if p.token_pairs is not None else None
+            residual = ops.embed_streams(self.embedding, step, p.embedding_scale, p.streams, self.pair_table, before, p.token_pairs)
         if self.position is not None:
             self.position.on_embedding(residual, step)
         entered = None
@@ -160,6 +176,11 @@ class CausalLM:
                 # the norm that reads the stream next: this block's last product may prepare its input
                 kw["next_norm"] = getattr(self.layers[runs[i + 1].layer].block, "first_norm", None)
             delta = block.forward(residual, delta, step, caches[i], self.position, write_cache=e.cache_from is None, **kw)
+        if p.streams is not None:
+            if step.logit_rows.numel() == 0:
+                return torch.empty((0, p.vocab_size), dtype=torch.float32, device=self.device)
+            x = _hyper_connections.read_streams(residual, delta, step.logit_rows, self.stream_sum, self.final_norm, self.dtype)
+            return self._logits(x)
         if isinstance(delta, COMPLETE):          # (a block handed one on although nothing asked: take the stream as it is)
             delta = None
         if step.logit_rows.numel() == 0:
@@ -167,5 +188,8 @@ class CausalLM:
         res_rows = ops.gather_rows(residual, step.logit_rows)
         delta_rows = ops.gather_rows(delta, step.logit_rows) if delta is not None else None
         x = self.final_norm.add_norm(res_rows, delta_rows)
+        return self._logits(x)
+
+    def _logits(self, x: torch.Tensor) -> torch.Tensor:
         logits = ops.linear(x, self.head, None, torch.float32)
         return ops.softcap_(logits, self.plan.logit_softcap) if self.plan.logit_softcap is not None else logits

@@ -70,6 +70,45 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0) -> 
     return out
 
 
+# ---- a stream of several copies ------------------------------------------------------------------------
+
+MAX_STREAMS = 16
+
+
+def embed_streams(table, step, scale: float, copies, pair_table=None, before=None, pairs=None) -> torch.Tensor:
+    """float32 ``[T, copies, H]`` (``[T, H]`` where ``copies`` is None), every copy the row of ``table`` at the step's token ids times
+    ``scale``; with ``pairs`` (`config.plan.TokenPairs`) plus the row of ``pair_table`` ``[buckets + 1, H]`` that the token and the
+    one before it name (the last row at position 0).  The token before a portion's first is the request's row of ``before`` (float32
+    ``[slots, 1]``), which then receives the portion's last token."""
+    _chk(table, pair_table, before, step.token_ids)
+    T, (V, H) = step.token_ids.numel(), table.shape
+    if pairs is not None and (pair_table is None or tuple(pair_table.shape) != (pairs.buckets + 1, H) or pair_table.dtype != table.dtype or
+                              before is None or before.dtype != torch.float32):
+        raise KernelError("embed_streams: pairs of tokens need their table [buckets + 1, H] and the tokens before, float32 [slots, 1]")
+    out = torch.empty((T, H) if copies is None else (T, int(copies), H), dtype=torch.float32, device=table.device)
+    call("sllm_embed_streams", _p(table), _dt(table), _p(step.token_ids), _p(out), T, H, V, float(scale), int(copies or 1), _p(pair_table),
+         *((int(pairs.buckets), int(pairs.mul_prev), int(pairs.mul_cur)) if pairs is not None else (0, 0, 0)), _p(step.positions),
+         _p(step.seq_of_token), _p(step.q_start), _p(step.state_slots), _p(before), _stream())
+    return out
+
+
+def streams_step(streams, term, mix, share, into, gain, eps: float, out_dtype, rows=None):
+    """One sublayer's border in a stream of several copies ``[T, s, W]`` (float32): with ``term`` (float32 ``[T, W]`` or a stack of
+    partial sums), every new stream r = sum over the old s of ``mix[s, r]`` times stream s, plus ``share[r]`` times the term, in place;
+    then the RMS norm (``gain`` float32 ``[W]``) of sum over s of ``into[s]`` times stream s, in ``out_dtype`` (``gain`` None: no
+    norm, nothing returned).  ``rows`` (int32): only these rows are computed, ``[len(rows), W]``, and no stream is written."""
+    _chk(streams, term, mix, share, into, gain, rows)
+    T, s, W = streams.shape
+    if streams.dtype != torch.float32 or (term is not None and (tuple(term.shape[-2:]) != (T, W) or tuple(mix.shape) != (s, s) or share.numel() != s)) or \
+            (gain is not None and (gain.numel() != W or into.numel() != s)):
+        raise KernelError("streams_step: float32 streams [T, s, W], a term that fits them, s x s and s weights")
+    R = T if rows is None else rows.numel()
+    h = torch.empty((R, W), dtype=out_dtype, device=streams.device) if gain is not None else None
+    call("sllm_streams_step", _p(streams), *_term(term), _p(mix), _p(share), _p(into), _p(gain), float(eps), _p(rows), _p(h),
+         _dtc(out_dtype) if h is not None else F32, R, T, s, W, _stream())
+    return h
+
+
 # ---- a stream with sinusoidal positions, a norm in groups, a token shift ----------------------------
 
 def add_sinusoid_(stream: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
@@ -333,6 +372,38 @@ def qk_norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, positions, table, rot
     return q
 
 
+def whole_norm_kv_write(qkv, bias, q_gain, k_gain, eps: float, positions, q_temp, nq: int, nkv: int, dim: int, vdim: int, slot_mapping,
+                        k_cache, v_cache, out_dtype) -> torch.Tensor:
+    """From a float32 product ``[T, nq*dim (+ nkv*(dim + vdim))]`` (or a stack of partial sums) plus ``bias``: all query rows over
+    their common root mean square times ``q_gain`` ``[nq*dim]``, times 1 + coef ln(floor((p + 1) / every) + 1) with ``q_temp`` =
+    (coef, every) (None: 1); the key rows likewise with ``k_gain`` ``[nkv*dim]``; values as they are.  The queries come back ``[T,
+    nq*D]`` in ``out_dtype`` with D the cache's head size (zeros beyond dim); keys and values go to ``slot_mapping`` in the pages (None: the
+    product holds queries alone)."""
+    _chk(qkv, bias, q_gain, k_gain, positions, slot_mapping, k_cache, v_cache)
+    T, ld = qkv.shape[-2:]
+    num_pages, nkv_c, page_size, D = k_cache.shape
+    want = nq * dim + (nkv * (dim + vdim) if slot_mapping is not None else 0)
+    if nkv_c != nkv or k_cache.dtype != out_dtype or tuple(v_cache.shape) != tuple(k_cache.shape) or ld < want or \
+            (bias is not None and bias.numel() != ld) or q_gain.numel() != nq * dim or (slot_mapping is not None and k_gain.numel() != nkv * dim):
+        raise KernelError(f"whole_norm_kv_write: a product of {want} columns, gains of the projections' sizes and a cache of the compute dtype")
+    q = torch.empty((T, nq * D), dtype=out_dtype, device=qkv.device)
+    coef, every = q_temp if q_temp is not None else (0.0, 1)
+    call("sllm_whole_norm_kv_write", *_term(qkv), ld, _p(bias), _p(q_gain), _p(k_gain), float(eps), _p(positions), float(coef), int(every), nq, nkv,
+         dim, vdim, D, _p(slot_mapping), page_size, num_pages, _p(k_cache), _p(v_cache), _p(q), _dtc(out_dtype), T, _stream())
+    return q
+
+
+def norm_cols(x, off: int, n: int, gain, eps: float, out_dtype) -> torch.Tensor:
+    """Columns ``off .. off+n`` of a float32 product over their root mean square, times ``gain``, in ``out_dtype``."""
+    _chk(x, gain)
+    T, ld = x.shape
+    if x.dtype != torch.float32 or gain.dtype != torch.float32 or gain.numel() != n:
+        raise KernelError("norm_cols: a float32 product and a float32 gain of as many values as columns")
+    out = torch.empty((T, n), dtype=out_dtype, device=x.device)
+    call("sllm_norm_cols", _p(x), ld, int(off), int(n), _p(gain), float(eps), _p(out), _dtc(out_dtype), T, _stream())
+    return out
+
+
 def short_conv_add(x, weight, state, step, out_dtype) -> torch.Tensor:
     """``x + conv(x)``: the float32 rows ``x [T, C]`` plus their causal convolution over time per channel (``weight`` float32
     ``[C, taps]``, the current token's tap last; the inputs before a request's portion from its row of ``state`` ``[slots, C,
@@ -344,25 +415,26 @@ def short_conv_add(x, weight, state, step, out_dtype) -> torch.Tensor:
             (taps > 1 and tuple(state.shape[1:]) != (C, taps - 1)):
         raise KernelError("short_conv_add: float32 input and taps [C, taps], and a state [slots, C, taps-1]")
     out = torch.empty((T, C), dtype=out_dtype, device=x.device)
-    call("sllm_short_conv", _p(x), C, 0, _p(weight), taps, _p(state) if taps > 1 else None, _p(step.seq_of_token), _p(step.q_start),
+    call("sllm_short_conv", _p(x), C, 0, _p(weight), None, taps, _p(state) if taps > 1 else None, _p(step.seq_of_token), _p(step.q_start),
          _p(step.state_slots), _p(out), _dtc(out_dtype), 1, T, step.num_seqs, C, _stream())
     if taps > 1:
         launches["own"] += 1          # the state's kernel
     return out
 
 
-def short_conv_silu(x, off: int, weight, state, step) -> torch.Tensor:
-    """``silu`` of a causal convolution over time, per channel, of columns ``off .. off+C`` of the float32 product ``x``:
+def short_conv_silu(x, off: int, weight, state, step, bias=None) -> torch.Tensor:
+    """``silu`` of a causal convolution over time (plus ``bias`` float32 ``[C]``), per channel, of columns ``off .. off+C`` of the float32 product ``x``:
     ``weight`` float32 ``[C, taps]`` with the current token's tap last; the ``taps - 1`` inputs before a request's portion
     come from its row of ``state`` (float32 ``[slots, C, taps-1]``, zeros at a sequence's start), which then receives the
     portion's last ones.  float32 ``[T, C]``."""
-    _chk(x, weight, state)
+    _chk(x, weight, state, bias)
     T, ld = x.shape
     C, taps = weight.shape
-    if x.dtype != torch.float32 or weight.dtype != torch.float32 or (taps > 1 and tuple(state.shape[1:]) != (C, taps - 1)):
-        raise KernelError("short_conv_silu: float32 input and taps, and a state [slots, C, taps-1]")
+    if x.dtype != torch.float32 or weight.dtype != torch.float32 or (taps > 1 and tuple(state.shape[1:]) != (C, taps - 1)) or \
+            (bias is not None and (bias.dtype != torch.float32 or bias.numel() != C)):
+        raise KernelError("short_conv_silu: float32 input, taps and bias, and a state [slots, C, taps-1]")
     out = torch.empty((T, C), dtype=torch.float32, device=x.device)
-    call("sllm_short_conv_silu", _p(x), ld, int(off), _p(weight), taps, _p(state) if taps > 1 else None, _p(step.seq_of_token),
+    call("sllm_short_conv_silu", _p(x), ld, int(off), _p(weight), _p(bias), taps, _p(state) if taps > 1 else None, _p(step.seq_of_token),
          _p(step.q_start), _p(step.state_slots), _p(out), T, step.num_seqs, C, _stream())
     if taps > 1:
         launches["own"] += 1          # the state's kernel
@@ -408,34 +480,38 @@ def moe_act(up, dense, ff: int, out_dtype) -> torch.Tensor:
     return out
 
 
-def moe_route_top_softmax(logits, top: int, scale: float = 1.0):
+def moe_route_top_softmax(logits, top: int, scale: float = 1.0, experts: "int | None" = None, gated: int = 0):
     """The ``top`` largest of the float32 router logits ``[T, E]`` win (the lower index on a tie); their weights are the
     softmax over the winners alone, times ``scale``.  (dense weights float32 ``[T, E]`` with zeros elsewhere, indices int32 ``[T, top]`` by
-    falling logit, weights float32 ``[T, top]``)."""
+    falling logit, weights float32 ``[T, top]``).  ``experts``: only so many of the logits' columns are experts; ``gated`` (0 or 1):
+    the column behind them is the logit of an expert every token uses, and the dense weights ``[T, E + gated]`` end with its sigmoid."""
     _chk(logits)
-    T, E = logits.shape
+    T, ld = logits.shape
+    E = int(experts or ld)
+    if gated not in (0, 1) or E + gated > ld:
+        raise KernelError(f"moe_route_top_softmax: {E} experts and {gated} gate columns in rows of {ld} logits")
     if logits.dtype != torch.float32:
         raise KernelError("moe_route_top_softmax: the router's logits are float32")
-    dense = torch.empty((T, E), dtype=torch.float32, device=logits.device)
+    dense = torch.empty((T, E + gated), dtype=torch.float32, device=logits.device)
     idx = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     wts = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    call("sllm_moe_route_top_softmax", _p(logits), T, E, int(top), float(scale), _p(dense), _p(idx), _p(wts), _stream())
+    call("sllm_moe_route_top_softmax", _p(logits), ld, T, E, int(gated), int(top), float(scale), _p(dense), _p(idx), _p(wts), _stream())
     return dense, idx, wts
 
 
 def gated_clamp_act(gu, interleave: int, limit: float, out_dtype, *, alpha: float = 1.702, dense=None, ff: int | None = None,
-                    act: str = "clamped_swish"):
+                    act: str = "clamped_swish", tail: int = 0):
     """``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)`` and ``u' = clamp(u, -limit, limit)`` of ``gu [T, 2N]``
     whose columns alternate between gate and up in blocks of ``interleave``.  With ``dense`` (float32 ``[T, E]``, the
     routing weights of E experts of ``ff`` columns each, N = E ff): also times the token's weight of the column's expert;
     the columns of an expert a token does not use are not read.  ``act`` ``silu``: ``g sigmoid(g) u`` instead (``limit`` and
-    ``alpha`` unused)."""
+    ``alpha`` unused).  ``tail``: so many columns behind the experts' belong to one more expert, with the last of the weights."""
     _chk(gu, dense)
     T, two_n = gu.shape
     N = two_n // 2
     E = dense.shape[1] if dense is not None else 0
     out = torch.empty((T, N), dtype=out_dtype, device=gu.device)
-    call("sllm_gated_clamp_act", _p(gu), _dt(gu), _p(dense), _p(out), _dtc(out_dtype), T, N, E, int(ff if dense is not None else N),
+    call("sllm_gated_clamp_act", _p(gu), _dt(gu), _p(dense), _p(out), _dtc(out_dtype), T, N, E, int(ff if dense is not None else N), int(tail),
          int(interleave), float(limit), float(alpha), {"clamped_swish": 0, "silu": 1}[act], _stream())
     return out
 
@@ -566,7 +642,7 @@ def retention_chunked_supports(dk: int, dv: int) -> bool:
     return bool(lib().sllm_retention_chunked_supports(int(dk), int(dv)))
 
 
-def retention_chunks(q_lens, ctx_lens, min_len: int, device):
+def portion_chunks(q_lens, ctx_lens, min_len: int, device):
     """The step's long portions cut into chunks of `RETENTION_CHUNK` tokens: (first tokens, their positions, lengths, chunks; requests,
     their first chunk, how many, requests) on the device, or None where no portion has ``min_len`` tokens."""
     t0, pos, n, seq, first, count = [], [], [], [], [], []
@@ -592,7 +668,7 @@ def retention_chunks(q_lens, ctx_lens, min_len: int, device):
 def retention_chunked(proj, offs, off_g: int, decay, table, rotary_dim: int, k_scale: float, eps: float, state, step, chunks, heads: int,
                       dk: int, dv: int, out) -> None:
     """Retention, the heads' norm and the silu gate (columns ``off_g`` of ``proj``) for the requests that ``chunks`` (see
-    `retention_chunks`) cuts, a chunk of tokens at a time; their rows of ``out`` ``[T, heads*dv]`` and their states are written, others
+    `portion_chunks`) cuts, a chunk of tokens at a time; their rows of ``out`` ``[T, heads*dv]`` and their states are written, others
     left alone."""
     _chk(proj, decay, table, state, out)
     if proj.dtype != torch.float32 or decay.dtype != torch.float32 or state.dtype != torch.float32:
@@ -620,7 +696,7 @@ def retention_gated(proj, offs, off_g: int, decay, table, rotary_dim: int, k_sca
     chunks, longest = None, 0
     if RETENTION_CHUNKED_FROM > 0 and step.max_q_len >= RETENTION_CHUNKED_FROM and step.q_lens and retention_chunked_supports(dk, dv):
         if "retention" not in step.attn_tiles:
-            step.attn_tiles["retention"] = retention_chunks(step.q_lens, step.ctx_lens, RETENTION_CHUNKED_FROM, proj.device)
+            step.attn_tiles["retention"] = portion_chunks(step.q_lens, step.ctx_lens, RETENTION_CHUNKED_FROM, proj.device)
         chunks, longest = step.attn_tiles["retention"], RETENTION_CHUNKED_FROM - 1
     if chunks is None:
         o = retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv)
@@ -630,6 +706,82 @@ def retention_gated(proj, offs, off_g: int, decay, table, rotary_dim: int, k_sca
     if chunks[7] < step.num_seqs:
         o = retention(proj, offs, decay, table, rotary_dim, k_scale, state, step, heads, dk, dv, max_len=longest)
         delta_out(o, None, proj, off_g, eps, heads, dv, out_dtype, "silu", out=out, step=step, max_len=longest)
+    return out
+
+
+# ---- a state-space recurrence: one decay per token and head ------------------------------------------------
+
+# Portions of at least so many tokens run in chunks (0: none does); below, token by token.
+STATE_SPACE_CHUNKED_FROM = int(os.environ.get("SLLM_STATE_SPACE_CHUNKED_FROM", "96"))
+
+
+@functools.lru_cache(maxsize=4096)
+def state_space_chunked_supports(n: int, dv: int) -> bool:
+    return bool(lib().sllm_state_space_chunked_supports(int(n), int(dv)))
+
+
+def _state_space_args(xbc, proj, off_dt, dt_bias, a_log, skip, state, heads, groups, n, dv, what):
+    _chk(xbc, proj, dt_bias, a_log, skip, state)
+    if any(t.dtype != torch.float32 for t in (xbc, proj, dt_bias, a_log, skip, state)):
+        raise KernelError(f"{what}: everything that enters the recurrence is float32")
+    if tuple(state.shape[1:]) != (heads, n, dv) or xbc.shape[1] != heads * dv + 2 * groups * n or heads % groups or off_dt + heads > proj.shape[1]:
+        raise KernelError(f"{what}: state {tuple(state.shape)} or inputs {tuple(xbc.shape)} do not fit {heads} heads of {n}x{dv} in {groups} groups")
+
+
+def state_space_walk(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, heads: int, groups: int, n: int, dv: int, max_len: int = 0, out=None):
+    """`state_space` token by token.  ``max_len`` > 0: requests that bring more tokens are left alone (neither their states nor
+    their rows of ``out`` are touched)."""
+    _state_space_args(xbc, proj, off_dt, dt_bias, a_log, skip, state, heads, groups, n, dv, "state_space")
+    if out is None:
+        out = torch.empty((xbc.shape[0], heads * dv), dtype=torch.float32, device=xbc.device)
+    call("sllm_state_space", _p(xbc), xbc.shape[1], _p(proj), proj.shape[1], int(off_dt), _p(dt_bias), _p(a_log), _p(skip), _p(state),
+         _p(step.q_start), _p(step.state_slots), _p(out), step.num_seqs, heads, groups, n, dv, int(step.max_q_len), int(max_len), _stream())
+    return out
+
+
+def state_space_chunked(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, chunks, heads: int, groups: int, n: int, dv: int, out) -> None:
+    """`state_space` for the requests that ``chunks`` (see `portion_chunks`) cuts, a chunk of tokens at a time; their rows of ``out`` and
+    their states are written, others left alone."""
+    _state_space_args(xbc, proj, off_dt, dt_bias, a_log, skip, state, heads, groups, n, dv, "state_space_chunked")
+    t0, _, count, C, seq, first, runs, R = chunks
+    scratch = torch.empty((C, heads, n, dv), dtype=torch.float32, device=xbc.device)
+    keeps = torch.empty((C, heads), dtype=torch.float32, device=xbc.device)
+    call("sllm_state_space_chunked", _p(xbc), xbc.shape[1], _p(proj), proj.shape[1], int(off_dt), _p(dt_bias), _p(a_log), _p(skip), _p(state),
+         _p(step.state_slots), _p(t0), _p(count), C, _p(seq), _p(first), _p(runs), R, _p(scratch), _p(keeps), _p(out), heads, groups, n, dv, _stream())
+    launches["own"] += 2           # the three kernels of the entry point
+
+
+def state_space(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, heads: int, groups: int, n: int, dv: int) -> torch.Tensor:
+    """The state-space recurrence over the step's tokens, request by request in token order, from and into the requests' rows of
+    ``state`` (float32 ``[slots, heads, n, dv]``): S <- exp(-exp(a_log_h) dt) S + dt B x^T; y = S^T C + skip_h x, with dt = softplus of
+    column ``off_dt + h`` of the float32 product ``proj`` plus ``dt_bias[h]``.  ``xbc`` float32 ``[T, heads*dv + 2*groups*n]`` holds x (head
+    by head), B and C (group by group; head h uses group h // (heads / groups)).  Returns y float32 ``[T, heads*dv]``.  Long prompt
+    portions run in chunks (states of up to 128 x 128), single tokens and short portions token by token; a step may hold both."""
+    chunks, longest = None, 0
+    if STATE_SPACE_CHUNKED_FROM > 0 and step.max_q_len >= STATE_SPACE_CHUNKED_FROM and step.q_lens and state_space_chunked_supports(n, dv):
+        key = ("chunks", STATE_SPACE_CHUNKED_FROM)
+        if key not in step.attn_tiles:
+            step.attn_tiles[key] = portion_chunks(step.q_lens, step.ctx_lens, STATE_SPACE_CHUNKED_FROM, xbc.device)
+        chunks, longest = step.attn_tiles[key], STATE_SPACE_CHUNKED_FROM - 1
+    args = (xbc, proj, off_dt, dt_bias, a_log, skip, state, step)
+    if chunks is None:
+        return state_space_walk(*args, heads, groups, n, dv)
+    out = torch.empty((xbc.shape[0], heads * dv), dtype=torch.float32, device=xbc.device)
+    state_space_chunked(*args, chunks, heads, groups, n, dv, out)
+    if chunks[7] < step.num_seqs:
+        state_space_walk(*args, heads, groups, n, dv, max_len=longest, out=out)
+    return out
+
+
+def gated_group_norm(y, gate, off_g: int, gain, eps: float, groups: int, out_dtype) -> torch.Tensor:
+    """``v = y * silu(gate[:, off_g ..])``, its channels in ``groups`` equal parts each over its own root mean square, times ``gain``, in
+    ``out_dtype``; ``y`` float32 ``[T, n]``, ``gate`` a float32 product."""
+    _chk(y, gate, gain)
+    T, n = y.shape
+    if y.dtype != torch.float32 or gate.dtype != torch.float32 or gain.numel() != n or n % groups or off_g + n > gate.shape[1]:
+        raise KernelError("gated_group_norm: float32 rows, gates and a gain of their width, in equal parts")
+    out = torch.empty((T, n), dtype=out_dtype, device=y.device)
+    call("sllm_gated_group_norm", _p(y), _p(gate), gate.shape[1], int(off_g), _p(gain), float(eps), int(groups), _p(out), _dtc(out_dtype), T, n, _stream())
     return out
 
 
@@ -738,7 +890,7 @@ def stream_supports(M: int, N: int, K: int) -> bool:
     return not linear_tc_supports(M, N, K)
 
 
-PLAIN_ACTS = {None: 0, "relu2": 1, "token": 2}      # SLLM_ACT_* of the kernels: activations of a plain (ungated) result
+PLAIN_ACTS = {None: 0, "relu2": 1, "token": 2, "gelu": 3}      # SLLM_ACT_* of the kernels: activations of a plain (ungated) result
 
 
 class TokenColumns:
@@ -959,15 +1111,15 @@ def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | 
     ``splits`` > 1 (float32 result, no other epilogue): K in that many slices, the result a stack ``[splits', M, N]``
     of partial sums (bias in the first) for the consumer to add.  ``act="gelu_tanh"``: the gated epilogue
     ``gelu_tanh(gate + bias) * (up + bias)`` in place of ``silu``'s (rows and bias interleaved in blocks of 8); ``"relu2"``:
-    bfloat16 ``max(v, 0)^2`` of the plain result; ``"token"``: bfloat16 ``gelu_tanh(v)`` times ``token``'s columns."""
+    bfloat16 ``max(v, 0)^2`` of the plain result; ``"gelu"``: its exact gelu; ``"token"``: bfloat16 ``gelu_tanh(v)`` times ``token``'s columns."""
     _chk(x, w, bias, residual, next_gain)
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_pair: bfloat16 operands only")
-    if act not in (None, "gelu_tanh", "relu2", "token") or (act and silu):
+    if act not in (None, "gelu_tanh", "relu2", "token", "gelu") or (act and silu):
         raise KernelError(f"gemm_pair: epilogue {act!r}")
-    plain_act = act if act in ("relu2", "token") else None
+    plain_act = act if act in ("relu2", "token", "gelu") else None
     gelu, silu = act == "gelu_tanh", silu or act == "gelu_tanh"
-    if plain_act and (residual is not None or bias is not None or out_dtype != torch.bfloat16 or (token is None) != (act == "relu2")):
+    if plain_act and (residual is not None or bias is not None or out_dtype != torch.bfloat16 or (token is not None) != (act == "token")):
         raise KernelError(f"gemm_pair: the {act} epilogue takes neither bias nor residual and gives bfloat16")
     M, K = x.shape
     N = w.shape[0]
@@ -999,7 +1151,7 @@ def gemm_pair(x, w, bias, out_dtype, *, silu: bool = False, wide: "bool | str | 
         real = int(lib().sllm_gemm_pair_splits(K, int(splits))) if splits > 1 else 1
         epi, out = 0, torch.empty((real, M, N) if real > 1 else (M, N), dtype=torch.float32, device=x.device)
     else:
-        epi, out = {None: 1, "relu2": 5, "token": 6}[plain_act], torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        epi, out = {None: 1, "relu2": 5, "token": 6, "gelu": 7}[plain_act], torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     if splits > 1 and (epi != 0 or scale is not None):
         raise KernelError("gemm_pair: slices of K leave float32 partial sums: no other epilogue, no owed norm")
     call("sllm_gemm_pair", _p(x), _p(w), _p(bias), _p(out), M, N, K, epi, code, int(splits),
@@ -1072,9 +1224,10 @@ def linear_tc(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False, act
     """The weight-streaming product on the tcgen05 tensor cores for up to 128 tokens.  With
     ``splits`` > 1 the result is a float32 stack ``[splits', M, N]`` of partial sums (bias in the
     first) that the consumer adds; with ``silu`` the matrix is gate|up interleaved in blocks of 8
-    and the bfloat16 result is ``silu(gate) * up`` of width N/2; with ``act="relu2"`` the bfloat16 result is ``max(v, 0)^2``."""
+    and the bfloat16 result is ``silu(gate) * up`` of width N/2; with ``act="relu2"`` the bfloat16 result is ``max(v, 0)^2``, with
+    ``"gelu"`` the exact gelu."""
     _chk(x, w, bias)
-    if act not in (None, "relu2") or (act and (silu or out_dtype != torch.bfloat16)):
+    if act not in (None, "relu2", "gelu") or (act and (silu or out_dtype != torch.bfloat16)):
         raise KernelError(f"linear_tc: epilogue {act!r}")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("linear_tc: bfloat16 operands only")
@@ -1090,7 +1243,7 @@ def linear_tc(x, w, bias, out_dtype, *, splits: int = 1, silu: bool = False, act
         epi = 0
         out = torch.empty((real, M, N) if real > 1 else (M, N), dtype=torch.float32, device=x.device)
     else:
-        epi, out = 3 if act else 1, torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        epi, out = {None: 1, "relu2": 3, "gelu": 4}[act], torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     call("sllm_linear_tc", _p(x), _p(w), _p(bias), _p(out), M, N, K, real, epi, _p(_status_word(x.device)), _stream())
     _tc_used["since_check"] += 1
     return out
@@ -1156,7 +1309,7 @@ def linear_ws(x, w, bias, out_dtype, residual=None, scale: RowScale | None = Non
     or, given ``residual`` (float32 ``[M, N]``), added into it in place (returns None).  ``scale``: a norm
     still owed on ``x`` (`RowScale`).  ``next_gain`` (with ``residual``): the gain of the norm that follows; the
     kernel then also writes that norm's input in the owed form and ``(xg, RowScale)`` is returned (the scale's
-    eps is left at 0 for the caller to set).  ``act`` (without ``residual``): ``"relu2"``, the result's ``max(v, 0)^2``, or
+    eps is left at 0 for the caller to set).  ``act`` (without ``residual``): ``"relu2"``, the result's ``max(v, 0)^2``, ``"gelu"``, its exact gelu, or
     ``"token"``, ``gelu_tanh(v)`` times ``token``'s columns."""
     _chk(x, w, bias, residual, next_gain)
     M, K = x.shape
@@ -1295,7 +1448,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias, out_dtype: torch.dtype, allow
 
 
 def plain_act(x, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
-    """``act`` of ``x [T, N]`` (or of the sum of a stack of partial sums ``[parts, T, N]``) in ``out_dtype``: ``relu2`` is ``max(x, 0)^2``, ``token`` is ``gelu_tanh(x)`` times ``token``'s columns
+    """``act`` of ``x [T, N]`` (or of the sum of a stack of partial sums ``[parts, T, N]``) in ``out_dtype``: ``relu2`` is ``max(x, 0)^2``, ``gelu`` the exact (erf) gelu, ``token`` is ``gelu_tanh(x)`` times ``token``'s columns
     (a table of ``out_dtype``)."""
     _chk(x)
     T, N = x.shape[-2:]
@@ -1313,7 +1466,7 @@ _PLAIN_ACT_FUSED = os.environ.get("SLLM_PLAIN_ACT_FUSED", "1") != "0"      # 0: 
 
 def linear_plain_act(x, w, out_dtype, act: str, token: "TokenColumns | None" = None) -> torch.Tensor:
     """``act(x @ w.T)`` in ``out_dtype`` (see `plain_act`).  bfloat16: the activation leaves with the product's tile (the warp-split
-    streaming product up to 16 tokens, the CTA-pair product of prompt portions; ``relu2`` of large matrices also on tensor memory).
+    streaming product up to 16 tokens, the CTA-pair product of prompt portions; ``relu2`` and ``gelu`` of large matrices also on tensor memory).
     Otherwise the product in float32, cut along K where that is faster, then the activation kernel, which adds the slices.
     (In a graph, us: 8,448 x 2,048 and 8 tokens 8.3 in the warp-split form, 8.7 in four slices and a kernel, 17.5 in the streaming
     form unsliced; 16,512 x 4,096 and 8 tokens 29.3 / 26.6 / 36.8, on tensor memory 28.0; 32 tokens of the former 13.0 / 11.5 / 20.6,
@@ -1325,7 +1478,7 @@ def linear_plain_act(x, w, out_dtype, act: str, token: "TokenColumns | None" = N
         large = N * K >= LINEAR_TC_LARGE
         if ws_supports(M, N, K) or (M <= 16 and not large and ws_takes(M, N, K)):
             return linear_ws(x, w, None, out_dtype, act=act, token=token)
-        if act == "relu2" and large and M >= LINEAR_TC_WIDE_FROM_ROWS and linear_tc_takes(M, N, K):
+        if act in ("relu2", "gelu") and large and M >= LINEAR_TC_WIDE_FROM_ROWS and linear_tc_takes(M, N, K):
             return linear_tc(x, w, None, out_dtype, act=act)
         if _pair_rows(M) and pair_supports(M, N, K):
             return gemm_pair(x, w, None, out_dtype, act=act, token=token)
@@ -1466,8 +1619,34 @@ def _gate_args(gate):
     return _p(t) + 4 * int(off), t.shape[1]
 
 
+class DistanceBias:
+    """A bias on attention scores by the distance from key to query and the query head: ``by_distance`` ``[n, heads]``, one row per distance
+    0 .. n-1, larger distances as the last one.  Held as ``table`` float32 ``[kv heads, n, heads of the group]`` (the rows a tile of
+    (token, head) pairs reads for one key lie side by side) beside each head's largest value.  ``narrow``: no head's values lie
+    further apart than `NARROW`, so that the largest may stand for a row's own maximum in a float32 softmax."""
+
+    NARROW = 40.0
+
+    def __init__(self, by_distance, nkv: int, device):
+        n, nq = by_distance.shape
+        t = by_distance.to(torch.float32)
+        self.n = int(n)
+        self.table = t.reshape(n, nkv, nq // nkv).permute(1, 0, 2).contiguous().to(device)
+        self.top = t.max(0).values.contiguous().to(device)
+        self.narrow = bool(((t.max(0).values - t.min(0).values) <= self.NARROW).all())
+
+    def nbytes(self) -> int:
+        return 4 * self.table.numel()
+
+    def args(self):
+        return _p(self.table), self.n, _p(self.top)
+
+
+_NO_REL = (None, 0, None)
+
+
 def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None,
-                   softcap: float = 0.0, gate=None):
+                   softcap: float = 0.0, gate=None, rel: "DistanceBias | None" = None):
     """The CUDA-core attention kernel: any head size up to 640 (one instance to 256, one beyond), float32 arithmetic.  ``sink`` (float32 ``[nq]``): the
     softmax's denominator also holds exp(sink_h), a term without key or value that the scale does not touch.  ``softcap``, ``gate``:
     see `paged_attention`."""
@@ -1479,7 +1658,8 @@ def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, n
     out = torch.empty_like(q)
     call("sllm_attention_simt", _p(q), _p(k_cache), _p(v_cache), _dt(q), _p(block_tables),
          block_tables.shape[1], _p(positions), _p(seq_of_token), T, nq, nkv, hd, page_size, float(scale),
-         int(window or 0), int(block or 0), _p(sink), float(softcap or 0.0), *_gate_args(gate), _p(out), _stream())
+         int(window or 0), int(block or 0), _p(sink), float(softcap or 0.0), *_gate_args(gate), *(rel.args() if rel else _NO_REL)[:2],
+         _p(out), _stream())
     return out
 
 
@@ -1553,7 +1733,7 @@ def choose_splits(num_small: int, nkv: int, max_ctx: int, ctas_per_sm: int = 2, 
 
 
 def attention_mma(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, decode: bool, num_splits: int,
-                  nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None):
+                  nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None, rel=None):
     """The tensor-core attention kernel on one tile list (see `attention_tiles`); the merge of a split context
     touches the rows of that list's requests only."""
     _chk(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles[0], tiles[1])
@@ -1569,7 +1749,7 @@ def attention_mma(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, de
     call("sllm_attention_mma", _p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_o), _p(part_lse), _p(block_tables),
          block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]), tiles[2], 1 if decode else 0,
          num_splits, T, nq, nkv, hd, k_cache.shape[2], float(scale), int(window or 0), int(block or 0), _p(sink),
-         float(softcap or 0.0), *_gate_args(gate), _stream())
+         float(softcap or 0.0), *_gate_args(gate), *(rel.args() if rel else _NO_REL)[:2], _stream())
     if num_splits > 1:
         launches["own"] += 1          # the combine kernel
     return out
@@ -1586,7 +1766,7 @@ def _tma_ctas_per_sm(hd: int) -> int:
 
 
 def attention_tma_decode(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, num_splits: int,
-                         nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None):
+                         nq, nkv, hd, scale, window, out=None, block=None, sink=None, softcap: float = 0.0, gate=None, rel=None):
     """The decode form fed by TMA (16-row tiles only; see `attention_tiles`)."""
     _chk(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles[0], tiles[1])
     if q.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16:
@@ -1601,7 +1781,7 @@ def attention_tma_decode(q, k_cache, v_cache, block_tables, q_start, ctx_len, ti
     call("sllm_attention_tma_decode", _p(q), _p(k_cache), _p(v_cache), k_cache.shape[0], _p(out), _p(part_o),
          _p(part_lse), _p(block_tables), block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]),
          tiles[2], num_splits, T, nq, nkv, hd, k_cache.shape[2], float(scale), int(window or 0), int(block or 0),
-         _p(sink), float(softcap or 0.0), *_gate_args(gate), _p(_status_word(q.device)), _stream())
+         _p(sink), float(softcap or 0.0), *_gate_args(gate), *(rel.args() if rel else _NO_REL)[:2], _p(_status_word(q.device)), _stream())
     _tc_used["since_check"] += 1
     if num_splits > 1:
         launches["own"] += 1
@@ -1637,7 +1817,7 @@ def choose_tc_splits(num_tiles: int, nkv: int, max_ctx: int) -> tuple[int, int]:
 
 
 def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq, nkv, hd, scale, out=None,
-                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, sink=None, softcap: float = 0.0, gate=None):
+                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, sink=None, softcap: float = 0.0, gate=None, rel=None):
     """The prefill form on tcgen05 (tiles of 128 * row_tiles rows, row_tiles 1 or 2; no window; see
     `attention_tiles`).  ``splits`` = (ranges, 64-key tiles a range) cuts the context into ranges
     that run as CTAs of their own and are merged afterwards; ranges x tiles must cover the longest
@@ -1659,7 +1839,7 @@ def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq,
          block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]), tiles[2], int(row_tiles), nq, nkv,
          hd, k_cache.shape[2], float(scale), n_splits, max(per, 1), T, _p(part_o), _p(part_lse),
          _p(parts[0]) if parts else None, _p(parts[1]) if parts else None, _p(sink), float(softcap or 0.0), *_gate_args(gate),
-         _p(_status_word(q.device)), _stream())
+         *(rel.args() if rel else _NO_REL), _p(_status_word(q.device)), _stream())
     if n_splits > 1:
         launches["own"] += 1               # the merge kernel
     _tc_used["since_check"] += 1
@@ -1706,10 +1886,11 @@ def mma_supports(hd: int) -> bool:
 
 
 def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, window, block=None, sink=None, softcap: float = 0.0,
-                    gate=None):
+                    gate=None, rel: "DistanceBias | None" = None):
     """Causal attention of the step's tokens over their requests' pages.  ``sink`` (float32 ``[nq]``): exp(sink_h) joins
     each head's softmax denominator (every form takes it).  ``softcap`` > 0: a score becomes softcap tanh(score / softcap) before
-    the softmax; ``gate`` = (float32 product, column): head h's output times sigmoid of column + h (every form takes both).  ``window``: only the last ``window`` keys;
+    the softmax; ``gate`` = (float32 product, column): head h's output times sigmoid of column + h; ``rel``: a bias on the scores by distance, added after scale and
+    cap (every form takes all three).  ``window``: only the last ``window`` keys;
     ``block``: only the keys of the query's own block of ``block`` positions, counted from the sequence's start (both
     run on the mma.sync and TMA-fed forms, not on tcgen05).  bfloat16 with a head size
     the tensor-core kernels take: requests of at most 16 (token, head-in-group) rows go to the decode
@@ -1719,11 +1900,12 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     g = step.groups[group]
     if q.dtype != torch.bfloat16 or not mma_supports(hd):
         return attention_simt(q, k_cache, v_cache, g.block_tables, step.positions, step.seq_of_token,
-                              nq, nkv, hd, scale, window, block, sink, softcap, gate)
+                              nq, nkv, hd, scale, window, block, sink, softcap, gate, rel)
     G = nq // nkv
     # blocks that start on page borders: the prefill form runs each block's part of a portion as a causal sequence of its own
     blocked_tc = bool(block) and block % k_cache.shape[2] == 0 and bool(step.ctx_lens)
-    use_tc = not window and (not block or blocked_tc) and _TC_ATTENTION and tc_attention_supports(hd, k_cache.shape[2])
+    use_tc = not window and (not block or blocked_tc) and _TC_ATTENTION and tc_attention_supports(hd, k_cache.shape[2]) and \
+        (rel is None or (rel.narrow and not block))
     key = ("mma", G, nkv, use_tc, block or 0)
     if key not in step.attn_tiles:
         # 128-row CTAs, two per SM.  (The kernel also has a form with two row tiles a CTA, one CTA per SM,
@@ -1747,19 +1929,19 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     out = torch.empty_like(q)
     if small and tma_attention_supports(hd, k_cache.shape[2]):
         attention_tma_decode(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, small, splits,
-                             nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
+                             nq, nkv, hd, scale, window, out, block, sink, softcap, gate, rel)
     elif small:
         attention_mma(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, small, True, splits,
-                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
+                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate, rel)
     if large and use_tc and parts is not None:
         attention_tc(q, k_cache, v_cache, g.block_tables, parts[0], parts[1], parts[3], nq, nkv, hd, scale, out,
                      row_tiles=rows // 128, parts=parts[2], sink=sink, softcap=softcap, gate=gate)
     elif large and use_tc:
         attention_tc(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, nq, nkv, hd, scale, out,
-                     row_tiles=rows // 128, splits=tc_splits, sink=sink, softcap=softcap, gate=gate)
+                     row_tiles=rows // 128, splits=tc_splits, sink=sink, softcap=softcap, gate=gate, rel=rel)
     elif large:
         attention_mma(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, False, 1,
-                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate)
+                      nq, nkv, hd, scale, window, out, block, sink, softcap, gate, rel)
     return out
 
 

@@ -59,8 +59,8 @@ def _declare(L):
         "sllm_qk_norm_rope_kv_write": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                        c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                        c_void_p],
-        "sllm_short_conv_silu": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                 c_int, c_int, c_void_p],
+        "sllm_short_conv_silu": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_norm_mean_add": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_void_p],
         "sllm_moe_route": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
         "sllm_moe_act": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -74,8 +74,9 @@ def _declare(L):
         "sllm_rope_kv_write": [c_void_p, c_int, c_int, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "sllm_gemm_f32": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-        "sllm_attention_simt": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                                c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
+        "sllm_attention_simt": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int,
+                                c_void_p, c_void_p],
         "sllm_sample_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "sllm_repetition_penalty": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "sllm_mark_seen": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
@@ -84,13 +85,15 @@ def _declare(L):
         "sllm_attention_tma_supports": [c_int, c_int],
         "sllm_attention_tma_ctas_per_sm": [c_int],
         "sllm_attention_tma_decode": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
-                                      c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                      c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
+                                      c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                      c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int,
+                                      c_void_p, c_void_p],
         "sllm_wait_probe": [c_void_p, ctypes.c_ulonglong, c_void_p, c_void_p],
         "sllm_attention_tc_supports": [c_int, c_int],
         "sllm_attention_tc": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
-                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
+                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int,
+                              c_void_p, c_void_p, c_void_p],
         "sllm_gemm_tcgen05_supports": [c_int, c_int, c_int],
         "sllm_gemm_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "sllm_gemm_pair_supports": [c_int, c_int, c_int],
@@ -117,9 +120,9 @@ def _declare(L):
         "sllm_linear_stream_splits": [c_int, c_int],
         "sllm_linear_stream": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                c_int, c_void_p],
-        "sllm_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                               c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                               c_int, c_int, c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p],
+        "sllm_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+                               c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p],
         "sllm_attention_mma_pooled": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
                                       c_int, c_int, c_int,
@@ -130,9 +133,10 @@ def _declare(L):
                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_mingru_scan": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                              c_int, c_void_p],
-        "sllm_gated_clamp_act": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                 c_int, c_void_p],
-        "sllm_moe_route_top_softmax": [c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
+        "sllm_gated_clamp_act": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                 c_float, c_int, c_void_p],
+        "sllm_moe_route_top_softmax": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
+                                       c_void_p],
         "sllm_add_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "sllm_norm_pair": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_forget_gate_attention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -144,8 +148,8 @@ def _declare(L):
                                        c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
         "sllm_rope_cols": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                            c_int, c_int, c_int, c_void_p],
-        "sllm_short_conv": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                            c_int, c_int, c_int, c_void_p],
+        "sllm_short_conv": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_decay_linear_attention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_retention": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
@@ -160,6 +164,23 @@ def _declare(L):
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_head_linear_strided": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
                                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_embed_streams": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p,
+                               ctypes.c_longlong, ctypes.c_longlong, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_void_p],
+        "sllm_streams_step": [c_void_p, c_void_p, c_int, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_whole_norm_kv_write": [c_void_p, c_int, c_size_t, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float,
+                                     c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                     c_void_p, c_int, c_int, c_void_p],
+        "sllm_norm_cols": [c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
+        "sllm_state_space": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_state_space_chunked_supports": [c_int, c_int],
+        "sllm_state_space_chunked": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                     c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                     c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "sllm_gated_group_norm": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_int,
+                                  c_void_p],
     }
     for name, argtypes in sigs.items():
         fn = getattr(L, name)

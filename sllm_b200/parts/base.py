@@ -46,7 +46,7 @@ import torch
 @dataclass(frozen=True)
 class TensorSpec:
     """A tensor a part expects.  ``role`` drives random initialisation
-    (matrix, bias, gain, embedding); optional tensors that only make sense
+    (matrix, bias, gain, embedding, and what `weights.random_init` knows besides); optional tensors that only make sense
     together share a ``together`` key.  An empty ``name`` is the tensor that carries
     the part's own prefix as its whole name.  A dimension of ``shape`` that is None is
     read from the checkpoint (a size the configuration does not give); random

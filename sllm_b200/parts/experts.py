@@ -16,6 +16,8 @@ either way once the batch holds a few tokens.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .. import ops
@@ -82,14 +84,17 @@ class GatedExperts(FeedForward):
         out = sum over the winners of weight_e * expert_e(x)
 
     With ``activation`` = ``silu`` an expert is W_down,e (silu(W_gate,e x) * W_up,e x) instead (no limit); ``scale`` (1 unless
-    given) multiplies the weights.  The softmax over the winners alone is also what a softmax over ALL experts gives once
+    given) multiplies the weights.  With ``router_bias`` the logits are W_router x + b (tensor ``router.b``), in the choice and in
+    the weights.  ``shared_ff`` > 0 adds one more such expert (``shared.*``, of its own size) that every token uses, times
+    sigmoid(w_sg x), one number per token (``shared.sg``).  The softmax over the winners alone is also what a softmax over ALL experts gives once
     the winners' scores are divided by their sum.
 
     Parameters: ``hidden_size``, ``experts``, ``top``, ``expert_ff``, ``limit``, ``alpha`` (1.702 unless given), ``activation``
-    (``clamped_swish`` unless given), ``scale``; no biases.  As
+    (``clamped_swish`` unless given), ``scale``, ``router_bias``, ``shared_ff``; the experts have no biases.  As
     in `RoutedExperts`, all experts' gate and up projections are ONE matrix (expert e's rows at 2 e ff, gate and up rows
     alternating in blocks of 8, or all of the expert's gate rows before its up rows where ff is no multiple of 8) and their
-    down projections one matrix side by side; a token's activation row carries its routing weights, so the second product
+    down projections one matrix side by side, the shared expert behind the others; w_sg is a row of the router's matrix (which is
+    padded with rows of zeros to a size the products' kernels take).  A token's activation row carries its routing weights, so the second product
     adds up the weighted experts in float32 in one order whatever the batch holds."""
 
     def __init__(self, params, **kw):
@@ -103,7 +108,13 @@ class GatedExperts(FeedForward):
             raise ValueError(f"gated_experts: activation {self.act!r}; known: clamped_swish, silu")
         self.limit, self.alpha = float(p.get("limit", 0.0) if self.act == "silu" else p["limit"]), float(p.get("alpha", 1.702))
         self.scale = float(p.get("scale", 1.0))
+        self.router_bias = bool(p.get("router_bias", False))
+        self.shared_ff = int(p.get("shared_ff") or 0)
+        if self.shared_ff and self.act != "silu":
+            raise ValueError("gated_experts: a shared expert goes with the silu activation")
         self.interleave = 8 if self.ff % 8 == 0 else self.ff
+        if self.shared_ff % self.interleave:            # blocks must not straddle two experts
+            self.interleave = math.gcd(self.interleave, self.shared_ff)
         if not 1 <= self.top <= self.E:
             raise ValueError(f"gated_experts: top={self.top} of {self.E} experts cannot be chosen")
 
@@ -113,28 +124,46 @@ class GatedExperts(FeedForward):
         for e in range(self.E):
             specs += [TensorSpec(f"e{e}.gate", (self.ff, W)), TensorSpec(f"e{e}.up", (self.ff, W)), TensorSpec(f"e{e}.down", (W, self.ff))]
         specs.append(TensorSpec("router", (self.E, W)))
+        if self.router_bias:
+            specs.append(TensorSpec("router.b", (self.E,), role="bias"))
+        if self.shared_ff:
+            s = self.shared_ff
+            specs += [TensorSpec("shared.gate", (s, W)), TensorSpec("shared.up", (s, W)), TensorSpec("shared.down", (W, s)),
+                      TensorSpec("shared.sg", (1, W))]
         return specs
 
     def bind(self, fetch):
         n, W = self.interleave, self.hidden
+        names = [f"e{e}" for e in range(self.E)] + (["shared"] if self.shared_ff else [])
         rows = []
-        for e in range(self.E):
-            g, u = fetch(f"e{e}.gate").reshape(self.ff // n, n, W), fetch(f"e{e}.up").reshape(self.ff // n, n, W)
-            rows.append(torch.stack([g, u], dim=1).reshape(2 * self.ff, W))
-        self.gate_up = Linear(self._matrix(torch.cat(rows, dim=0)))                                          # [2 E ff, W]
-        self.down = Linear(self._matrix(torch.cat([fetch(f"e{e}.down") for e in range(self.E)], dim=1)))     # [W, E ff]
-        self.router = Linear(self._matrix(fetch("router")))
+        for e in names:
+            g, u = fetch(f"{e}.gate"), fetch(f"{e}.up")
+            rows.append(torch.stack([g.reshape(-1, n, W), u.reshape(-1, n, W)], dim=1).reshape(2 * g.shape[0], W))
+        self.gate_up = Linear(self._matrix(torch.cat(rows, dim=0)))                                # [2 (E ff + shared), W]
+        self.down = Linear(self._matrix(torch.cat([fetch(f"{e}.down") for e in names], dim=1)))    # [W, E ff + shared]
+        router, bias = fetch("router"), None
+        if self.shared_ff:
+            router = torch.cat([router, fetch("shared.sg")], dim=0)
+        if self.router_bias or self.shared_ff:
+            pad = -router.shape[0] % 16
+            router = torch.cat([router, torch.zeros((pad, W), dtype=router.dtype)], dim=0)
+            if self.router_bias:
+                bias = torch.zeros(router.shape[0], dtype=torch.float32)
+                bias[:self.E] = fetch("router.b").float()
+                bias = self._f32(bias)
+        self.router = Linear(self._matrix(router), bias)
 
     accepts_residual = True
 
     def route(self, x):
-        """(dense weights [T, E], indices [T, top], weights [T, top]) of the normed rows ``x``."""
-        return ops.moe_route_top_softmax(self.router(x, torch.float32), self.top, self.scale)
+        """(dense weights [T, E], or [T, E + 1] with a shared expert, indices [T, top], weights [T, top]) of the normed rows ``x``."""
+        return ops.moe_route_top_softmax(self.router(x, torch.float32), self.top, self.scale, experts=self.E, gated=1 if self.shared_ff else 0)
 
     def forward(self, x, step, residual=None):
         dense, _, _ = self.route(x)
         gu = self.gate_up(x, self.dtype)                                                                     # [T, 2 E ff]
-        act = ops.gated_clamp_act(gu, self.interleave, self.limit, self.dtype, alpha=self.alpha, dense=dense, ff=self.ff, act=self.act)
+        act = ops.gated_clamp_act(gu, self.interleave, self.limit, self.dtype, alpha=self.alpha, dense=dense, ff=self.ff, act=self.act,
+                                  tail=self.shared_ff)
         return self.down.into(act, residual)
 
     def weight_bytes(self):

@@ -34,6 +34,11 @@ class LatentAttention(Mixer):
     score is the sum of both dot products.  The cache then holds [latent | rotated key part] per token as one key-and-value
     head (its value is read from the latent's columns only), a query is [its carried form | its rotated part].
     ``sink`` true: a learned number per head (``sink``) whose exponential joins the softmax's denominator.
+    ``q_rank`` > 0: queries go through a latent of their own, q = W_uq (rmsnorm(W_dq x) * gain) (tensors ``dq``, ``dq.norm`` and
+    ``uq`` in place of ``q``).  ``window``: a query sees the keys of the last ``window`` positions, its own among them.  ``rotary``
+    with ``interleaved`` true pairs channel 2i with 2i + 1 in place of i with i + rotary_dim/2: a dot product of two rotated vectors
+    does not change when the channels of both are put in another order, so the rows of the two matrices that make the rotated
+    parts are reordered when they are bound, and the kernels see the usual layout.
     ``shared_kv`` true: the layer has no down-projection of its own and reads the cache another run wrote."""
 
     MAX_RANK = 640      # the CUDA-core attention kernel's largest head (its second instance; the tensor-core forms end at 128)
@@ -57,6 +62,9 @@ class LatentAttention(Mixer):
         rot = params.get("rotary") if self.rot_dim else None
         self.rot_params = dict(rot) if rot else None
         self.rot = int(rot["rotary_dim"]) if rot else 0
+        self.interleaved = bool(self.rot_params.pop("interleaved", False)) if rot else False
+        self.q_rank = int(params.get("q_rank") or 0)
+        self.window = int(params["window"]) if params.get("window") else None
         if self.rot % 2 or self.rot > self.rot_dim:
             raise ValueError(f"latent_attention: {self.rot} rotated channels must be even and at most rot_dim={self.rot_dim}")
         D = self.rank + self.rot_dim
@@ -70,11 +78,15 @@ class LatentAttention(Mixer):
         self.sink = None
 
     def cache_need(self):
-        return PagedKV(1, self.D, None, values=False)
+        return PagedKV(1, self.D, self.window, values=False)
 
     def tensor_specs(self):
         H, W, r = self.heads, self.hidden, self.rank
-        specs = [TensorSpec("q", (H * (self.dim + self.rot_dim), W))]
+        Q = H * (self.dim + self.rot_dim)
+        if self.q_rank:
+            specs = [TensorSpec("dq", (self.q_rank, W)), TensorSpec("dq.norm", (self.q_rank,), role="gain"), TensorSpec("uq", (Q, self.q_rank))]
+        else:
+            specs = [TensorSpec("q", (Q, W))]
         if not self.shared_kv:
             specs += [TensorSpec("dkv", (r + self.rot_dim, W)), TensorSpec("dkv.norm", (r,), role="gain")]
         specs += [TensorSpec("uk", (H * self.dim, r)), TensorSpec("uv", (H * self.vdim, r))]
@@ -87,10 +99,17 @@ class LatentAttention(Mixer):
 
     def bind(self, fetch):
         H, r = self.heads, self.rank
-        names = ["q"] + ([] if self.shared_kv else ["dkv"]) + (["g"] if self.gate else [])
-        self.inp = Linear(self._matrix(torch.cat([fetch(n) for n in names], dim=0)))
         self.qdim = self.dim + self.rot_dim
-        self.off_c = H * self.qdim
+        q = self._usual_order(fetch("uq" if self.q_rank else "q"), H, self.qdim, self.dim)
+        rows = [fetch("dq") if self.q_rank else q]
+        if not self.shared_kv:
+            rows.append(self._usual_order(fetch("dkv"), 1, r + self.rot_dim, r))
+        if self.gate:
+            rows.append(fetch("g"))
+        self.inp = Linear(self._matrix(torch.cat(rows, dim=0)))
+        self.uq = Linear(self._matrix(q)) if self.q_rank else None
+        self.q_gain = self._f32(fetch("dq.norm")) if self.q_rank else None
+        self.off_c = self.q_rank or H * self.qdim
         self.off_g = self.off_c + (0 if self.shared_kv else r + self.rot_dim)
         self.c_gain = None if self.shared_kv else self._f32(fetch("dkv.norm"))
         # [H, rank, dim]: carries a head's query into the latent space;  [H, vdim, rank]: a head's latent sum out of it
@@ -103,12 +122,23 @@ class LatentAttention(Mixer):
             from .side_by_side import rotary_for
             self.rotary = rotary_for(self.rot_params, self.dtype, self.device)
 
+    def _usual_order(self, w, heads: int, rows: int, first: int):
+        """The rows ``first .. first + rot`` of each of ``heads`` blocks of ``rows`` rows put from pairs (2i, 2i+1) into halves."""
+        if not self.interleaved:
+            return w
+        order = list(range(first)) + list(range(first, first + self.rot, 2)) + list(range(first + 1, first + self.rot, 2)) + \
+            list(range(first + self.rot, rows))
+        return w.reshape(heads, rows, -1)[:, order].reshape(w.shape).contiguous()
+
     accepts_residual = True
 
     def forward(self, x, step: StepContext, cache: LayerCache, position, write_cache=True, residual=None):
         g = step.groups[cache.group]
         table = self.rotary.table if self.rotary is not None else None
         proj = self.inp(x, torch.float32)                                           # [T, H*(dim+rot_dim) (+ rank+rot_dim) (+ gate)] float32
+        q = proj
+        if self.q_rank:
+            q = self.uq(ops.norm_cols(proj, 0, self.q_rank, self.q_gain, self.eps, self.dtype), torch.float32)
         if write_cache and not self.shared_kv:
             if self.rot_dim:
                 ops.latent_rope_write(proj, self.off_c, self.rank, self.rot_dim, self.rot, self.c_gain, self.eps, step.positions,
@@ -116,14 +146,14 @@ class LatentAttention(Mixer):
             else:
                 ops.latent_write(proj, self.off_c, self.rank, self.c_gain, self.eps, g.slot_mapping, cache.k)
         # [T, H*D] queries: a head's unrotated part carried into the latent space, its rotated part behind it
-        ql = ops.head_linear(proj, 0, self.uk_t, self.dtype, xstride=self.qdim, ostride=self.D)
+        ql = ops.head_linear(q, 0, self.uk_t, self.dtype, xstride=self.qdim, ostride=self.D)
         if self.D > self.rank:
-            ops.rope_cols_(ql, self.rank, self.D, proj, self.dim, self.qdim, self.rot_dim, self.rot, step.positions, table, self.heads)
-        al = ops.paged_attention(ql, cache.k, cache.v, step, cache.group, self.heads, 1, self.D, self.scale, None, sink=self.sink)
+            ops.rope_cols_(ql, self.rank, self.D, q, self.dim, self.qdim, self.rot_dim, self.rot, step.positions, table, self.heads)
+        al = ops.paged_attention(ql, cache.k, cache.v, step, cache.group, self.heads, 1, self.D, self.scale, self.window, sink=self.sink)
         y = ops.head_linear(al, 0, self.uv, self.dtype, gate=proj if self.gate else None, goff=self.off_g,
                             gate_elem=self.gate == "element", xstride=self.D)      # [T, H*vdim]
         return self.out.into(y, residual)
 
     def weight_bytes(self):
-        n = self.inp.nbytes() + self.out.nbytes() + 4 * self.rank + (4 * self.heads if self.has_sink else 0)
+        n = self.inp.nbytes() + self.out.nbytes() + (self.uq.nbytes() + 4 * self.q_rank if self.q_rank else 0) + 4 * self.rank + (4 * self.heads if self.has_sink else 0)
         return n + (self.uk_t.numel() + self.uv.numel()) * self.uk_t.element_size()

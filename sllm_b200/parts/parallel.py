@@ -156,10 +156,10 @@ class GatedDense(FeedForward):
 
 @FEED_FORWARDS.register("plain_dense")
 class PlainDense(FeedForward):
-    """down(act(up(x))): two matrices without biases and an activation between them, ``relu2`` (max(z, 0)^2).  The activation
-    leaves with the first product's tile where that product's kernel has it (`ops.linear_plain_act`)."""
+    """down(act(up(x))): two matrices without biases and an activation between them, ``relu2`` (max(z, 0)^2) or ``gelu`` (the exact
+    one, by erf).  The activation leaves with the first product's tile where that product's kernel has it (`ops.linear_plain_act`)."""
 
-    ACTIVATIONS = ("relu2",)
+    ACTIVATIONS = ("relu2", "gelu")
 
     def __init__(self, params, **kw):
         super().__init__(params, **kw)

@@ -4,7 +4,8 @@
 gain of the head's size, shared by the heads, or none) before they are rotated; it owns its rotary table (each layer may have
 other frequencies, and a two-regime frequency scaling); a query may be restricted to the keys of its own block of
 positions; the value size may differ from the key size; scores may be capped, a head's output gated, and the keys and values
-another layer's.
+another layer's.  Or the norms run over the whole query and key projections before the heads are split, with biases, a query
+factor that grows with the position, and a learned bias on the scores by bucketed distance.
 
 `SideBySide`: both mixers read the same input; the layer's term is the mean of their outputs, each first RMS-normed over
 the model width with a gain of its own.
@@ -24,6 +25,21 @@ from .. import ops
 from ..config.plan import PartSpec
 from .base import MIXERS, POSITIONS, LayerCache, Mixer, PagedKV, StepContext, TensorSpec, flatten_needs, join_name
 from .standard import Linear
+
+def distance_buckets(buckets: int, limit: int) -> list:
+    """The bucket of every distance 0 .. limit (larger distances share the last one's): n itself below h = buckets // 2, else
+    min(buckets - 1, h + floor(ln(n / h) / ln(limit / h) * (buckets - h))).  In whole numbers, so that a distance on a bucket's
+    border falls where the formula puts it: floor(...) >= k where (n / h)^(buckets - h) >= (limit / h)^k."""
+    h = buckets // 2
+    if h < 1 or limit <= h:
+        raise ValueError(f"distance buckets: {buckets} buckets up to a distance of {limit} (needs at least 2 buckets and more than half as many distances)")
+    out, k = list(range(h)), 0
+    for n in range(h, limit + 1):
+        while k < buckets - 1 - h and n ** (buckets - h) * h ** (k + 1) >= limit ** (k + 1) * h ** (buckets - h):
+            k += 1
+        out.append(h + k)
+    return out
+
 
 _TABLES: dict = {}       # rotary tables by their parameters: layers with the same frequencies share one
 
@@ -46,6 +62,11 @@ class NormedAttention(Mixer):
     norms have no gain, so that norming before or after the rotation is the same), ``softcap`` (scores become softcap
     tanh(score / softcap)), ``head_gate`` (true: a matrix ``g`` with a row per query head, whose output is multiplied by
     sigmoid(g x)_h), ``shared_kv`` (true: the layer has no keys and values of its own and reads the cache another run wrote).
+    ``norm_over`` = ``projection`` (``head`` unless given): the norms run over all rows of the query and of the key projection at once,
+    with gains of those sizes; no rotation then.  ``bias`` and ``out_bias``: the projections (``q.b``, ``k.b``, ``v.b``) and the output
+    (``o.b``) have biases.  ``q_temp`` (``coef``, ``every``): q times 1 + coef ln(floor((p + 1) / every) + 1) at position p.
+    ``distance_bias``: a table ``rel`` ``[buckets, heads]`` whose row for the distance's bucket (`distance_buckets` up to this distance)
+    is added to the score after scale and cap; the number of buckets is the tensor's.
     All of the layer's input matrices are one product.
 
     The cache's head holds max(dim, vdim) channels (rounded up to a size the tensor-core kernels take, in bfloat16):
@@ -71,6 +92,15 @@ class NormedAttention(Mixer):
         rot = p.get("rotary")
         self.rot_params = dict(rot, max_positions=self.max_positions) if rot else None
         self.rot = int(rot["rotary_dim"]) if rot else 0
+        self.whole_norm = p.get("norm_over", "head") == "projection"
+        self.has_bias, self.out_bias = bool(p.get("bias", False)), bool(p.get("out_bias", False))
+        qt = p.get("q_temp")
+        self.q_temp = (float(qt["coef"]), int(qt["every"])) if qt else None
+        self.distance_bias = int(p["distance_bias"]) if p.get("distance_bias") else None
+        self.rel = None
+        if (self.has_bias or self.q_temp) and not self.whole_norm or self.whole_norm and (self.rot or not self.head_gain or self.head_gate):
+            raise ValueError("normed_attention: biases and the query factor go with norms over the whole projections, those with gains, and "
+                             "without rotation or head gates")
         if self.nq % self.nkv:
             raise ValueError(f"normed_attention: {self.nq} query heads are no multiple of {self.nkv} key/value heads")
         if self.rot % 2 or self.rot > self.dim:
@@ -91,10 +121,18 @@ class NormedAttention(Mixer):
         specs = [TensorSpec("q", (self.nq * self.dim, W))]
         if not self.shared_kv:
             specs += [TensorSpec("k", (self.nkv * self.dim, W)), TensorSpec("v", (self.nkv * self.vdim, W))]
-        if self.head_gain:
-            specs.append(TensorSpec("q.norm", (self.dim,), role="gain"))
+        if self.has_bias:
+            specs.append(TensorSpec("q.b", (self.nq * self.dim,), role="bias"))
             if not self.shared_kv:
-                specs.append(TensorSpec("k.norm", (self.dim,), role="gain"))
+                specs += [TensorSpec("k.b", (self.nkv * self.dim,), role="bias"), TensorSpec("v.b", (self.nkv * self.vdim,), role="bias")]
+        if self.head_gain:
+            specs.append(TensorSpec("q.norm", (self.nq * self.dim if self.whole_norm else self.dim,), role="gain"))
+            if not self.shared_kv:
+                specs.append(TensorSpec("k.norm", (self.nkv * self.dim if self.whole_norm else self.dim,), role="gain"))
+        if self.distance_bias:
+            specs.append(TensorSpec("rel", (None, self.nq), role="bias", shape_default=(16, self.nq)))
+        if self.out_bias:
+            specs.append(TensorSpec("o.b", (W,), role="bias"))
         if self.head_gate:
             specs.append(TensorSpec("g", (self.nq, W)))
         return specs + [TensorSpec("o", (W, self.nq * self.vdim))]
@@ -102,6 +140,10 @@ class NormedAttention(Mixer):
     def bind(self, fetch):
         names = ["q"] + ([] if self.shared_kv else ["k", "v"]) + (["g"] if self.head_gate else [])
         self.qkv = Linear(self._matrix(torch.cat([fetch(n) for n in names], dim=0)))
+        self.qkv_b = self._f32(torch.cat([fetch(f"{n}.b").float() for n in names])) if self.has_bias else None   # added where the norms are taken
+        if self.distance_bias:
+            rel = fetch("rel").float()
+            self.rel = ops.DistanceBias(rel[distance_buckets(rel.shape[0], self.distance_bias)], self.nkv, self.device)
         self.off_g = self.nq * self.dim + (0 if self.shared_kv else self.nkv * (self.dim + self.vdim))
         if self.head_gain:
             self.q_gain = self._f32(fetch("q.norm"))
@@ -113,7 +155,7 @@ class NormedAttention(Mixer):
             wide = torch.zeros((self.hidden, self.nq, self.D), dtype=o.dtype)
             wide[:, :, :self.vdim] = o.reshape(self.hidden, self.nq, self.vdim)
             o = wide.reshape(self.hidden, self.nq * self.D)
-        self.out = Linear(self._matrix(o))
+        self.out = Linear(self._matrix(o), self._f32(fetch("o.b")) if self.out_bias else None)
         if self.rot_params is not None:
             self.rotary = rotary_for(self.rot_params, self.dtype, self.device)
 
@@ -121,19 +163,27 @@ class NormedAttention(Mixer):
 
     def mix(self, x, step: StepContext, cache: LayerCache, position=None, write_cache=True):
         g = step.groups[cache.group]
+        if self.whole_norm:
+            qkv = self.qkv(x, torch.float32, True)                                   # (maybe in parts: the next kernel adds them)
+            q = ops.whole_norm_kv_write(qkv, self.qkv_b, self.q_gain, self.k_gain, self.eps, step.positions, self.q_temp, self.nq, self.nkv,
+                                        self.dim, self.vdim, g.slot_mapping if write_cache and not self.shared_kv else None, cache.k, cache.v,
+                                        self.dtype)
+            return ops.paged_attention(q, cache.k, cache.v, step, cache.group, self.nq, self.nkv, self.D, self.scale, None, self.block,
+                                       softcap=self.softcap, rel=self.rel)
         qkv = self.qkv(x, torch.float32)                                             # [T, (nq+nkv) dim + nkv vdim (+ nq)] float32
         write_cache = write_cache and not self.shared_kv
         q = ops.qk_norm_rope_kv_write(qkv, self.q_gain, self.k_gain, self.eps, step.positions,
                                       self.rotary.table if self.rotary is not None else None, self.rot, self.nq, self.nkv,
                                       self.dim, self.vdim, g.slot_mapping if write_cache else None, cache.k, cache.v, self.dtype)
         return ops.paged_attention(q, cache.k, cache.v, step, cache.group, self.nq, self.nkv, self.D, self.scale, None, self.block,
-                                   softcap=self.softcap, gate=(qkv, self.off_g) if self.head_gate else None)
+                                   softcap=self.softcap, gate=(qkv, self.off_g) if self.head_gate else None, rel=self.rel)
 
     def forward(self, x, step, cache, position, write_cache=True, residual=None):
         return self.out.into(self.mix(x, step, cache, position, write_cache), residual)
 
     def weight_bytes(self):
-        return self.qkv.nbytes() + self.out.nbytes() + 8 * self.dim
+        n = self.qkv.nbytes() + self.out.nbytes() + 4 * (self.q_gain.numel() + self.k_gain.numel())
+        return n + (4 * self.qkv_b.numel() if self.has_bias else 0) + (self.rel.nbytes() if self.rel is not None else 0)
 
 
 @MIXERS.register("side_by_side")

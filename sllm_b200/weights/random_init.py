@@ -39,6 +39,10 @@ def random_tensors(specs, seed: int, *, std: float = 0.02, bias_std: float | Non
             a = gain_std * rng.standard_normal(shape, dtype=np.float32) if gain_std else np.zeros(shape, np.float32)
         elif s.role == "bias":
             a = bias_std * rng.standard_normal(shape, dtype=np.float32)
+        elif s.role == "identity":         # a square matrix near the identity
+            a = np.eye(shape[0], shape[1], dtype=np.float32) + std * rng.standard_normal(shape, dtype=np.float32)
+        elif s.role == "share":            # weights of a sum, near equal parts of one
+            a = 1.0 / shape[0] + std * rng.standard_normal(shape, dtype=np.float32)
         elif s.role == "mix":              # a blend between two vectors, per channel: values in (0, 1)
             a = rng.uniform(0.05, 0.95, shape).astype(np.float32)
         else:

@@ -17,6 +17,37 @@ def embed_gather(table, ids, scale=1.0):
     return table[ids.long()].float() * scale
 
 
+def embed_streams(table, step, scale, copies, pair_table=None, before=None, pairs=None):
+    ids = step.token_ids.long()
+    x = table[ids].float() * scale
+    if pairs is not None:
+        prev = torch.zeros_like(ids)
+        prev[1:] = ids[:-1]
+        starts = step.q_start.long().tolist()
+        for s in range(step.num_seqs):
+            slot = int(step.state_slots[s])
+            prev[starts[s]] = int(before[slot, 0])
+            before[slot, 0] = float(ids[starts[s + 1] - 1])
+        row = torch.where(step.positions.long() == 0, torch.full_like(ids, pairs.buckets), (prev * pairs.mul_prev + ids * pairs.mul_cur) % pairs.buckets)
+        x = x + pair_table[row].float()
+    return x if copies is None else x[:, None, :].repeat(1, copies, 1)
+
+
+def streams_step(streams, term, mix, share, into, gain, eps, out_dtype, rows=None):
+    x = streams if rows is None else streams[rows.long()]
+    if term is not None:
+        t = term.float().sum(0) if term.dim() == 3 else term.float()
+        if rows is not None:
+            t = t[rows.long()]
+        x = torch.einsum("tsw,sr->trw", x, mix) + share[None, :, None] * t[:, None, :]
+        if rows is None:
+            streams.copy_(x)
+    if gain is None:
+        return None
+    u = torch.einsum("tsw,s->tw", x, into)
+    return (u * (u.pow(2).mean(-1, keepdim=True) + eps).rsqrt() * gain).to(out_dtype)
+
+
 def add_sinusoid_(stream, positions, inv_freq):
     ang = positions.float()[:, None] * inv_freq[None, :]
     stream[:, 0::2] += torch.sin(ang)
@@ -220,7 +251,62 @@ def qk_norm_rope_kv_write(qkv, q_gain, k_gain, eps, positions, table, rotary_dim
     return qk[:, :nq].reshape(T, nq * D).to(out_dtype)
 
 
-def short_conv_silu(x, off, weight, state, step):
+def whole_norm_kv_write(qkv, bias, q_gain, k_gain, eps, positions, q_temp, nq, nkv, dim, vdim, slot_mapping, k_cache, v_cache, out_dtype):
+    x = qkv.float().sum(0) if qkv.dim() == 3 else qkv.float()
+    if bias is not None:
+        x = x + bias
+    T, D = x.shape[0], k_cache.shape[3]
+
+    def normed(y, gain):
+        return y * (y.pow(2).mean(-1, keepdim=True) + eps).rsqrt() * gain
+    q = normed(x[:, :nq * dim], q_gain)
+    if q_temp is not None:
+        coef, every = q_temp
+        q = q * (1.0 + coef * torch.log((positions.long() + 1).div(every, rounding_mode="floor").float() + 1.0))[:, None]
+    pad = lambda y, h, d: torch.nn.functional.pad(y.reshape(T, h, d), (0, D - d))
+    if slot_mapping is not None:
+        ps = k_cache.shape[2]
+        ok = slot_mapping >= 0
+        page, off = slot_mapping[ok].long() // ps, slot_mapping[ok].long() % ps
+        k = normed(x[:, nq * dim:(nq + nkv) * dim], k_gain)
+        k_cache[page, :, off, :] = pad(k, nkv, dim)[ok].to(k_cache.dtype)
+        v_cache[page, :, off, :] = pad(x[:, (nq + nkv) * dim:(nq + nkv) * dim + nkv * vdim], nkv, vdim)[ok].to(v_cache.dtype)
+    return pad(q, nq, dim).reshape(T, nq * D).to(out_dtype)
+
+
+def norm_cols(x, off, n, gain, eps, out_dtype):
+    y = x[:, off:off + n]
+    return (y * (y.pow(2).mean(-1, keepdim=True) + eps).rsqrt() * gain).to(out_dtype)
+
+
+def state_space_walk(xbc, proj, off_dt, dt_bias, a_log, skip, state, step, heads, groups, n, dv, max_len=0, out=None):
+    T, I, rep = xbc.shape[0], heads * dv, heads // groups
+    x = xbc[:, :I].reshape(T, heads, dv)
+    B = xbc[:, I:I + groups * n].reshape(T, groups, n).repeat_interleave(rep, dim=1)
+    C = xbc[:, I + groups * n:].reshape(T, groups, n).repeat_interleave(rep, dim=1)
+    dt = torch.nn.functional.softplus(proj[:, off_dt:off_dt + heads] + dt_bias)
+    keep = torch.exp(-torch.exp(a_log) * dt)
+    y = torch.empty((T, heads, dv), dtype=torch.float32, device=xbc.device)
+
+    def token(t, S):
+        S = keep[t][:, None, None] * S + (dt[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+        return S, torch.einsum("hij,hi->hj", S, C[t]) + skip[:, None] * x[t]
+    _walk(step, state, y, token)
+    return y.reshape(T, I)
+
+
+def state_space(*args):
+    return state_space_walk(*args)
+
+
+def gated_group_norm(y, gate, off_g, gain, eps, groups, out_dtype):
+    T, n = y.shape
+    z = gate[:, off_g:off_g + n]
+    v = (y * z * torch.sigmoid(z)).reshape(T, groups, n // groups)
+    return ((v * (v.pow(2).mean(-1, keepdim=True) + eps).rsqrt()).reshape(T, n) * gain).to(out_dtype)
+
+
+def short_conv_silu(x, off, weight, state, step, bias=None):
     C, taps = weight.shape
     T = x.shape[0]
     out = torch.empty((T, C), dtype=torch.float32, device=x.device)
@@ -234,6 +320,8 @@ def short_conv_silu(x, off, weight, state, step):
         acc = torch.zeros((b - a, C), dtype=torch.float32, device=x.device)
         for j in range(taps):
             acc += padded[j:j + b - a] * weight[:, j]
+        if bias is not None:
+            acc = acc + bias
         out[a:b] = acc * torch.sigmoid(acc)
         if taps > 1:
             state[slot] = padded[padded.shape[0] - (taps - 1):].t()
@@ -349,7 +437,10 @@ def short_conv_add(x, weight, state, step, out_dtype):
     return out.to(out_dtype)
 
 
-def moe_route_top_softmax(logits, top, scale=1.0):
+def moe_route_top_softmax(logits, top, scale=1.0, experts=None, gated=0):
+    if experts is not None:
+        dense, idx, wts = moe_route_top_softmax(logits[:, :experts], top, scale)
+        return torch.cat([dense, torch.sigmoid(logits[:, experts:experts + gated].float())], dim=1), idx, wts
     T, E = logits.shape
     idx = torch.sort(-logits.float(), dim=-1, stable=True).indices[:, :top]
     wts = torch.softmax(logits.float().gather(1, idx), dim=-1) * scale
@@ -358,7 +449,7 @@ def moe_route_top_softmax(logits, top, scale=1.0):
     return dense, idx.int(), wts
 
 
-def gated_clamp_act(gu, interleave, limit, out_dtype, *, alpha=1.702, dense=None, ff=None, act="clamped_swish"):
+def gated_clamp_act(gu, interleave, limit, out_dtype, *, alpha=1.702, dense=None, ff=None, act="clamped_swish", tail=0):
     T, two_n = gu.shape
     N = two_n // 2
     v = gu.float().reshape(T, N // interleave, 2, interleave)
@@ -370,7 +461,9 @@ def gated_clamp_act(gu, interleave, limit, out_dtype, *, alpha=1.702, dense=None
         u = v[:, :, 1, :].reshape(T, N).clamp(-limit, limit)
         y = g * torch.sigmoid(alpha * g) * (u + 1.0)
     if dense is not None:
-        y = y * dense.repeat_interleave(ff, dim=1)
+        w = dense.repeat_interleave(ff, dim=1) if not tail else \
+            torch.cat([dense[:, :-1].repeat_interleave(ff, dim=1), dense[:, -1:].expand(T, tail)], dim=1)
+        y = y * w
     return y.to(out_dtype)
 
 
@@ -398,6 +491,8 @@ def plain_act(x, out_dtype, act, token=None):
     x = x.float().sum(0) if x.dim() == 3 else x
     if act == "relu2":
         return torch.relu(x.float()).square().to(out_dtype)
+    if act == "gelu":
+        return torch.nn.functional.gelu(x.float()).to(out_dtype)
     e = token.table[token.ids.long(), token.off:token.off + x.shape[1]].float()
     return (torch.nn.functional.gelu(x.float(), approximate="tanh") * e).to(out_dtype)
 
@@ -527,7 +622,7 @@ def rope_kv_write(qkv, bias, positions, table, rotary_dim, nq, nkv, hd, slot_map
 
 
 def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, nq, nkv, hd, scale, window, block=None, sink=None,
-                   softcap=0.0, gate=None):
+                   softcap=0.0, gate=None, rel=None):
     T = q.shape[0]
     ps = k_cache.shape[2]
     out = torch.empty((T, nq, hd), dtype=torch.float32, device=q.device)
@@ -547,6 +642,8 @@ def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, n
         s = torch.einsum("hd,nhd->hn", qf[t], k) * scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
+        if rel is not None:                                # table [kv heads, distances, heads of the group]
+            s = s + rel.table[:, torch.clamp(pos - j, max=rel.n - 1)].permute(0, 2, 1).reshape(nq, -1)
         if sink is not None:                               # one more term of the denominator: no key, no value, not scaled
             p = torch.softmax(torch.cat([s, sink.float()[:, None]], dim=-1), dim=-1)[:, :-1]
         else:
@@ -557,10 +654,10 @@ def attention_simt(q, k_cache, v_cache, block_tables, positions, seq_of_token, n
     return out.reshape(T, nq * hd).to(q.dtype)
 
 
-def paged_attention(q, k_cache, v_cache, step, group, nq, nkv, hd, scale, window, block=None, sink=None, softcap=0.0, gate=None):
+def paged_attention(q, k_cache, v_cache, step, group, nq, nkv, hd, scale, window, block=None, sink=None, softcap=0.0, gate=None, rel=None):
     g = step.groups[group]
     return attention_simt(q, k_cache, v_cache, g.block_tables, step.positions, step.seq_of_token,
-                          nq, nkv, hd, scale, window, block, sink, softcap, gate)
+                          nq, nkv, hd, scale, window, block, sink, softcap, gate, rel)
 
 
 def pool_kv_write(k_cache, v_cache, step, group, pk_cache, pv_cache, pool_group, pool):
@@ -658,7 +755,7 @@ def penalty_from_seen_(logits, seen, step, penalty):
     return logits
 
 
-ALL = ["retention", "retention_gated", "post_add_copy", "softcap_", "plain_act", "linear_plain_act", "forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
+ALL = ["embed_streams", "streams_step", "whole_norm_kv_write", "norm_cols", "state_space_walk", "state_space", "gated_group_norm", "retention", "retention_gated", "post_add_copy", "softcap_", "plain_act", "linear_plain_act", "forget_gate_attention", "add_rows_", "norm_pair", "pool_kv_write", "pooled_attention", "post_add_norm_conv", "latent_rope_write", "rope_cols_", "short_conv_add", "moe_route_top_softmax", "gated_clamp_act", "post_add_norm", "mingru_scan",
        "decay_linear_attention", "gated_delta_rule", "gated_linear_attention", "qk_norm_rope_kv_write", "short_conv_silu", "norm_mean_add_", "moe_route", "moe_act",
        "add_sinusoid_", "add_group_ssq", "group_norm_shift", "act_mul", "linear_act_mul", "tanh_cols", "delta_rule", "delta_out", "latent_write",
        "head_linear", "embed_gather", "add_rmsnorm", "linear", "can_accumulate", "linear_accumulate", "silu_mul", "linear_silu_mul", "rope_kv_write",
