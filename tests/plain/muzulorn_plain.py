@@ -225,7 +225,9 @@ def gated_unit(h, w, p):
     return (silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
-def experts(h, w, p, mlp):
+def experts(h, w, p, mlp, margins=None):
+    """``margins`` (a list) receives, per token, the gap between the last chosen expert's logit and the best one left out, relative to
+    the logits' spread."""
     z = h @ w[p + "router"].T + w[p + "router.b"]
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
@@ -234,13 +236,17 @@ def experts(h, w, p, mlp):
             out[t] += weight * gated_unit(h[t:t + 1], w, f"{p}e{e}.")[0]
     if mlp.get("shared") is not None:
         out = out + gated_unit(h, w, p + "shared.") * sigmoid(h @ w[p + "shared.sg"].T)
+    top = mlp["router"]["top"]
+    if margins is not None and top < z.shape[1]:
+        s = -np.sort(-z, axis=1)
+        margins.append((s[:, top - 1] - s[:, top]) / np.sqrt((z * z).mean(-1)))
     return out
 
 
-def feed_forward(h, w, p, mlp):
+def feed_forward(h, w, p, mlp, margins=None):
     if mlp["kind"] == "dense":
         return gelu(h @ w[p + "up"].T) @ w[p + "down"].T
-    return experts(h, w, p, mlp)
+    return experts(h, w, p, mlp, margins)
 
 
 # ---- the streams --------------------------------------------------------------------------------------
@@ -255,8 +261,9 @@ def connect(streams, w, p, mult, sublayer):
 
 # ---- the model ------------------------------------------------------------------------------------
 
-def forward(ids, cfg, w, after_layers=None):
-    """Logits [T, vocab] of one whole sequence.  ``after_layers`` (a list) receives the sum of the streams after every layer."""
+def forward(ids, cfg, w, after_layers=None, margins=None):
+    """Logits [T, vocab] of one whole sequence.  ``after_layers`` (a list) receives the sum of the streams after every layer,
+    ``margins`` what `experts` says of every router."""
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     x = embedding(list(ids), cfg, w)
     streams = np.repeat(x[None], cfg["streams"], axis=0)
@@ -276,7 +283,7 @@ def forward(ids, cfg, w, after_layers=None):
             return attention(h, w, p + "mix.", m, eps, kept[i if src is None else src])
         streams = connect(streams, w, p + "hc1.", mult, mixer)
         if layer["mlp"] is not None:
-            streams = connect(streams, w, p + "hc2.", mult, lambda u: feed_forward(norm_around_zero(u, w[p + "norm2"], eps), w, p + "mlp.", layer["mlp"]))
+            streams = connect(streams, w, p + "hc2.", mult, lambda u: feed_forward(norm_around_zero(u, w[p + "norm2"], eps), w, p + "mlp.", layer["mlp"], margins))
         if after_layers is not None:
             after_layers.append(streams.sum(0))
     return norm_around_zero(streams.sum(0), w["final.norm"], eps) @ w["head"].T
