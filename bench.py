@@ -494,6 +494,35 @@ def sezopel_config(sz: dict) -> dict:
             "token_side": {"dim": 256}, "logit_softcap": 30.0, "layers": layers}
 
 
+def muzulorn_config(sz: dict) -> dict:
+    """Muzulorn at one size: the same width, depth and vocabulary, four streams, rows by pairs of tokens; layers go round attention with keys and
+    values of its own (an eighth of the heads as kv heads, scores capped, a bias by distance up to 128), a state-space layer (twice
+    the width in heads of 64 channels, states of 128 rows, one group, four taps), latent attention with Kidolorn's cached row (a
+    latent of 96 and a rotated part of 32 at these sizes) over a window of 1,024 tokens, queries through a latent of half the width,
+    and attention that reads the first one's cache.  The attention layers have Sezopel's two-matrix feed-forward, the others Nutopel's mixture:
+    eight experts of a quarter of the dense size, two of them used, beside a shared one of half the dense size."""
+    W, H, D = sz["width"], sz["heads"], sz["dim"]
+    rot, rank = D // 4, sz["kv_rank"] - D // 4
+    dense = {"kind": "dense", "ff": sz["ff"] * 3 // 2 // 64 * 64}
+    moe = {"kind": "moe", "expert": {"ff": sz["ff"] // 4 // 64 * 64}, "shared": {"ff": sz["ff"] // 2 // 64 * 64}, "router": {"experts": 8, "top": 2}}
+    attention = {"heads": H, "kv_heads": max(1, H // 8), "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 30.0, "bias_max": 128,
+                 "q_temp": {"coef": 0.1, "every": 1024}}
+    ssm = {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    latent = {"heads": H, "dim": D - rot, "rot_dim": rot, "vdim": D, "q_rank": W // 2, "kv_rank": rank, "scale": D ** -0.5,
+              "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": rot}}
+    layers = []
+    for i in range(sz["layers"]):
+        kind = i % 4
+        if kind == 1:
+            layers.append({"type": "mamba2", "mixer": ssm, "mlp": moe})
+        elif kind == 2:
+            layers.append({"type": "latent_attention", "mixer": latent, "mlp": moe})
+        else:
+            layers.append({"type": "attention", "mixer": dict(attention, kv_from=i - 3) if kind else attention, "mlp": dense})
+    return {"architecture": "Muzulorn", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "streams": 4, "residual_mult": 0.5,
+            "embedding": {"bigram": {"buckets": 65536, "mul_prev": 31, "mul_cur": 17}}, "layers": layers}
+
+
 def design_run(args) -> dict:
     global PREFILL_TOKENS
     import torch
@@ -517,6 +546,9 @@ def design_run(args) -> dict:
         if args.workload == "sezopel":
             # beside Kidolorn (fixed-decay linear attention, norms behind the sublayers) and Qwen2 (grouped-query attention)
             designs = [("sezopel", sezopel_config(sz)), ("kidolorn", kidolorn_config(sz)), designs[-1]]
+        if args.workload == "muzulorn":
+            # beside Kidolorn (latent attention, experts, recurrences) and Sezopel (capped attention on its own or a borrowed cache, chunked retention)
+            designs = [("muzulorn", muzulorn_config(sz)), ("kidolorn", kidolorn_config(sz)), ("sezopel", sezopel_config(sz))]
         for which, config in designs:
             model, _ = build_random_model(config, seed=0, dtype="bfloat16", device="cuda:0", std=0.02)
             cfg = {"vocab_size": sz["vocab"]}
@@ -791,7 +823,7 @@ def base_config(cfg, args, prompt_len) -> dict:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", choices=("decode", "rososun", "nutopel", "kidolorn", "gerupel", "sezopel") + tuple(SERVING), default="decode",
+    ap.add_argument("--workload", choices=("decode", "rososun", "nutopel", "kidolorn", "gerupel", "sezopel", "muzulorn") + tuple(SERVING), default="decode",
                     help="decode: the default run; serve-*: the baseline's serving workloads through LLM.generate")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=32)
@@ -830,7 +862,7 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         print(json.dumps({"error": "no CUDA device"}))
         return 1
-    if args.workload in ("rososun", "nutopel", "kidolorn", "gerupel", "sezopel"):
+    if args.workload in ("rososun", "nutopel", "kidolorn", "gerupel", "sezopel", "muzulorn"):
         print(json.dumps(design_run(args)))
         return 0
     if args.workload != "decode":

@@ -69,6 +69,7 @@ struct AttnTcParams {
   const int* tile_row0;          // [tiles]
   int* status;
   int max_pages, page_size, nq, nkv;
+  int window;                    // > 0: a query sees its own key and the window - 1 before it (num_splits == 1 then)
   int page_runs;                 // the run maps are valid: a key tile whose pages have consecutive ids is one box of K and one of V
   float scale_log2;              // scale * log2(e)
   // the context cut in num_splits ranges of tiles_per_split key tiles each (grid z); with more than one,
@@ -217,7 +218,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
   // per row tile t: its keys end at key_end[t] (exclusive), in n_of[t] key tiles; later rows see more keys
   // This CTA's range of the context: key tiles [tile0, tile0 + tiles_per_split).  Key tile j below is
   // the range's j-th, key tile tile0 + j of the request.
-  const int tile0 = (int)blockIdx.z * p.tiles_per_split;
+  // With a window the walk begins at the key tile the first row's window begins in (every later row's begins there or further on).
+  const int tile_first = p.window > 0 ? max(0, pos0 + row0 / G - p.window + 1) / TC_BN : 0;
+  const int tile0 = tile_first + (int)blockIdx.z * p.tiles_per_split;
   int key_end[RT], n_of[RT];
 #pragma unroll
   for (int t = 0; t < RT; ++t) {
@@ -252,11 +255,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           tma_load_5d(dst, which ? &run_v : &run_k, 0, 0, bt[first_pi], 0, kvh, full);
           return;
         }
-        mbar_expect_tx(full, (uint32_t)(pages * HALVES * ps * 128));
+        // (a page that a window gave back holds no key any row of the tile sees: what an earlier tile left in its place stays)
+        int held = 0;
+        for (int i = 0; i < pages; ++i) held += first_pi + i < max_pages && bt[first_pi + i] >= 0;
+        mbar_expect_tx(full, (uint32_t)(held * HALVES * ps * 128));
         for (int i = 0; i < pages; ++i) {
-          const int pi = first_pi + i;
-          int page = pi < max_pages ? bt[pi] : 0;
-          if (page < 0) page = 0;                   // no page lies inside a causal range without a window
+          const int pi = first_pi + i, page = pi < max_pages ? bt[pi] : -1;
+          if (page < 0) continue;
           const int y = (page * p.nkv + kvh) * ps;
 #pragma unroll
           for (int h = 0; h < HALVES; ++h)
@@ -401,7 +406,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     const int row = row0 + t * TC_BM + r;
     const bool valid = row < rows_total;
     const int my_tiles = RT == 1 ? n_of[0] : (t == 0 ? n_of[0] : n_of[RT - 1]);
-    const int hi = valid ? pos0 + row / G + 1 : 0;                     // keys [0, hi) are this row's
+    const int hi = valid ? pos0 + row / G + 1 : 0;                     // keys [lo, hi) are this row's
+    const int lo = p.window > 0 ? hi - p.window : 0;
     const uint32_t t_lane = tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + t * L::TMEM_TILE;
     uint64_t* my_s_full = s_full + t * 2;
     uint64_t* my_p_full = p_full + t * 2;
@@ -448,14 +454,14 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       // the scale is positive, so the maximum of the scaled scores is the scaled maximum: the
       // scaling itself is folded into the exponent's multiply-add below
       float mx = -INFINITY;
-      if (__all_sync(0xffffffffu, kbase + TC_BN <= hi)) {
+      if (__all_sync(0xffffffffu, kbase + TC_BN <= hi && kbase >= lo)) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) mx = max3(mx, __uint_as_float(s0[i]), __uint_as_float(s1[i]));
       } else {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (kbase + i >= hi) s0[i] = 0xff800000u;          // -inf
-          if (kbase + 32 + i >= hi) s1[i] = 0xff800000u;
+          if (kbase + i >= hi || kbase + i < lo) s0[i] = 0xff800000u;          // -inf
+          if (kbase + 32 + i >= hi || kbase + 32 + i < lo) s1[i] = 0xff800000u;
           mx = max3(mx, __uint_as_float(s0[i]), __uint_as_float(s1[i]));
         }
       }
@@ -497,7 +503,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       float2 sums = make_float2(0.f, 0.f);                  // of the even and of the odd keys
       if constexpr (CAP) {
         // 2^(capped score - max) = 2^(cap - max - 2 cap / (2^(slope s) + 1)); the two reciprocals of a pair come from one
-        const bool edge = kbase + TC_BN > hi;
+        const bool edge = kbase + TC_BN > hi || kbase < lo;
+        auto unseen = [&](int key) { return edge && (key >= hi || key < lo); };
         const float top = p.cap_log2 + neg_m, two_cap = -2.0f * p.cap_log2;
         auto capped_pair = [&](uint32_t sa, uint32_t sb, int key) {
           const float2 z = fma_x2(__uint_as_float(sa), __uint_as_float(sb), p.cap_slope, 0.f);
@@ -506,7 +513,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           const float rr = __fdividef(1.0f, d.x * d.y);
           float2 x = fma_x2(d.y * rr, d.x * rr, two_cap, top);
           if (REL && !far) x = add_x2(x, make_float2(near_bias(key), near_bias(key + 1)));
-          return make_float2(edge && key >= hi ? 0.f : ex2(x.x), edge && key + 1 >= hi ? 0.f : ex2(x.y));
+          return make_float2(unseen(key) ? 0.f : ex2(x.x), unseen(key + 1) ? 0.f : ex2(x.y));
         };
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
@@ -681,7 +688,7 @@ SLLM_EXPORT int sllm_attention_tc_supports(int hd, int page_size) {
 }
 
 // The prefill form: tiles of up to 128 * row_tiles (token, head-in-group) rows (row_tiles 1 or 2; tile_row0
-// in steps of that many rows), no window.  num_splits > 1 cuts the context into that many ranges of
+// in steps of that many rows).  num_splits > 1 cuts the context into that many ranges of
 // tiles_per_split 64-key tiles (num_splits * tiles_per_split must cover the longest context), each range a
 // CTA of its own; part_o [num_splits, total_tokens, nq, hd] and part_lse [num_splits, total_tokens, nq]
 // float32 are the scratch the ranges' results pass through; part_lse must be -inf everywhere before the
@@ -691,7 +698,7 @@ SLLM_EXPORT int sllm_attention_tc_supports(int hd, int page_size) {
 SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void* v_cache, long long num_pages, void* out,
                                   const int* block_tables, int max_pages, const int* q_start, const int* ctx_len,
                                   const int* tile_seq, const int* tile_row0, int tiles, int row_tiles, int nq, int nkv,
-                                  int hd, int page_size, float scale, int num_splits, int tiles_per_split, int total_tokens,
+                                  int hd, int page_size, float scale, int window, int num_splits, int tiles_per_split, int total_tokens,
                                   float* part_o, float* part_lse, const int* seq_row, const int* page_shift, const float* sink,
                                   float softcap, const float* gate, int gate_ld, const float* rel, int rel_n, const float* rel_top,
                                   int* status, cudaStream_t stream) {
@@ -709,6 +716,7 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
   SLLM_REQUIRE(scale > 0.f, "attention_tc: the score scale must be positive (the row maximum is taken before scaling)");
   SLLM_REQUIRE(((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0 && ((uintptr_t)q & 15) == 0 &&
                    ((uintptr_t)out & 15) == 0, "attention_tc: operands must be 16-byte aligned");
+  SLLM_REQUIRE(window >= 0 && (window == 0 || (num_splits == 1 && seq_row == nullptr)), "attention_tc: a window goes with whole requests and an uncut context");
   if (tiles == 0) return SLLM_OK;
   CUtensorMap mk, mv;
   const long long rows = num_pages * nkv * page_size;
@@ -725,7 +733,7 @@ SLLM_EXPORT int sllm_attention_tc(const void* q, const void* k_cache, const void
   p.ctx_len = ctx_len; p.tile_seq = tile_seq; p.tile_row0 = tile_row0; p.status = status; p.max_pages = max_pages;
   p.page_size = page_size; p.nq = nq; p.nkv = nkv; p.scale_log2 = scale * 1.4426950408889634f;
   p.num_splits = num_splits; p.tiles_per_split = num_splits == 1 ? (1 << 30) / TC_BN : tiles_per_split;
-  p.total_tokens = total_tokens; p.part_o = part_o; p.part_lse = part_lse; p.seq_row = seq_row; p.page_shift = page_shift;
+  p.total_tokens = total_tokens; p.part_o = part_o; p.part_lse = part_lse; p.window = window; p.seq_row = seq_row; p.page_shift = page_shift;
   p.sink = sink;
   p.cap_log2 = softcap * 1.4426950408889634f; p.cap_slope = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
   p.gate = gate; p.gate_ld = gate_ld; p.rel = rel; p.rel_n = rel_n; p.rel_top = rel_top;

@@ -85,6 +85,9 @@ def build_random_model(config: dict, seed: int, dtype="bfloat16", device="cuda:0
             if gain_std:
                 t += gain_std * torch.randn(shape, generator=gen, device=device)
             return t
+        if s.role in ("identity", "share"):
+            t = torch.eye(*shape, device=device) if s.role == "identity" else torch.full(shape, 1.0 / shape[0], device=device)
+            return t + std * torch.randn(shape, generator=gen, device=device)
         if s.role == "mix":
             return torch.empty(shape, dtype=torch.float32, device=device).uniform_(0.05, 0.95, generator=gen)
         t = torch.empty(shape, dtype=dt if s.role != "bias" else torch.float32, device=device)

@@ -1817,8 +1817,8 @@ def choose_tc_splits(num_tiles: int, nkv: int, max_ctx: int) -> tuple[int, int]:
 
 
 def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq, nkv, hd, scale, out=None,
-                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, sink=None, softcap: float = 0.0, gate=None, rel=None):
-    """The prefill form on tcgen05 (tiles of 128 * row_tiles rows, row_tiles 1 or 2; no window; see
+                 row_tiles: int = 1, splits: tuple[int, int] = (1, 0), parts=None, window=None, sink=None, softcap: float = 0.0, gate=None, rel=None):
+    """The prefill form on tcgen05 (tiles of 128 * row_tiles rows, row_tiles 1 or 2; see
     `attention_tiles`).  ``splits`` = (ranges, 64-key tiles a range) cuts the context into ranges
     that run as CTAs of their own and are merged afterwards; ranges x tiles must cover the longest
     context among the tiles' requests.  ``parts`` = (row of ``block_tables``, first page) per sequence of ``q_start`` /
@@ -1837,7 +1837,7 @@ def attention_tc(q, k_cache, v_cache, block_tables, q_start, ctx_len, tiles, nq,
         launches["library"] += 1           # the fill
     call("sllm_attention_tc", _p(q), _p(k_cache), _p(v_cache), k_cache.shape[0], _p(out), _p(block_tables),
          block_tables.shape[1], _p(q_start), _p(ctx_len), _p(tiles[0]), _p(tiles[1]), tiles[2], int(row_tiles), nq, nkv,
-         hd, k_cache.shape[2], float(scale), n_splits, max(per, 1), T, _p(part_o), _p(part_lse),
+         hd, k_cache.shape[2], float(scale), int(window or 0), n_splits, max(per, 1), T, _p(part_o), _p(part_lse),
          _p(parts[0]) if parts else None, _p(parts[1]) if parts else None, _p(sink), float(softcap or 0.0), *_gate_args(gate),
          *(rel.args() if rel else _NO_REL), _p(_status_word(q.device)), _stream())
     if n_splits > 1:
@@ -1891,12 +1891,10 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     each head's softmax denominator (every form takes it).  ``softcap`` > 0: a score becomes softcap tanh(score / softcap) before
     the softmax; ``gate`` = (float32 product, column): head h's output times sigmoid of column + h; ``rel``: a bias on the scores by distance, added after scale and
     cap (every form takes all three).  ``window``: only the last ``window`` keys;
-    ``block``: only the keys of the query's own block of ``block`` positions, counted from the sequence's start (both
-    run on the mma.sync and TMA-fed forms, not on tcgen05).  bfloat16 with a head size
+    ``block``: only the keys of the query's own block of ``block`` positions, counted from the sequence's start.  bfloat16 with a head size
     the tensor-core kernels take: requests of at most 16 (token, head-in-group) rows go to the decode
     form (fed by TMA where the head and page sizes allow, split over the context), the others to the
-    prefill form in 128-row tiles (on tcgen05 where there is no window and the sizes allow, else on
-    mma.sync).  Otherwise the CUDA-core kernel."""
+    prefill form in 128-row tiles (on tcgen05 where the sizes allow, else on mma.sync).  Otherwise the CUDA-core kernel."""
     g = step.groups[group]
     if q.dtype != torch.bfloat16 or not mma_supports(hd):
         return attention_simt(q, k_cache, v_cache, g.block_tables, step.positions, step.seq_of_token,
@@ -1904,9 +1902,9 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
     G = nq // nkv
     # blocks that start on page borders: the prefill form runs each block's part of a portion as a causal sequence of its own
     blocked_tc = bool(block) and block % k_cache.shape[2] == 0 and bool(step.ctx_lens)
-    use_tc = not window and (not block or blocked_tc) and _TC_ATTENTION and tc_attention_supports(hd, k_cache.shape[2]) and \
+    use_tc = (not block or (blocked_tc and not window)) and _TC_ATTENTION and tc_attention_supports(hd, k_cache.shape[2]) and \
         (rel is None or (rel.narrow and not block))
-    key = ("mma", G, nkv, use_tc, block or 0)
+    key = ("mma", G, nkv, use_tc, block or 0, bool(window))
     if key not in step.attn_tiles:
         # 128-row CTAs, two per SM.  (The kernel also has a form with two row tiles a CTA, one CTA per SM,
         # that fetches each key/value tile once for 256 rows; measured at 28/4 heads of 128 it is the
@@ -1922,7 +1920,7 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
             small_ctx = max((c for c, n in zip(step.ctx_lens, step.q_lens) if n * G <= 16), default=step.max_ctx_len) \
                 if step.ctx_lens else step.max_ctx_len
             splits = choose_splits(small[2], nkv, small_ctx, per_sm, 0 if tma else MMA_MAX_SPLITS)
-        tc_splits = choose_tc_splits(large[2], nkv, step.max_ctx_len) if (large and use_tc and not block) else (1, 0)
+        tc_splits = choose_tc_splits(large[2], nkv, step.max_ctx_len) if (large and use_tc and not block and not window) else (1, 0)
         parts = block_parts(step.q_lens, step.ctx_lens, G, block, k_cache.shape[2], q.device, rows) if (large and use_tc and block) else None
         step.attn_tiles[key] = (small, large, splits, rows, tc_splits, parts)
     small, large, splits, rows, tc_splits, parts = step.attn_tiles[key]
@@ -1938,7 +1936,7 @@ def paged_attention(q, k_cache, v_cache, step, group: int, nq, nkv, hd, scale, w
                      row_tiles=rows // 128, parts=parts[2], sink=sink, softcap=softcap, gate=gate)
     elif large and use_tc:
         attention_tc(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, nq, nkv, hd, scale, out,
-                     row_tiles=rows // 128, splits=tc_splits, sink=sink, softcap=softcap, gate=gate, rel=rel)
+                     row_tiles=rows // 128, splits=tc_splits, window=window, sink=sink, softcap=softcap, gate=gate, rel=rel)
     elif large:
         attention_mma(q, k_cache, v_cache, g.block_tables, step.q_start, step.ctx_len, large, False, 1,
                       nq, nkv, hd, scale, window, out, block, sink, softcap, gate, rel)

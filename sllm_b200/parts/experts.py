@@ -146,9 +146,9 @@ class GatedExperts(FeedForward):
             router = torch.cat([router, fetch("shared.sg")], dim=0)
         if self.router_bias or self.shared_ff:
             pad = -router.shape[0] % 16
-            router = torch.cat([router, torch.zeros((pad, W), dtype=router.dtype)], dim=0)
+            router = torch.cat([router, torch.zeros((pad, W), dtype=router.dtype, device=router.device)], dim=0)
             if self.router_bias:
-                bias = torch.zeros(router.shape[0], dtype=torch.float32)
+                bias = torch.zeros(router.shape[0], dtype=torch.float32, device=router.device)
                 bias[:self.E] = fetch("router.b").float()
                 bias = self._f32(bias)
         self.router = Linear(self._matrix(router), bias)

@@ -429,8 +429,8 @@ def test_attention_and_a_second_layer_on_the_same_keys_and_values(dev, H, G, dk,
     (5, 12, 0, 8, 16, 16, 7, 0, 16, "float32"), (4, 128, 64, 128, 128, 512, 50, 64, 16, "bfloat16"), (3, 16, 8, 24, 40, 40, None, 6, 8, "float32")])
 def test_latent_attention_in_a_window(dev, H, dk, dr, dv, q_rank, rank, window, dims, ps, dtype):
     """Queries through a latent of their own, pairs of neighbouring channels rotated (all, part or none of the shared key part), a window whose edge
-    single tokens and portions meet at every place in a page, a sink, a gate per channel.  Pages the window has passed are poisoned.  The
-    key just inside the window and the one just outside are made to stand out for some tokens, so an edge that is off by one shows."""
+    single tokens and portions meet at every place in a page, a sink, a gate per channel.  Pages the window has passed are poisoned.  Scores are
+    several units wide, so that for some tokens the key at the window's edge takes most of the weight and an edge that is off by one shows."""
     from sllm_b200.config.plan import PartSpec
     from sllm_b200.parts import MIXERS, GroupView, LayerCache
     if dev == "cpu" and dtype != "float32":
@@ -456,7 +456,7 @@ def test_latent_attention_in_a_window(dev, H, dk, dr, dv, q_rank, rank, window, 
     if window is not None and window > 1:           # the edge matters here: one key more or less changes rows by more than the tolerance
         for other in (window - 1, window + 1):
             d = _relative(plain.latent_attention(xs[0], w, "m.", dict(m, mask={"size": other}), eps), want[0])
-            assert np.quantile(d[window + 1:], 0.9) > 0.05
+            assert np.quantile(d[window + 1:], 0.95) > 0.03 and d.max() > 0.2
     D = need.head_dim
     _, _, tables, _ = _paged(dev, 1, D, ps, list(lens.values()), rng)
     kc = torch.full((int(tables.max()) + 1, 1, ps, D), 3.0, dtype=td, device=dev)
@@ -480,6 +480,45 @@ def test_latent_attention_in_a_window(dev, H, dk, dr, dv, q_rank, rank, window, 
         else:
             e = _relative(got[s], want[s])
             assert e.max() < 0.08 and np.quantile(e, 0.9) < 0.03, (s, float(e.max()), int(e.argmax()))
+
+
+@pytest.mark.parametrize("D,ps,dtype,nq,nkv,window", [
+    (27, 4, "float32", 3, 1, 10), (64, 16, "bfloat16", 8, 2, 100), (64, 16, "bfloat16", 24, 1, 64), (128, 32, "bfloat16", 6, 3, 33), (32, 8, "bfloat16", 2, 2, 21),
+    (128, 16, "bfloat16", 16, 1, 130), (64, 8, "bfloat16", 4, 4, 1), (160, 16, "bfloat16", 6, 1, 50), (128, 64, "bfloat16", 5, 1, 17)])
+def test_window_with_a_sink_over_every_form(dev, D, ps, dtype, nq, nkv, window):
+    """Single tokens and portions in one step, hundreds of tokens into a request; pages the window has passed are given back and poisoned.  For every
+    query the key at the window's edge, the one just outside, or its own stands out in its first head."""
+    import sllm_b200.ops as ops
+    if dev == "cpu" and dtype != "float32":
+        pytest.skip("the stand-ins are float32")
+    rng = np.random.default_rng(D + nq + window)
+    scale = 0.3
+    cases = [(1, 1), (1, 2), (1, 700), (1, 3 * ps + 1), (2, 2), (5, 5), (2, 2 * ps + 1), (ps + 3, 4 * ps + 2), (3, 333), (150, 150), (130, 400), (40, 640), (1, window), (1, window + 1)]
+    q_lens, ctx = [c[0] for c in cases], [c[1] for c in cases]
+    k, v, tables, g = _paged(dev, nkv, D, ps, ctx, rng)
+    T = sum(q_lens)
+    q = rng.standard_normal((T, nq, D)).astype(np.float32)
+    full = tables.copy()
+    for s, (n, c) in enumerate(cases):
+        gone = max(0, c - n - window + 1) // ps
+        k[tables[s, :gone]] = v[tables[s, :gone]] = np.nan
+        tables[s, :gone] = -1
+    g.block_tables.copy_(torch.from_numpy(tables))
+    step = _step(dev, q_lens, list(range(len(cases))), ctx, g)
+    pos, seq = step.positions.cpu().numpy(), step.seq_of_token.cpu().numpy()
+    for t in range(T):
+        j = (max(pos[t] - window + 1, 0), max(pos[t] - window, 0), pos[t])[t % 3]
+        if tables[seq[t], j // ps] >= 0:
+            k[tables[seq[t], j // ps], 0, j % ps] = q[t, 0] * (12.0 / np.sqrt(D))
+    sink = rng.standard_normal(nq) * 2
+    td = torch.float32 if dtype == "float32" else torch.bfloat16
+    qd, kd, vd = (torch.from_numpy(a).to(dev).to(td).contiguous() for a in (q.reshape(T, nq * D), k, v))
+    got = ops.paged_attention(qd, kd, vd, step, 0, nq, nkv, D, scale, window, sink=_to(dev)(sink)).float().cpu().numpy().reshape(T, nq, D)
+    qf, kf, vf = (a.float().cpu().numpy().astype(np.float64) for a in (qd, kd, vd))
+    tol = 3e-5 if dtype == "float32" else 3e-2
+    for t in range(T):
+        want = _attend(kf, vf, full, seq[t], pos[t], qf.reshape(T, nq, D)[t], ps, nq, nkv, scale, 0.0, None, window, sink)
+        np.testing.assert_allclose(got[t], want, rtol=tol, atol=tol, err_msg=f"token {t} (position {pos[t]})")
 
 
 def _state_space_case(rng, dev, H, dv, N, G, taps, parts, W=40, eps=1e-2):
@@ -821,6 +860,20 @@ def test_command_line_with_random_weights(tmp_path, capsys, dev, monkeypatch):
                      "--dtype", "float32", "--log-level", "ERROR"]) == 0
     got = [int(t) for t in capsys.readouterr().out.strip().split(",")]
     assert len(got) == 5 and all(0 <= t < 260 for t in got)
+
+
+@pytest.mark.gpu
+def test_weights_drawn_on_the_device():
+    """A model without a folder (`build_random_model`, what the benchmarks use), a prompt and decode steps through it."""
+    from sllm_b200.engine import Engine, StepEntry, build_random_model
+    if not torch.cuda.is_available():
+        pytest.skip("no CUDA device")
+    for config in (MID, ODD):
+        model, _ = build_random_model(config, seed=1, dtype="bfloat16", device="cuda:0")
+        eng = Engine(model, page_size=16, num_pages=16, max_requests=2)
+        ids = _requests(config["vocab"], (150,))["r0"]
+        out = [eng.step([StepEntry("a", ids[:140], [139])])] + [eng.step([StepEntry("a", ids[p:p + 1], [0])]) for p in range(140, 150)]
+        assert all(bool(torch.isfinite(o).all()) for o in out)
 
 
 @pytest.mark.gpu
