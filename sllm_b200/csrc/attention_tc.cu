@@ -48,6 +48,7 @@
 #include <stdio.h>
 
 #include <mutex>
+#include <type_traits>
 #include <unordered_map>
 
 #include "tcgen05.cuh"
@@ -432,12 +433,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       if (lane == 0) mbar_arrive(&q_full[t]);
     }
     // REL: the row's place in the bias table (rows of G; neighbouring rows of a tile read neighbouring numbers), its last and largest bias
-    const float* rel_h = nullptr;
+    int rel_row = 0;
     const int rel_pos = pos0 + row / G;
     float rel_far = 0.f, rel_top = 0.f;
     if constexpr (REL) {
-      rel_h = p.rel + (size_t)kvh * p.rel_n * G + row % G;
-      rel_far = __ldg(rel_h + (size_t)(p.rel_n - 1) * G) * 1.4426950408889634f;
+      rel_row = kvh * p.rel_n * G + row % G;
+      rel_far = __ldg(p.rel + rel_row + (p.rel_n - 1) * G) * 1.4426950408889634f;
       rel_top = __ldg(p.rel_top + kvh * G + row % G) * 1.4426950408889634f;
     }
     float m_used = -INFINITY, l = 0.f;                                 // the maximum in scaled (log2) units
@@ -454,7 +455,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
       // the scale is positive, so the maximum of the scaled scores is the scaled maximum: the
       // scaling itself is folded into the exponent's multiply-add below
       float mx = -INFINITY;
-      if (__all_sync(0xffffffffu, kbase + TC_BN <= hi && kbase >= lo)) {
+      const bool inside = __all_sync(0xffffffffu, kbase + TC_BN <= hi && kbase >= lo);
+      if (inside) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) mx = max3(mx, __uint_as_float(s0[i]), __uint_as_float(s1[i]));
       } else {
@@ -497,46 +499,56 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      const float neg_m = (m_used == -INFINITY ? 0.f : -m_used) + (far ? rel_far : 0.f);
-      auto near_bias = [&](int key) { return __ldg(rel_h + (size_t)min(max(rel_pos - key, 0), p.rel_n - 1) * G) * 1.4426950408889634f; };
+      float neg_m = (m_used == -INFINITY ? 0.f : -m_used) + (far ? rel_far : 0.f);
       uint32_t pk[32];                                      // column i: keys 2i (low half) and 2i+1
       float2 sums = make_float2(0.f, 0.f);                  // of the even and of the odd keys
-      if constexpr (CAP) {
-        // 2^(capped score - max) = 2^(cap - max - 2 cap / (2^(slope s) + 1)); the two reciprocals of a pair come from one
-        const bool edge = kbase + TC_BN > hi || kbase < lo;
-        auto unseen = [&](int key) { return edge && (key >= hi || key < lo); };
-        const float top = p.cap_log2 + neg_m, two_cap = -2.0f * p.cap_log2;
-        auto capped_pair = [&](uint32_t sa, uint32_t sb, int key) {
-          const float2 z = fma_x2(__uint_as_float(sa), __uint_as_float(sb), p.cap_slope, 0.f);
-          // (beyond 2^60 the quotient is nothing; the bound keeps the product of the two finite)
-          const float2 d = add_x2(make_float2(ex2(fminf(z.x, 60.f)), ex2(fminf(z.y, 60.f))), make_float2(1.f, 1.f));
-          const float rr = __fdividef(1.0f, d.x * d.y);
-          float2 x = fma_x2(d.y * rr, d.x * rr, two_cap, top);
-          if (REL && !far) x = add_x2(x, make_float2(near_bias(key), near_bias(key + 1)));
-          return make_float2(unseen(key) ? 0.f : ex2(x.x), unseen(key + 1) ? 0.f : ex2(x.y));
+      // The walk over the row's keys comes in up to three copies, chosen for the whole warp, so that the tiles in the middle of a
+      // context pay for neither masks nor the bias table.  MASKED: some key of the tile is not this warp's to see (its score is -inf
+      // already; capped it would not be); NEAR: the bias is read key by key.
+      auto walk = [&](auto masked, auto near_keys) {
+        constexpr bool MASKED = decltype(masked)::value, NEAR = decltype(near_keys)::value;
+        const int d0 = rel_pos - kbase;
+        auto biased = [&](float2 x, int key) {
+          if constexpr (NEAR) {
+            x.x = fmaf(__ldg(p.rel + (rel_row + __viaddmin_s32_relu(d0, -key, p.rel_n - 1) * G)), 1.4426950408889634f, x.x);
+            x.y = fmaf(__ldg(p.rel + (rel_row + __viaddmin_s32_relu(d0, -key - 1, p.rel_n - 1) * G)), 1.4426950408889634f, x.y);
+          }
+          return x;
+        };
+        // 2^(score - max) of keys `key` and `key + 1` of the tile
+        auto pair = [&](uint32_t sa, uint32_t sb, int key) {
+          if constexpr (CAP) {
+            // 2^(capped score - max) = 2^(cap - max - 2 cap / (2^(slope s) + 1)); the two reciprocals of a pair come from one
+            const float2 z = fma_x2(__uint_as_float(sa), __uint_as_float(sb), p.cap_slope, 0.f);
+            // (beyond 2^60 the quotient is nothing; the bound keeps the product of the two finite)
+            const float2 d = add_x2(make_float2(ex2(fminf(z.x, 60.f)), ex2(fminf(z.y, 60.f))), make_float2(1.f, 1.f));
+            const float rr = __fdividef(1.0f, d.x * d.y);
+            const float2 x = biased(fma_x2(d.y * rr, d.x * rr, -2.0f * p.cap_log2, p.cap_log2 + neg_m), key);
+            return make_float2(MASKED && sa == 0xff800000u ? 0.f : ex2(x.x), MASKED && sb == 0xff800000u ? 0.f : ex2(x.y));
+          } else {
+            const float2 x = biased(fma_x2(__uint_as_float(sa), __uint_as_float(sb), p.scale_log2, neg_m), key);
+            return make_float2(ex2(x.x), ex2(x.y));
+          }
         };
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float2 e01 = capped_pair(s0[2 * i], s0[2 * i + 1], kbase + 2 * i), e23 = capped_pair(s1[2 * i], s1[2 * i + 1], kbase + 32 + 2 * i);
+          const float2 e01 = pair(s0[2 * i], s0[2 * i + 1], 2 * i), e23 = pair(s1[2 * i], s1[2 * i + 1], 32 + 2 * i);
           sums = add_x2(sums, add_x2(e01, e23));
           pk[i] = pack2(e01.x, e01.y);
           pk[16 + i] = pack2(e23.x, e23.y);
         }
+      };
+      using Yes = std::true_type;
+      using No = std::false_type;
+      if constexpr (REL) {
+        if (far && inside) walk(No{}, No{});
+        else if (inside) walk(No{}, Yes{});
+        else { neg_m = m_used == -INFINITY ? 0.f : -m_used; walk(Yes{}, Yes{}); }      // (the table holds the far bias too)
+      } else if constexpr (CAP) {
+        if (inside) walk(No{}, No{});
+        else walk(Yes{}, No{});
       } else {
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        float2 x01 = fma_x2(__uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]), p.scale_log2, neg_m);
-        float2 x23 = fma_x2(__uint_as_float(s1[2 * i]), __uint_as_float(s1[2 * i + 1]), p.scale_log2, neg_m);
-        if (REL && !far) {
-          const int key = kbase + 2 * i;
-          x01 = add_x2(x01, make_float2(near_bias(key), near_bias(key + 1)));
-          x23 = add_x2(x23, make_float2(near_bias(key + 32), near_bias(key + 33)));
-        }
-        const float2 e01 = make_float2(ex2(x01.x), ex2(x01.y)), e23 = make_float2(ex2(x23.x), ex2(x23.y));
-        sums = add_x2(sums, add_x2(e01, e23));
-        pk[i] = pack2(e01.x, e01.y);
-        pk[16 + i] = pack2(e23.x, e23.y);
-      }
+        walk(No{}, No{});                                    // (a score of -inf gives zero by itself)
       }
       l += sums.x + sums.y;
       tmem_st32(t_lane + b * TC_BN, pk);

@@ -18,12 +18,19 @@ namespace sllm {
 constexpr int HC_THREADS = 256;
 constexpr int HC_MAX_STREAMS = 16;
 
+__device__ __forceinline__ float4 load4_of(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4_of(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(HC_THREADS)
 embed_streams_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out, int H, int V, float scale, int copies,
                      const T* __restrict__ pair_table, unsigned long long buckets, unsigned long long mul_prev, unsigned long long mul_cur,
                      const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ q_start,
-                     const int* __restrict__ state_slots, float* __restrict__ before) {
+                     const int* __restrict__ state_slots, float* __restrict__ before, int vec) {
   __shared__ int prev_s;
   pdl_launch_dependents();
   pdl_wait();
@@ -47,6 +54,18 @@ embed_streams_kernel(const T* __restrict__ table, const int* __restrict__ ids, f
   }
   const T* src = table + (size_t)id * H;
   float* dst = out + (size_t)t * copies * H;
+  if (vec) {                                      // rows in whole pieces of four channels
+    for (int i = threadIdx.x * 4; i < H; i += HC_THREADS * 4) {
+      float4 v = load4_of(src + i);
+      v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+      if (pair != nullptr) {
+        const float4 q = load4_of(pair + i);
+        v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+      }
+      for (int c = 0; c < copies; ++c) *reinterpret_cast<float4*>(dst + (size_t)c * H + i) = v;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += HC_THREADS) {
     float v = to_f32(src[i]) * scale;
     if (pair != nullptr) v += to_f32(pair[i]);
@@ -208,10 +227,11 @@ SLLM_EXPORT int sllm_embed_streams(const void* table, int dtype, const int* ids,
   SLLM_REQUIRE(pair_table == nullptr || (buckets >= 1 && mul_prev >= 0 && mul_cur >= 0 && positions && seq_of_token && q_start && state_slots && before),
                "embed_streams: pairs of tokens need their buckets, the batch's description and the tokens before");
   if (T == 0) return SLLM_OK;
+  const int vec = H % 4 == 0 && (((uintptr_t)table | (uintptr_t)pair_table | (uintptr_t)out) & 15) == 0;
 #define ES(T_)                                                                                                                      \
   launch_kernel(embed_streams_kernel<T_>, (unsigned)T, HC_THREADS, 0, stream, (const T_*)table, ids, out, H, V, scale, copies,       \
                 (const T_*)pair_table, (unsigned long long)buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, positions, \
-                seq_of_token, q_start, state_slots, before)
+                seq_of_token, q_start, state_slots, before, vec)
   if (dtype == SLLM_F32) ES(float);
   else if (dtype == SLLM_BF16) ES(__nv_bfloat16);
   else SLLM_REQUIRE(false, "embed_streams: unknown dtype %d", dtype);

@@ -79,24 +79,67 @@ qk_norm_rope_kv_write_kernel(const float* __restrict__ qkv, int ld, const float*
   for (int d = rot + lane; d < D; d += 32) dst[d] = from_f32<TC>(d < dim ? x[d] * inv * (gain ? gain[d] : 1.f) : 0.f);
 }
 
+// VEC (1 or 4) consecutive channels at a time
+template <int VEC> struct WnVec { float v[VEC]; };
+template <int VEC> __device__ __forceinline__ WnVec<VEC> wn_load(const float* p) {
+  WnVec<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
+  } else {
+    r.v[0] = *p;
+  }
+  return r;
+}
+template <int VEC, typename T> __device__ __forceinline__ void wn_store(T* p, const WnVec<VEC>& r) {
+  if constexpr (VEC == 4 && sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  } else if constexpr (VEC == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(r.v[0], r.v[1]), b = __floats2bfloat162_rn(r.v[2], r.v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
+  } else {
+    *p = from_f32<T>(r.v[0]);
+  }
+}
+
 // A CTA per token; the token's queries and keys (sums of `parts` partial products, plus their biases) wait in shared memory for the
-// root mean squares.  q_every >= 1: the query's factor 1 + q_coef ln(floor((p + 1) / q_every) + 1).
-template <typename TC>
+// root mean squares.  q_every >= 1: the query's factor 1 + q_coef ln(floor((p + 1) / q_every) + 1).  VEC 4: head sizes, the cache's head
+// and the product's rows are multiples of 4.
+template <typename TC, int VEC>
 __global__ void __launch_bounds__(256)
 whole_norm_kv_write_kernel(const float* __restrict__ qkv, int parts, size_t part_stride, int ld, const float* __restrict__ bias,
                            const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, const int* __restrict__ positions,
                            float q_coef, int q_every, int nq, int nkv, int dim, int vdim, int D, const int* __restrict__ slot_mapping,
                            int page_size, int num_pages, TC* __restrict__ k_cache, TC* __restrict__ v_cache, TC* __restrict__ q_out) {
-  extern __shared__ float wn_x[];                                    // [(nq + nkv) * dim]
+  extern __shared__ __align__(16) float wn_x[];                      // [(nq + nkv) * dim]
   __shared__ float red[33];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, tid = threadIdx.x;
+  const int t = blockIdx.x, step = blockDim.x * VEC, first = threadIdx.x * VEC;
   const float* row = qkv + (size_t)t * ld;
   auto value = [&](int c) {
-    float v = row[c];
-    for (int p = 1; p < parts; ++p) v += row[p * part_stride + c];
-    return bias != nullptr ? v + bias[c] : v;
+    WnVec<VEC> v = wn_load<VEC>(row + c);
+    for (int p = 1; p < parts; ++p) {
+      const WnVec<VEC> w = wn_load<VEC>(row + p * part_stride + c);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v.v[i] += w.v[i];
+    }
+    if (bias != nullptr) {
+      const WnVec<VEC> w = wn_load<VEC>(bias + c);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v.v[i] += w.v[i];
+    }
+    return v;
+  };
+  // channels c .. of x times a factor and their gains, zeros beyond the head's own
+  auto scaled = [&](const float* x, const float* gain, float f, int c, bool in) {
+    WnVec<VEC> r = {};
+    if (in) {
+      const WnVec<VEC> a = wn_load<VEC>(x + c), g = wn_load<VEC>(gain + c);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) r.v[i] = a.v[i] * f * g.v[i];
+    }
+    return r;
   };
   int slot = -1;
   if (slot_mapping != nullptr) {
@@ -105,28 +148,31 @@ whole_norm_kv_write_kernel(const float* __restrict__ qkv, int parts, size_t part
   }
   const int Q = nq * dim, K = slot >= 0 ? nkv * dim : 0;
   float sq = 0.f, sk = 0.f;
-  for (int c = tid; c < Q + K; c += blockDim.x) {
-    const float v = value(c);
-    wn_x[c] = v;
-    if (c < Q) sq = fmaf(v, v, sq);
-    else sk = fmaf(v, v, sk);
+  for (int c = first; c < Q + K; c += step) {
+    const WnVec<VEC> v = value(c);
+    wn_store<VEC>(wn_x + c, v);
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s = fmaf(v.v[i], v.v[i], s);
+    if (c < Q) sq += s;
+    else sk += s;
   }
   sq = block_sum(sq, red);
   float qi = 1.0f / sqrtf(sq / (float)Q + eps);
   if (q_coef != 0.f) qi *= 1.0f + q_coef * logf((float)((positions[t] + 1) / q_every) + 1.0f);
   TC* q = q_out + (size_t)t * nq * D;
-  for (int e = tid; e < nq * D; e += blockDim.x) {
-    const int h = e / D, d = e - h * D, c = h * dim + d;
-    q[e] = from_f32<TC>(d < dim ? wn_x[c] * qi * q_gain[c] : 0.f);
+  for (int e = first; e < nq * D; e += step) {
+    const int h = e / D, d = e - h * D;
+    wn_store<VEC>(q + e, scaled(wn_x, q_gain, qi, h * dim + d, d < dim));
   }
   if (slot < 0) return;                                              // (the whole CTA: no place to write to)
   sk = block_sum(sk, red);
   const float ki = 1.0f / sqrtf(sk / (float)(nkv * dim) + eps);
   const size_t head = (size_t)page_size * D, base = (size_t)(slot / page_size) * nkv * head + (size_t)(slot % page_size) * D;
-  for (int e = tid; e < nkv * D; e += blockDim.x) {
-    const int h = e / D, d = e - h * D, c = h * dim + d;
-    k_cache[base + h * head + d] = from_f32<TC>(d < dim ? wn_x[Q + c] * ki * k_gain[c] : 0.f);
-    v_cache[base + h * head + d] = from_f32<TC>(d < vdim ? value(Q + nkv * dim + h * vdim + d) : 0.f);
+  for (int e = first; e < nkv * D; e += step) {
+    const int h = e / D, d = e - h * D;
+    wn_store<VEC>(k_cache + base + h * head + d, scaled(wn_x + Q, k_gain, ki, h * dim + d, d < dim));
+    wn_store<VEC>(v_cache + base + h * head + d, d < vdim ? value(Q + nkv * dim + h * vdim + d) : WnVec<VEC>{});
   }
 }
 
@@ -395,22 +441,24 @@ SLLM_EXPORT int sllm_whole_norm_kv_write(const float* qkv, int parts, size_t par
   const size_t smem = (size_t)(nq + nkv) * dim * sizeof(float);
   SLLM_REQUIRE(smem <= 200 * 1024, "whole_norm: %d channels of queries and keys do not fit the shared memory", (nq + nkv) * dim);
   if (T == 0) return SLLM_OK;
-#define LAUNCH(TC)                                                                                                                         \
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && D % 4 == 0 && ld % 4 == 0 && part_stride % 4 == 0 &&
+                   (((uintptr_t)qkv | (uintptr_t)bias | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)q_out) & 15) == 0;
+#define LAUNCH(TC, VEC)                                                                                                                    \
   do {                                                                                                                                     \
     static size_t allowed = 48 * 1024;                                                                                                     \
     if (smem > allowed) {                                                                                                                  \
-      if (cudaFuncSetAttribute(whole_norm_kv_write_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {   \
+      if (cudaFuncSetAttribute(whole_norm_kv_write_kernel<TC, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) { \
         cudaGetLastError();                                                                                                                \
         set_error("whole_norm: the kernel's shared memory could not be raised");                                                           \
         return SLLM_ERR_LAUNCH;                                                                                                            \
       }                                                                                                                                    \
       allowed = smem;                                                                                                                      \
     }                                                                                                                                      \
-    launch_kernel(whole_norm_kv_write_kernel<TC>, (unsigned)T, 256, smem, stream, qkv, parts, part_stride, ld, bias, q_gain, k_gain, eps,    \
+    launch_kernel(whole_norm_kv_write_kernel<TC, VEC>, (unsigned)T, 256, smem, stream, qkv, parts, part_stride, ld, bias, q_gain, k_gain, eps, \
                   positions, q_coef, q_every, nq, nkv, dim, vdim, D, slot_mapping, page_size, num_pages, (TC*)k_cache, (TC*)v_cache, (TC*)q_out); \
   } while (0)
-  if (cache_dtype == SLLM_F32) LAUNCH(float);
-  else if (cache_dtype == SLLM_BF16) LAUNCH(__nv_bfloat16);
+  if (cache_dtype == SLLM_F32) { if (vec) LAUNCH(float, 4); else LAUNCH(float, 1); }
+  else if (cache_dtype == SLLM_BF16) { if (vec) LAUNCH(__nv_bfloat16, 4); else LAUNCH(__nv_bfloat16, 1); }
   else SLLM_REQUIRE(false, "whole_norm: unknown dtype %d", cache_dtype);
 #undef LAUNCH
   return launch_status("whole_norm_kv_write");

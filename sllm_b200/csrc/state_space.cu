@@ -305,8 +305,9 @@ static int launch_ssd(const SsdParams& p, int chunks, int runs, cudaStream_t str
   return launch_status("state_space_chunked");
 }
 
-template <typename TO>
-__global__ void __launch_bounds__(256)
+// VEC channels a thread at a time; the gated row waits in shared memory for its root mean square
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(512)
 gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, int ldg, int off_g, const float* __restrict__ gain, float eps,
                         int groups, TO* __restrict__ out, int n) {
   extern __shared__ __align__(16) float gg_v[];          // [n / groups]
@@ -314,17 +315,34 @@ gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ g
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x / groups, part = blockIdx.x % groups, size = n / groups;
-  const size_t base = (size_t)t * n + (size_t)part * size;
+  const float* x = y + (size_t)t * n + (size_t)part * size;
   const float* z = gate + (size_t)t * ldg + off_g + part * size;
+  TO* o = out + (size_t)t * n + (size_t)part * size;
+  gain += part * size;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < size; i += blockDim.x) {
-    const float g = z[i], v = y[base + i] * (g / (1.0f + expf(-g)));
-    gg_v[i] = v;
-    ss = fmaf(v, v, ss);
+  for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {
+    if constexpr (VEC == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(x + i), g = *reinterpret_cast<const float4*>(z + i);
+      const float4 v = make_float4(a.x * rc_silu<TO>(g.x), a.y * rc_silu<TO>(g.y), a.z * rc_silu<TO>(g.z), a.w * rc_silu<TO>(g.w));
+      *reinterpret_cast<float4*>(gg_v + i) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    } else {
+      const float v = x[i] * rc_silu<TO>(z[i]);
+      gg_v[i] = v;
+      ss = fmaf(v, v, ss);
+    }
   }
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)size + eps);
-  for (int i = threadIdx.x; i < size; i += blockDim.x) out[base + i] = from_f32<TO>(gg_v[i] * inv * gain[part * size + i]);
+  for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {      // (each thread reads what it wrote itself)
+    if constexpr (VEC == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(gg_v + i), w = *reinterpret_cast<const float4*>(gain + i);
+      const float r[4] = {v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w};
+      rc_store4(o + i, r);
+    } else {
+      o[i] = from_f32<TO>(gg_v[i] * inv * gain[i]);
+    }
+  }
 }
 
 }  // namespace sllm
@@ -367,15 +385,18 @@ SLLM_EXPORT int sllm_gated_group_norm(const float* y, const float* gate, int ldg
   SLLM_REQUIRE(smem <= 200 * 1024, "gated_group_norm: parts of %d channels do not fit the shared memory", n / groups);
   if (T == 0) return SLLM_OK;
   const unsigned blocks = (unsigned)T * (unsigned)groups;
-  const int threads = n / groups >= 256 ? 256 : (n / groups + 31) / 32 * 32;
-  static size_t allowed_f = 48 * 1024, allowed_b = 48 * 1024;
-  if (out_dtype == SLLM_F32) {
-    if (int rc = rc_smem(gated_group_norm_kernel<float>, smem, allowed_f)) return rc;
-    launch_kernel(gated_group_norm_kernel<float>, blocks, threads, smem, stream, y, gate, ldg, off_g, gain, eps, groups, (float*)out, n);
-  } else if (out_dtype == SLLM_BF16) {
-    if (int rc = rc_smem(gated_group_norm_kernel<__nv_bfloat16>, smem, allowed_b)) return rc;
-    launch_kernel(gated_group_norm_kernel<__nv_bfloat16>, blocks, threads, smem, stream, y, gate, ldg, off_g, gain, eps, groups, (__nv_bfloat16*)out, n);
-  } else
-    SLLM_REQUIRE(false, "gated_group_norm: unknown dtype %d", out_dtype);
-  return launch_status("gated_group_norm");
+  const int size = n / groups;
+  const bool vec = size % 4 == 0 && ldg % 4 == 0 && off_g % 4 == 0 && (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out) & 15) == 0;
+  const int per = vec ? size / 4 : size, threads = per >= 512 ? 512 : (per + 31) / 32 * 32;
+#define GG(TO_, VEC_)                                                                                                                        \
+  do {                                                                                                                                       \
+    static size_t allowed = 48 * 1024;                                                                                                       \
+    if (int rc = rc_smem(gated_group_norm_kernel<TO_, VEC_>, smem, allowed)) return rc;                                                      \
+    launch_kernel(gated_group_norm_kernel<TO_, VEC_>, blocks, threads, smem, stream, y, gate, ldg, off_g, gain, eps, groups, (TO_*)out, n);   \
+    return launch_status("gated_group_norm");                                                                                                \
+  } while (0)
+  if (out_dtype == SLLM_F32) { if (vec) GG(float, 4); else GG(float, 1); }
+  if (out_dtype == SLLM_BF16) { if (vec) GG(__nv_bfloat16, 4); else GG(__nv_bfloat16, 1); }
+#undef GG
+  SLLM_REQUIRE(false, "gated_group_norm: unknown dtype %d", out_dtype);
 }
