@@ -2,7 +2,8 @@
 // vector per token, and only that vector is cached.
 //
 //   * latent_write: the latent of each new token (columns of a float32 product) over its root mean square,
-//     times a gain, written to the token's place in the paged cache in the cache's dtype.
+//     times a gain, written to the token's place in the paged cache in the cache's dtype.  Queries that go through a latent of
+//     their own have theirs normed by the same launch (or, where nothing is written, by norm_cols).
 //   * head_linear: a product per head, out[t, h, :] = W_h x[t, h, :], with W [H, dout, din].  It carries a
 //     head's query into the latent space (W_h = the head's key up-projection, transposed: the score of a
 //     query against a key is then its carried form against the cached latent) and the head's weighted sum
@@ -14,17 +15,32 @@
 
 namespace sllm {
 
+// dst[i] = x[i] / rms(x) * gain[i] by the whole CTA
+template <typename TO>
+__device__ __forceinline__ void norm_row(const float* __restrict__ x, int n, const float* __restrict__ gain, float eps, TO* __restrict__ dst, float* red) {
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f32<TO>(x[i] * inv * gain[i]);
+}
+
 // With `tail` > 0 the `tail` columns after the latent are one more key part that every head shares: not normed, its first
 // `rot` channels rotated by position (rotate-half layout), written behind the latent; rows of the cache are D wide,
 // zeros beyond rank + tail.
 template <typename TC>
 __global__ void latent_write_kernel(const float* __restrict__ proj, int ld, int off, int rank, const float* __restrict__ gain,
                                     float eps, const int* __restrict__ slot_mapping, TC* __restrict__ cache, int D, int tail,
-                                    int rot, const int* __restrict__ positions, const float* __restrict__ table, int max_pos) {
+                                    int rot, const int* __restrict__ positions, const float* __restrict__ table, int max_pos,
+                                    int q_off, int q_n, const float* __restrict__ q_gain, TC* __restrict__ q_out) {
   __shared__ float red[33];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
+  if (blockIdx.y == 1) {              // the queries' latent of the same row
+    norm_row(proj + (size_t)t * ld + q_off, q_n, q_gain, eps, q_out + (size_t)t * q_n, red);
+    return;
+  }
   const int slot = slot_mapping[t];
   const float* x = proj + (size_t)t * ld + off;
   float ss = 0.f;
@@ -206,13 +222,7 @@ __global__ void norm_cols_kernel(const float* __restrict__ x, int ld, int off, i
   __shared__ float red[33];
   pdl_launch_dependents();
   pdl_wait();
-  const float* row = x + (size_t)blockIdx.x * ld + off;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-  ss = block_sum(ss, red);
-  const float inv = 1.0f / sqrtf(ss / (float)n + eps);
-  TO* dst = out + (size_t)blockIdx.x * n;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f32<TO>(row[i] * inv * gain[i]);
+  norm_row(x + (size_t)blockIdx.x * ld + off, n, gain, eps, out + (size_t)blockIdx.x * n, red);
 }
 
 }  // namespace sllm
@@ -231,7 +241,8 @@ SLLM_EXPORT int sllm_norm_cols(const float* x, int ld, int off, int n, const flo
 
 SLLM_EXPORT int sllm_latent_rope_write(const float* proj, int ld, int off, int rank, int tail, int rot, const float* gain, float eps,
                                        const int* positions, const float* table, int max_pos, const int* slot_mapping, void* cache,
-                                       int cache_dtype, int D, int T, cudaStream_t stream) {
+                                       int cache_dtype, int D, int q_off, int q_n, const float* q_gain, void* q_out, int T, cudaStream_t stream) {
+  SLLM_REQUIRE(q_out == nullptr || (q_gain != nullptr && q_n > 0 && q_off >= 0 && q_off + q_n <= ld), "latent_write: the queries' latent in columns %d..%d of %d", q_off, q_off + q_n, ld);
   SLLM_REQUIRE(T >= 0 && rank > 0 && tail >= 0 && off >= 0 && off + rank + tail <= ld, "latent_write: columns %d..%d of %d", off,
                off + rank + tail, ld);
   SLLM_REQUIRE(D >= rank + tail, "latent_write: rows of %d do not hold %d + %d", D, rank, tail);
@@ -239,12 +250,13 @@ SLLM_EXPORT int sllm_latent_rope_write(const float* proj, int ld, int off, int r
   SLLM_REQUIRE(rot == 0 || (positions != nullptr && table != nullptr && max_pos > 0), "latent_write: rotary table missing");
   if (T == 0) return SLLM_OK;
   const int threads = rank >= 512 ? 256 : 128;
+  const dim3 grid((unsigned)T, q_out != nullptr ? 2 : 1);
   if (cache_dtype == SLLM_F32)
-    launch_kernel(latent_write_kernel<float>, T, threads, 0, stream, proj, ld, off, rank, gain, eps, slot_mapping, (float*)cache, D,
-                  tail, rot, positions, table, max_pos);
+    launch_kernel(latent_write_kernel<float>, grid, threads, 0, stream, proj, ld, off, rank, gain, eps, slot_mapping, (float*)cache, D,
+                  tail, rot, positions, table, max_pos, q_off, q_n, q_gain, (float*)q_out);
   else if (cache_dtype == SLLM_BF16)
-    launch_kernel(latent_write_kernel<__nv_bfloat16>, T, threads, 0, stream, proj, ld, off, rank, gain, eps, slot_mapping,
-                  (__nv_bfloat16*)cache, D, tail, rot, positions, table, max_pos);
+    launch_kernel(latent_write_kernel<__nv_bfloat16>, grid, threads, 0, stream, proj, ld, off, rank, gain, eps, slot_mapping,
+                  (__nv_bfloat16*)cache, D, tail, rot, positions, table, max_pos, q_off, q_n, q_gain, (__nv_bfloat16*)q_out);
   else
     SLLM_REQUIRE(false, "latent_write: unknown dtype %d", cache_dtype);
   return launch_status("latent_write");
@@ -252,8 +264,8 @@ SLLM_EXPORT int sllm_latent_rope_write(const float* proj, int ld, int off, int r
 
 SLLM_EXPORT int sllm_latent_write(const float* proj, int ld, int off, int rank, const float* gain, float eps,
                                   const int* slot_mapping, void* cache, int cache_dtype, int T, cudaStream_t stream) {
-  return sllm_latent_rope_write(proj, ld, off, rank, 0, 0, gain, eps, nullptr, nullptr, 0, slot_mapping, cache, cache_dtype, rank, T,
-                                stream);
+  return sllm_latent_rope_write(proj, ld, off, rank, 0, 0, gain, eps, nullptr, nullptr, 0, slot_mapping, cache, cache_dtype, rank,
+                                0, 0, nullptr, nullptr, T, stream);
 }
 
 // Heads `xstride` apart in x (>= din) and `ostride` apart in rows of `ldo` of the output (>= dout; what lies between is

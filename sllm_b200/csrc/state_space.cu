@@ -9,10 +9,12 @@
 //   S'  = exp(L_(n-1)) S + sum_s exp(L_(n-1) - L_s) dt_s B_s x_s^T
 //
 // and every exponent is at most zero.  Three kernels, everything but the passing on of S side by side over all chunks and heads:
-//   1. ssd_state  per (chunk, head): what the chunk adds to a state, to scratch, and its decay exp(L_(n-1));
+//   1. ssd_state  per (chunk, head): what the chunk adds to a state, to scratch, and its decay exp(L_(n-1)); per (chunk, group), as CTAs of
+//                 the same launch: the products C_t . B_s, which all heads of a group share, to scratch;
 //   2. ssd_scan   per (request, head, element): from the request's state slot through its chunks in order; scratch then holds the
 //                 state each chunk meets, the slot the portion's last state;
 //   3. ssd_out    per (chunk, head): y.
+// Where every request of a step brings one token, ssd_token is all there is: a CTA per (request, head) streams the state through its registers.
 // Heads share B and C in groups.  All arithmetic is float32 multiply-adds on the CUDA cores; a warp owns 16 rows of a product and all
 // its columns (retention.cu says how the operands lie).
 //
@@ -38,9 +40,11 @@ struct SsdParams {
   const int* run_first;        // [runs] ... its first chunk ...
   const int* run_count;        // [runs] ... and how many it has
   float* scratch;              // [chunks, H, dk, dv]
+  float* scores;               // [chunks, groups, RC, RC]: C_t . B_s at [t][s] (s <= t)
   float* keeps;                // [chunks, H]
   float* out;                  // [T, H * dv]
   int H, hdiv, dk, dv;         // hdiv: heads per group
+  int groups;
   int vec_bc, vec_x;           // B and C / x and the output lie in whole 16-byte pieces
 };
 
@@ -67,7 +71,48 @@ __device__ __forceinline__ void ssd_steps(const SsdParams& p, int h, int t0, int
   __syncthreads();
 }
 
-// grid (chunks, H), 2 DK threads: a warp owns 16 of the state's rows
+// The products C_t . B_s of one chunk and group by a CTA of THREADS threads: a lane has 1024 / THREADS tokens t and every sixteenth s.
+template <int DK, int THREADS>
+__device__ __forceinline__ void ssd_scores(const SsdParams& p, float* sm, int chunk, int grp) {
+  constexpr int LD = DK + 4, R = RC * 16 / THREADS;
+  float* cs = sm;                      // [RC][LD]
+  float* bs = sm + RC * LD;            // [RC][LD]
+  const int t0 = p.chunk_t0[chunk], n = p.chunk_n[chunk];
+  const float* row0 = p.xbc + (size_t)t0 * p.ldx;
+  load_block<RC, DK, LD>(cs, row0 + p.off_c + grp * p.dk, p.ldx, n, p.dk, p.vec_bc != 0);
+  load_block<RC, DK, LD>(bs, row0 + p.off_b + grp * p.dk, p.ldx, n, p.dk, p.vec_bc != 0);
+  asm volatile("cp.async.wait_group 0;\n" ::);
+  __syncthreads();
+  const int row = (int)(threadIdx.x >> 4) * R, l16 = threadIdx.x & 15;
+  const int last_c = (2 * R * (int)(threadIdx.x >> 5) + 2 * R - 1) / 16;      // the block of 16 tokens that holds the warp's last
+  float sc[R][4];
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) sc[r][c] = 0.f;
+#pragma unroll 2
+  for (int k = 0; k < DK; k += 4) {
+    float4 a[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) a[r] = *reinterpret_cast<const float4*>(cs + (row + r) * LD + k);
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      if (c > last_c) break;           // (whole warps)
+      const float4 b = *reinterpret_cast<const float4*>(bs + (l16 + 16 * c) * LD + k);
+#pragma unroll
+      for (int r = 0; r < R; ++r)
+        sc[r][c] = fmaf(a[r].w, b.w, fmaf(a[r].z, b.z, fmaf(a[r].y, b.y, fmaf(a[r].x, b.x, sc[r][c]))));
+    }
+  }
+  pdl_launch_dependents();
+  float* out = p.scores + ((size_t)chunk * p.groups + grp) * RC * RC;
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) out[(row + r) * RC + l16 + 16 * c] = sc[r][c];
+}
+
+// grid (chunks, H + groups), 2 DK threads: a warp owns 16 of the state's rows; the last `groups` rows of CTAs make the scores
 template <int DK, int DV>
 __global__ void __launch_bounds__(2 * DK) ssd_state_kernel(const SsdParams p) {
   extern __shared__ __align__(16) float rc_sm[];
@@ -77,6 +122,10 @@ __global__ void __launch_bounds__(2 * DK) ssd_state_kernel(const SsdParams p) {
   float* L_s = dt_s + RC;              // [RC]
   pdl_wait();
   const int chunk = blockIdx.x, h = blockIdx.y;
+  if (h >= p.H) {
+    ssd_scores<DK, 2 * DK>(p, rc_sm, chunk, h - p.H);
+    return;
+  }
   const int t0 = p.chunk_t0[chunk], n = p.chunk_n[chunk];
   const float* row0 = p.xbc + (size_t)t0 * p.ldx;
   load_block<RC, DK, DK>(ks, row0 + p.off_b + (h / p.hdiv) * p.dk, p.ldx, n, p.dk, p.vec_bc != 0);
@@ -171,11 +220,11 @@ __global__ void __launch_bounds__(RC_SCAN_THREADS) ssd_scan_kernel(const SsdPara
 }
 
 template <int DK, int DV> struct SsdOutSmem {
-  static constexpr int LQ = DK + 4, LKV = (DK > DV ? DK : DV) + 4;      // row strides: a multiple of 4 that walks the banks
-  static constexpr int Q = RC * LQ;                                      // C; then, row by row, the warps' scores
-  static constexpr int KV = RC * LKV;                                    // B, then x
+  static constexpr int LQ = DK + 4, LX = DV + 4;                         // row strides: a multiple of 4 that walks the banks
+  static constexpr int Q = RC * LQ;                                      // C; then, row by row, the warps' weighted scores
+  static constexpr int X = RC * LX;
   static constexpr int S = 2 * RC_SLICE * DV;                            // two slices of the state
-  static constexpr int BYTES = (Q + KV + S + 2 * RC + 4) * 4;
+  static constexpr int BYTES = (Q + X + S + 2 * RC + 4) * 4;
 };
 
 // grid (chunks, H)
@@ -184,8 +233,8 @@ __global__ void __launch_bounds__(RC_OUT_THREADS) ssd_out_kernel(const SsdParams
   using L = SsdOutSmem<DK, DV>;
   extern __shared__ __align__(16) float rc_sm[];
   float* qs = rc_sm;
-  float* kv = qs + L::Q;
-  float* ss = kv + L::KV;
+  float* xs = qs + L::Q;
+  float* ss = xs + L::X;
   float* dt_s = ss + L::S;             // [RC]
   float* L_s = dt_s + RC;              // [RC]
   constexpr int TN = DV / 16, SLICES = DK / RC_SLICE;
@@ -202,40 +251,23 @@ __global__ void __launch_bounds__(RC_OUT_THREADS) ssd_out_kernel(const SsdParams
                                  p.dk - sl * RC_SLICE, p.dv, vec_s);
   };
   load_block<RC, DK, L::LQ>(qs, row0 + p.off_c + grp * p.dk, p.ldx, n, p.dk, p.vec_bc != 0);
-  load_block<RC, DK, L::LKV>(kv, row0 + p.off_b + grp * p.dk, p.ldx, n, p.dk, p.vec_bc != 0);
   load_slice(0);
   load_slice(1);                       // (SLICES >= 2)
-  ssd_steps(p, h, t0, n, dt_s, L_s, L_s + RC);
-  asm volatile("cp.async.wait_group 2;\n" ::);
-  __syncthreads();                     // B and C have landed
-  // scores of the lane's 8 tokens against tokens l16 + 16 c, c up to the warp's own 16 tokens
+  load_block<RC, DV, L::LX>(xs, row0 + h * p.dv, p.ldx, n, p.dv, p.vec_x != 0);
+  // the scores of the lane's 8 tokens against tokens l16 + 16 c, c up to the warp's own 16 tokens
   float sc[8][4];
+  const float* scores = p.scores + ((size_t)chunk * p.groups + grp) * RC * RC;
 #pragma unroll
-  for (int r = 0; r < 8; ++r)
+  for (int c = 0; c < 4; ++c)
 #pragma unroll
-    for (int c = 0; c < 4; ++c) sc[r][c] = 0.f;
-#pragma unroll 1
-  for (int k = 0; k < DK; k += 4) {
-    float4 a[8];
-#pragma unroll
-    for (int r = 0; r < 8; ++r) a[r] = *reinterpret_cast<const float4*>(qs + (row + r) * L::LQ + k);
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      if (c > warp) break;             // (whole warps)
-      const float4 b = *reinterpret_cast<const float4*>(kv + (l16 + 16 * c) * L::LKV + k);
-#pragma unroll
-      for (int r = 0; r < 8; ++r)
-        sc[r][c] = fmaf(a[r].w, b.w, fmaf(a[r].z, b.z, fmaf(a[r].y, b.y, fmaf(a[r].x, b.x, sc[r][c]))));
-    }
-  }
-  __syncthreads();                     // B is read: its place takes x
-  load_block<RC, DV, L::LKV>(kv, row0 + h * p.dv, p.ldx, n, p.dv, p.vec_x != 0);
+    for (int r = 0; r < 8; ++r) sc[r][c] = c <= warp ? scores[(row + r) * RC + l16 + 16 * c] : 0.f;
+  ssd_steps(p, h, t0, n, dt_s, L_s, L_s + RC);
   float acc[8][TN];
 #pragma unroll
   for (int r = 0; r < 8; ++r)
 #pragma unroll
     for (int c = 0; c < TN; ++c) acc[r][c] = 0.f;
-  // groups in flight by age: slice 0, slice 1, x, slice 2, slice 3
+  // groups in flight by age: C, slice 0, slice 1, x, slice 2, slice 3
 #pragma unroll
   for (int sl = 0; sl < SLICES; ++sl) {
     if (sl == 0) asm volatile("cp.async.wait_group 2;\n" ::);
@@ -266,7 +298,7 @@ __global__ void __launch_bounds__(RC_OUT_THREADS) ssd_out_kernel(const SsdParams
   }
   asm volatile("cp.async.wait_group 0;\n" ::);
   __syncthreads();                     // x has landed
-  rows_times_block<L::LQ, L::LKV, TN>(acc, qs + row * L::LQ, kv, 16 * (warp + 1));
+  rows_times_block<L::LQ, L::LX, TN>(acc, qs + row * L::LQ, xs, 16 * (warp + 1));
   pdl_launch_dependents();
   const float skip = p.skip[h];
 #pragma unroll
@@ -274,7 +306,7 @@ __global__ void __launch_bounds__(RC_OUT_THREADS) ssd_out_kernel(const SsdParams
     const int t = row + r;
     if (t >= n) break;
     float* o = p.out + ((size_t)(t0 + t) * p.H + h) * p.dv + 4 * l16;
-    const float* x = kv + t * L::LKV + 4 * l16;
+    const float* x = xs + t * L::LX + 4 * l16;
 #pragma unroll
     for (int q = 0; q < TN / 4; ++q) {
       if (4 * l16 + 64 * q >= p.dv) continue;
@@ -291,15 +323,80 @@ __global__ void __launch_bounds__(RC_OUT_THREADS) ssd_out_kernel(const SsdParams
   }
 }
 
+constexpr int ST_THREADS = 256;
+
+struct SsdTokenParams {
+  const float* xbc; const float* dtp;
+  int ldx, off_b, off_c, ldd, off_dt;
+  const float *dt_bias, *a_log, *skip;
+  float* state;                // [slots, H, N, dv]
+  const int* state_slots;      // [S]
+  float* out;                  // [S, H * dv]
+  int H, hdiv, N, dv;
+};
+
+// One token a request (request s's is row s): grid (S, H).  A thread holds PER pieces of four columns of the state, PER rows apart by
+// 256 / (dv / 4); all of them are in flight while the step size and the rows of B and C arrive.  dv / 4 divides 256.
+template <int PER>
+__global__ void __launch_bounds__(ST_THREADS) ssd_token_kernel(const SsdTokenParams p) {
+  __shared__ __align__(16) float4 part[ST_THREADS];
+  pdl_wait();
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int quads = p.dv >> 2, cq = tid % quads, r0 = tid / quads, rows = ST_THREADS / quads;
+  float4* S = reinterpret_cast<float4*>(p.state + ((size_t)p.state_slots[s] * p.H + h) * p.N * p.dv) + cq;
+  float4 v[PER];
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int r = r0 + k * rows;
+    v[k] = r < p.N ? S[(size_t)r * quads] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const float* row = p.xbc + (size_t)s * p.ldx;
+  const float* B = row + p.off_b + (h / p.hdiv) * p.N;
+  const float* C = row + p.off_c + (h / p.hdiv) * p.N;
+  const float dt = ssd_softplus(p.dtp[(size_t)s * p.ldd + p.off_dt + h] + p.dt_bias[h]), keep = expf(-expf(p.a_log[h]) * dt);
+  const float* xp = row + h * p.dv + 4 * cq;
+  const float4 x = make_float4(xp[0], xp[1], xp[2], xp[3]);
+  float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int r = r0 + k * rows;
+    if (r >= p.N) break;
+    const float b = B[r] * dt, c = C[r];
+    v[k].x = fmaf(b, x.x, keep * v[k].x); v[k].y = fmaf(b, x.y, keep * v[k].y);
+    v[k].z = fmaf(b, x.z, keep * v[k].z); v[k].w = fmaf(b, x.w, keep * v[k].w);
+    S[(size_t)r * quads] = v[k];
+    y.x = fmaf(c, v[k].x, y.x); y.y = fmaf(c, v[k].y, y.y); y.z = fmaf(c, v[k].z, y.z); y.w = fmaf(c, v[k].w, y.w);
+  }
+  pdl_launch_dependents();
+  part[tid] = y;
+  __syncthreads();
+  for (int half = rows >> 1; half > 0; half >>= 1) {      // (rows is a power of two)
+    if (r0 < half) {
+      const float4 o = part[tid + half * quads];
+      float4 m = part[tid];
+      m.x += o.x; m.y += o.y; m.z += o.z; m.w += o.w;
+      part[tid] = m;
+    }
+    __syncthreads();
+  }
+  if (r0 == 0) {
+    const float4 m = part[tid];
+    const float d = p.skip[h];
+    float* o = p.out + ((size_t)s * p.H + h) * p.dv + 4 * cq;
+    o[0] = fmaf(d, x.x, m.x); o[1] = fmaf(d, x.y, m.y); o[2] = fmaf(d, x.z, m.z); o[3] = fmaf(d, x.w, m.w);
+  }
+}
+
 template <int DK, int DV>
 static int launch_ssd(const SsdParams& p, int chunks, int runs, cudaStream_t stream) {
   static size_t allowed_state = 48 * 1024, allowed_out = 48 * 1024;      // (per instantiation)
-  constexpr size_t smem_state = (size_t)(RC * DK + RC * DV + 2 * RC + 4) * 4, smem_out = SsdOutSmem<DK, DV>::BYTES;
+  constexpr size_t for_state = (size_t)(RC * DK + RC * DV + 2 * RC + 4) * 4, for_scores = (size_t)2 * RC * (DK + 4) * 4;
+  constexpr size_t smem_state = for_state > for_scores ? for_state : for_scores, smem_out = SsdOutSmem<DK, DV>::BYTES;
   int rc = rc_smem(ssd_state_kernel<DK, DV>, smem_state, allowed_state);
   if (rc == SLLM_OK) rc = rc_smem(ssd_out_kernel<DK, DV>, smem_out, allowed_out);
   if (rc != SLLM_OK) return rc;
   const dim3 grid((unsigned)chunks, (unsigned)p.H);
-  launch_kernel(ssd_state_kernel<DK, DV>, grid, 2 * DK, smem_state, stream, p);
+  launch_kernel(ssd_state_kernel<DK, DV>, dim3((unsigned)chunks, (unsigned)(p.H + p.groups)), 2 * DK, smem_state, stream, p);
   launch_kernel(ssd_scan_kernel, dim3((unsigned)((p.dk * p.dv + RC_SCAN_THREADS - 1) / RC_SCAN_THREADS), (unsigned)p.H, (unsigned)runs), RC_SCAN_THREADS, 0, stream, p);
   launch_kernel(ssd_out_kernel<DK, DV>, grid, RC_OUT_THREADS, smem_out, stream, p);
   return launch_status("state_space_chunked");
@@ -353,21 +450,21 @@ SLLM_EXPORT int sllm_state_space_chunked_supports(int n, int dv) { return n >= 1
 
 // x | B | C in the columns of `xbc` [T, ldx] (x head by head, B and C group by group), step logits at columns off_dt + h of `dtp` [T, ldd].  `chunks` pieces
 // of at most 64 tokens that belong to `runs` requests (run_seq: rows of state_slots; run_first, run_count: their chunks, consecutive).
-// scratch: float32 [chunks, H, N, dv], keeps [chunks, H].  Rows of other requests are neither read nor written.
+// scratch: float32 [chunks, H, N, dv], scores [chunks, groups, 64, 64], keeps [chunks, H].  Rows of other requests are neither read nor written.
 SLLM_EXPORT int sllm_state_space_chunked(const float* xbc, int ldx, const float* dtp, int ldd, int off_dt, const float* dt_bias, const float* a_log,
                                          const float* skip, float* state, const int* state_slots, const int* chunk_t0, const int* chunk_n, int chunks,
-                                         const int* run_seq, const int* run_first, const int* run_count, int runs, float* scratch, float* keeps, float* out,
+                                         const int* run_seq, const int* run_first, const int* run_count, int runs, float* scratch, float* scores, float* keeps, float* out,
                                          int H, int groups, int N, int dv, cudaStream_t stream) {
-  SLLM_REQUIRE(chunks >= 0 && runs >= 0 && runs <= 65535 && H > 0 && H <= 65535 && groups > 0 && H % groups == 0, "state_space_chunked: bad sizes chunks=%d runs=%d H=%d groups=%d",
+  SLLM_REQUIRE(chunks >= 0 && runs >= 0 && runs <= 65535 && H > 0 && groups > 0 && H + groups <= 65535 && H % groups == 0, "state_space_chunked: bad sizes chunks=%d runs=%d H=%d groups=%d",
                chunks, runs, H, groups);
   SLLM_REQUIRE(sllm_state_space_chunked_supports(N, dv), "state_space_chunked: states of %d x %d are outside 1..128", N, dv);
   SLLM_REQUIRE(ldx >= H * dv + 2 * groups * N && off_dt >= 0 && off_dt + H <= ldd, "state_space_chunked: columns outside the inputs' %d and %d", ldx, ldd);
-  SLLM_REQUIRE(scratch != nullptr && keeps != nullptr && ((uintptr_t)scratch & 15) == 0, "state_space_chunked: scratch must be 16-byte aligned");
+  SLLM_REQUIRE(scratch != nullptr && scores != nullptr && keeps != nullptr && ((uintptr_t)scratch & 15) == 0, "state_space_chunked: scratch must be 16-byte aligned");
   if (chunks == 0 || runs == 0) return SLLM_OK;
   SsdParams p;
   p.xbc = xbc; p.ldx = ldx; p.off_b = H * dv; p.off_c = H * dv + groups * N; p.dtp = dtp; p.ldd = ldd; p.off_dt = off_dt;
   p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.state = state; p.state_slots = state_slots; p.chunk_t0 = chunk_t0; p.chunk_n = chunk_n;
-  p.run_seq = run_seq; p.run_first = run_first; p.run_count = run_count; p.scratch = scratch; p.keeps = keeps; p.out = out;
+  p.run_seq = run_seq; p.run_first = run_first; p.run_count = run_count; p.scratch = scratch; p.scores = scores; p.groups = groups; p.keeps = keeps; p.out = out;
   p.H = H; p.hdiv = H / groups; p.dk = N; p.dv = dv;
   const bool base16 = ((uintptr_t)xbc & 15) == 0 && ldx % 4 == 0;
   p.vec_bc = base16 && N % 4 == 0 && (H * dv) % 4 == 0;
@@ -376,6 +473,34 @@ SLLM_EXPORT int sllm_state_space_chunked(const float* xbc, int ldx, const float*
   if (N <= 64) return launch_ssd<64, 128>(p, chunks, runs, stream);
   if (dv <= 64) return launch_ssd<128, 64>(p, chunks, runs, stream);
   return launch_ssd<128, 128>(p, chunks, runs, stream);
+}
+
+SLLM_EXPORT int sllm_state_space_token_supports(int N, int dv) {
+  const int quads = dv / 4;
+  return N >= 1 && dv % 4 == 0 && quads >= 1 && quads <= ST_THREADS && (quads & (quads - 1)) == 0 && (N + ST_THREADS / quads - 1) / (ST_THREADS / quads) <= 32;
+}
+
+// One token a request: row s of `xbc` and `dtp` is request s's.
+SLLM_EXPORT int sllm_state_space_token(const float* xbc, int ldx, const float* dtp, int ldd, int off_dt, const float* dt_bias, const float* a_log,
+                                       const float* skip, float* state, const int* state_slots, float* out, int S, int H, int groups, int N, int dv,
+                                       cudaStream_t stream) {
+  SLLM_REQUIRE(S >= 0 && H > 0 && H <= 65535 && groups > 0 && H % groups == 0, "state_space_token: bad sizes S=%d H=%d groups=%d", S, H, groups);
+  SLLM_REQUIRE(sllm_state_space_token_supports(N, dv), "state_space_token: a state of %d x %d is not taken", N, dv);
+  SLLM_REQUIRE(ldx >= H * dv + 2 * groups * N && off_dt >= 0 && off_dt + H <= ldd, "state_space_token: columns outside the inputs' %d and %d", ldx, ldd);
+  SLLM_REQUIRE(((uintptr_t)state & 15) == 0, "state_space_token: the states must be 16-byte aligned");
+  if (S == 0) return SLLM_OK;
+  SsdTokenParams p;
+  p.xbc = xbc; p.dtp = dtp; p.ldx = ldx; p.off_b = H * dv; p.off_c = H * dv + groups * N; p.ldd = ldd; p.off_dt = off_dt;
+  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.state = state; p.state_slots = state_slots; p.out = out;
+  p.H = H; p.hdiv = H / groups; p.N = N; p.dv = dv;
+  const int rows = ST_THREADS / (dv / 4), per = (N + rows - 1) / rows;
+  const dim3 grid((unsigned)S, (unsigned)H);
+  if (per <= 2) launch_kernel(ssd_token_kernel<2>, grid, ST_THREADS, 0, stream, p);
+  else if (per <= 4) launch_kernel(ssd_token_kernel<4>, grid, ST_THREADS, 0, stream, p);
+  else if (per <= 8) launch_kernel(ssd_token_kernel<8>, grid, ST_THREADS, 0, stream, p);
+  else if (per <= 16) launch_kernel(ssd_token_kernel<16>, grid, ST_THREADS, 0, stream, p);
+  else launch_kernel(ssd_token_kernel<32>, grid, ST_THREADS, 0, stream, p);
+  return launch_status("state_space_token");
 }
 
 SLLM_EXPORT int sllm_gated_group_norm(const float* y, const float* gate, int ldg, int off_g, const float* gain, float eps, int groups, void* out,

@@ -711,8 +711,9 @@ def retention_gated(proj, offs, off_g: int, decay, table, rotary_dim: int, k_sca
 
 # ---- a state-space recurrence: one decay per token and head ------------------------------------------------
 
-# Portions of at least so many tokens run in chunks (0: none does); below, token by token.
-STATE_SPACE_CHUNKED_FROM = int(os.environ.get("SLLM_STATE_SPACE_CHUNKED_FROM", "96"))
+# Portions of at least so many tokens run in chunks (0: none does), shorter ones token by token.  In a graph, one portion at 64 heads of 128 x 64,
+# us: 64 tokens 20 token by token and 34 in chunks, 128 tokens 36 and 35, 256 tokens 68 and 45, 2,048 tokens 520 and 199; four of 512: 304 and 225.
+STATE_SPACE_CHUNKED_FROM = int(os.environ.get("SLLM_STATE_SPACE_CHUNKED_FROM", "128"))
 
 
 @functools.lru_cache(maxsize=4096)
@@ -746,9 +747,26 @@ def state_space_chunked(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, ste
     t0, _, count, C, seq, first, runs, R = chunks
     scratch = torch.empty((C, heads, n, dv), dtype=torch.float32, device=xbc.device)
     keeps = torch.empty((C, heads), dtype=torch.float32, device=xbc.device)
+    scores = torch.empty((C, groups, RETENTION_CHUNK, RETENTION_CHUNK), dtype=torch.float32, device=xbc.device)
     call("sllm_state_space_chunked", _p(xbc), xbc.shape[1], _p(proj), proj.shape[1], int(off_dt), _p(dt_bias), _p(a_log), _p(skip), _p(state),
-         _p(step.state_slots), _p(t0), _p(count), C, _p(seq), _p(first), _p(runs), R, _p(scratch), _p(keeps), _p(out), heads, groups, n, dv, _stream())
+         _p(step.state_slots), _p(t0), _p(count), C, _p(seq), _p(first), _p(runs), R, _p(scratch), _p(scores), _p(keeps), _p(out), heads, groups, n, dv, _stream())
     launches["own"] += 2           # the three kernels of the entry point
+
+
+@functools.lru_cache(maxsize=4096)
+def state_space_token_supports(n: int, dv: int) -> bool:
+    return bool(lib().sllm_state_space_token_supports(int(n), int(dv)))
+
+
+def state_space_token(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, heads: int, groups: int, n: int, dv: int) -> torch.Tensor:
+    """`state_space` for a step in which every request brings ONE token: the states stream through registers once."""
+    _state_space_args(xbc, proj, off_dt, dt_bias, a_log, skip, state, heads, groups, n, dv, "state_space_token")
+    if xbc.shape[0] != step.num_seqs:
+        raise KernelError(f"state_space_token: {xbc.shape[0]} tokens of {step.num_seqs} requests; this form takes one token a request")
+    out = torch.empty((xbc.shape[0], heads * dv), dtype=torch.float32, device=xbc.device)
+    call("sllm_state_space_token", _p(xbc), xbc.shape[1], _p(proj), proj.shape[1], int(off_dt), _p(dt_bias), _p(a_log), _p(skip), _p(state),
+         _p(step.state_slots), _p(out), step.num_seqs, heads, groups, n, dv, _stream())
+    return out
 
 
 def state_space(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, heads: int, groups: int, n: int, dv: int) -> torch.Tensor:
@@ -756,7 +774,10 @@ def state_space(xbc, proj, off_dt: int, dt_bias, a_log, skip, state, step, heads
     ``state`` (float32 ``[slots, heads, n, dv]``): S <- exp(-exp(a_log_h) dt) S + dt B x^T; y = S^T C + skip_h x, with dt = softplus of
     column ``off_dt + h`` of the float32 product ``proj`` plus ``dt_bias[h]``.  ``xbc`` float32 ``[T, heads*dv + 2*groups*n]`` holds x (head
     by head), B and C (group by group; head h uses group h // (heads / groups)).  Returns y float32 ``[T, heads*dv]``.  Long prompt
-    portions run in chunks (states of up to 128 x 128), single tokens and short portions token by token; a step may hold both."""
+    portions run in chunks (states of up to 128 x 128), short ones and single tokens beside them token by token; where every request
+    brings one token a form of its own streams the states."""
+    if xbc.shape[0] == step.num_seqs and state_space_token_supports(n, dv):
+        return state_space_token(xbc, proj, off_dt, dt_bias, a_log, skip, state, step, heads, groups, n, dv)
     chunks, longest = None, 0
     if STATE_SPACE_CHUNKED_FROM > 0 and step.max_q_len >= STATE_SPACE_CHUNKED_FROM and step.q_lens and state_space_chunked_supports(n, dv):
         key = ("chunks", STATE_SPACE_CHUNKED_FROM)
@@ -788,11 +809,14 @@ def gated_group_norm(y, gate, off_g: int, gain, eps: float, groups: int, out_dty
 # ---- latent attention ------------------------------------------------------------------------------------
 
 def latent_rope_write(proj, off: int, rank: int, tail: int, rotary_dim: int, gain, eps: float, positions, table, slot_mapping,
-                      cache) -> None:
+                      cache, queries=None):
     """`latent_write` with ``tail`` more columns behind the latent: a key part all heads share, not normed, its first
     ``rotary_dim`` channels rotated by position (``table`` float32 ``[positions, 2, rotary_dim/2]``).  Rows of the cache
-    ``[pages, 1, page_size, D]`` receive latent, tail and zeros up to D."""
+    ``[pages, 1, page_size, D]`` receive latent, tail and zeros up to D.  ``queries`` = (column, gain): also `norm_cols` of as many
+    columns as the gain has values, in the cache's dtype, by the same launch; they are returned."""
     _chk(proj, gain, positions, table, slot_mapping, cache)
+    q_off, q_gain = queries if queries is not None else (0, None)
+    q = torch.empty((proj.shape[0], q_gain.numel()), dtype=cache.dtype, device=proj.device) if q_gain is not None else None
     D = cache.shape[3]
     if proj.dtype != torch.float32 or cache.shape[1] != 1 or D < rank + tail:
         raise KernelError("latent_rope_write: a float32 product and a cache [pages, 1, page_size, D >= rank + tail]")
@@ -802,7 +826,9 @@ def latent_rope_write(proj, off: int, rank: int, tail: int, rotary_dim: int, gai
             raise KernelError("latent_rope_write: rotary table must be float32 [positions, 2, rotary_dim/2]")
         max_pos = table.shape[0]
     call("sllm_latent_rope_write", _p(proj), proj.shape[1], int(off), int(rank), int(tail), int(rotary_dim), _p(gain), float(eps),
-         _p(positions), _p(table), max_pos, _p(slot_mapping), _p(cache), _dt(cache), D, proj.shape[0], _stream())
+         _p(positions), _p(table), max_pos, _p(slot_mapping), _p(cache), _dt(cache), D, int(q_off),
+         q_gain.numel() if q_gain is not None else 0, _p(q_gain), _p(q), proj.shape[0], _stream())
+    return q
 
 
 def rope_cols_(out, ooff: int, ostride: int, x, xoff: int, xstride: int, n: int, rotary_dim: int, positions, table, heads: int) -> None:

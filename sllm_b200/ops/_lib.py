@@ -161,7 +161,7 @@ def _declare(L):
         "sllm_softcap": [c_void_p, ctypes.c_longlong, c_float, c_void_p],
         "sllm_plain_act": [c_void_p, c_int, c_int, c_size_t, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "sllm_latent_rope_write": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int,
-                                   c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
         "sllm_head_linear_strided": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
                                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_embed_streams": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p,
@@ -178,9 +178,12 @@ def _declare(L):
         "sllm_state_space_chunked_supports": [c_int, c_int],
         "sllm_state_space_chunked": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                      c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                     c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                                     c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "sllm_gated_group_norm": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_int,
                                   c_void_p],
+        "sllm_state_space_token_supports": [c_int, c_int],
+        "sllm_state_space_token": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                   c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     }
     for name, argtypes in sigs.items():
         fn = getattr(L, name)

@@ -136,15 +136,16 @@ class LatentAttention(Mixer):
         g = step.groups[cache.group]
         table = self.rotary.table if self.rotary is not None else None
         proj = self.inp(x, torch.float32)                                           # [T, H*(dim+rot_dim) (+ rank+rot_dim) (+ gate)] float32
-        q = proj
-        if self.q_rank:
-            q = self.uq(ops.norm_cols(proj, 0, self.q_rank, self.q_gain, self.eps, self.dtype), torch.float32)
+        cq = None
         if write_cache and not self.shared_kv:
-            if self.rot_dim:
-                ops.latent_rope_write(proj, self.off_c, self.rank, self.rot_dim, self.rot, self.c_gain, self.eps, step.positions,
-                                      table, g.slot_mapping, cache.k)
+            if self.rot_dim or self.q_rank:
+                cq = ops.latent_rope_write(proj, self.off_c, self.rank, self.rot_dim, self.rot, self.c_gain, self.eps, step.positions,
+                                           table, g.slot_mapping, cache.k, queries=(0, self.q_gain) if self.q_rank else None)
             else:
                 ops.latent_write(proj, self.off_c, self.rank, self.c_gain, self.eps, g.slot_mapping, cache.k)
+        q = proj
+        if self.q_rank:
+            q = self.uq(cq if cq is not None else ops.norm_cols(proj, 0, self.q_rank, self.q_gain, self.eps, self.dtype), torch.float32)
         # [T, H*D] queries: a head's unrotated part carried into the latent space, its rotated part behind it
         ql = ops.head_linear(q, 0, self.uk_t, self.dtype, xstride=self.qdim, ostride=self.D)
         if self.D > self.rank:

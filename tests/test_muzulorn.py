@@ -453,6 +453,11 @@ def test_latent_attention_in_a_window(dev, H, dk, dr, dv, q_rank, rank, window, 
     lens = {0: 110, 1: 37}
     xs = {s: _bf16_exact({"x": rng.standard_normal((n, W))})["x"] for s, n in lens.items()}
     want = {s: plain.latent_attention(x, w, "m.", m, eps) for s, x in xs.items()}
+    if dtype == "float32":                          # the queries' norm alone (a layer that writes no latents of its own runs it so)
+        import sllm_b200.ops as ops
+        z = rng.standard_normal((5, q_rank + 9))
+        got = ops.norm_cols(_to(dev)(z), 4, q_rank, _to(dev)(w["m.dq.norm"]), eps, torch.float32).cpu().numpy()
+        np.testing.assert_allclose(got, plain.norm(z[:, 4:4 + q_rank], w["m.dq.norm"], eps), rtol=2e-5, atol=2e-5)
     if window is not None and window > 1:           # the edge matters here: one key more or less changes rows by more than the tolerance
         for other in (window - 1, window + 1):
             d = _relative(plain.latent_attention(xs[0], w, "m.", dict(m, mask={"size": other}), eps), want[0])

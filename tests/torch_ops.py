@@ -397,7 +397,7 @@ def _rotate(x, positions, table, rot):
     return torch.cat([u * c - v * sn, v * c + u * sn, x[..., rot:]], dim=-1)
 
 
-def latent_rope_write(proj, off, rank, tail, rotary_dim, gain, eps, positions, table, slot_mapping, cache):
+def latent_rope_write(proj, off, rank, tail, rotary_dim, gain, eps, positions, table, slot_mapping, cache, queries=None):
     x = proj[:, off:off + rank]
     c = x * (x.pow(2).mean(-1, keepdim=True) + eps).rsqrt() * gain
     row = torch.zeros((proj.shape[0], cache.shape[3]), dtype=torch.float32, device=proj.device)
@@ -407,6 +407,7 @@ def latent_rope_write(proj, off, rank, tail, rotary_dim, gain, eps, positions, t
     ok = slot_mapping >= 0
     slots = slot_mapping[ok].long()
     cache[slots // ps, 0, slots % ps, :] = row[ok].to(cache.dtype)
+    return norm_cols(proj, queries[0], queries[1].numel(), queries[1], eps, cache.dtype) if queries is not None else None
 
 
 def rope_cols_(out, ooff, ostride, x, xoff, xstride, n, rotary_dim, positions, table, heads):
