@@ -99,7 +99,7 @@ __device__ __forceinline__ void hc_out(__nv_bfloat16* p, const float (&v)[4]) {
 // NS > 0: that many streams, their channels and weights in registers; 0: `ns` streams (up to HC_MAX_STREAMS), weights in shared memory.
 // VEC channels a thread at a time.
 template <int NS, int VEC, typename TO>
-__global__ void __launch_bounds__(HC_THREADS)
+__global__ void __launch_bounds__(HC_THREADS, NS > 0 && NS <= 4 ? 3 : 1)
 streams_step_kernel(float* __restrict__ streams, const float* __restrict__ term, int parts, size_t part_stride, const float* __restrict__ mix,
                     const float* __restrict__ share, const float* __restrict__ into, const float* __restrict__ gain, float eps,
                     const int* __restrict__ rows, TO* __restrict__ h, int T, int ns, int W) {
@@ -211,7 +211,8 @@ static int dispatch_streams_step(float* streams, const float* term, int parts, s
     case 4: HC_GO(4);
     case 6: HC_GO(6);
     case 8: HC_GO(8);
-    default: HC_GO(0);
+    default:               // (any other number, one channel at a time)
+      return launch_streams_step<0, 1, TO>(streams, term, parts, part_stride, mix, share, into, gain, eps, rows, h, R, T, ns, W, stream);
   }
 #undef HC_GO
 }

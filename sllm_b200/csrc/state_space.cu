@@ -186,32 +186,36 @@ __global__ void __launch_bounds__(2 * DK) ssd_state_kernel(const SsdParams p) {
   }
 }
 
-// grid (ceil(dk dv / 256), H, runs): an element of a state a thread, through the request's chunks in order
+// grid (ceil(dk dv / (256 VEC)), H, runs): VEC elements of a state a thread, through the request's chunks in order
+template <int VEC>
 __global__ void __launch_bounds__(RC_SCAN_THREADS) ssd_scan_kernel(const SsdParams p) {
+  struct alignas(4 * VEC) Piece { float v[VEC]; };
   pdl_wait();
   const int h = blockIdx.y, run = blockIdx.z, size = p.dk * p.dv;
-  const int e = blockIdx.x * RC_SCAN_THREADS + threadIdx.x;
+  const int e = (blockIdx.x * RC_SCAN_THREADS + threadIdx.x) * VEC;
   const int first = p.run_first[run], count = p.run_count[run];
   if (e < size) {
-    float* slot = p.state + ((size_t)p.state_slots[p.run_seq[run]] * p.H + h) * size + e;
+    Piece* slot = reinterpret_cast<Piece*>(p.state + ((size_t)p.state_slots[p.run_seq[run]] * p.H + h) * size + e);
     float* sc = p.scratch + ((size_t)first * p.H + h) * size + e;
     const float* keep = p.keeps + (size_t)first * p.H + h;
     const size_t step = (size_t)p.H * size;
-    float S = *slot;
-    constexpr int AHEAD = 16;
+    Piece S = *slot;
+    constexpr int AHEAD = 8;
     for (int c0 = 0; c0 < count; c0 += AHEAD) {
-      float kv[AHEAD], d[AHEAD];
+      Piece kv[AHEAD];
+      float d[AHEAD];
 #pragma unroll
       for (int q = 0; q < AHEAD; ++q)
         if (c0 + q < count) {
-          kv[q] = sc[(size_t)(c0 + q) * step];
+          kv[q] = *reinterpret_cast<const Piece*>(sc + (size_t)(c0 + q) * step);
           d[q] = keep[(size_t)(c0 + q) * p.H];
         }
 #pragma unroll
       for (int q = 0; q < AHEAD; ++q)
         if (c0 + q < count) {
-          sc[(size_t)(c0 + q) * step] = S;
-          S = fmaf(d[q], S, kv[q]);
+          *reinterpret_cast<Piece*>(sc + (size_t)(c0 + q) * step) = S;
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) S.v[i] = fmaf(d[q], S.v[i], kv[q].v[i]);
         }
     }
     *slot = S;
@@ -397,7 +401,12 @@ static int launch_ssd(const SsdParams& p, int chunks, int runs, cudaStream_t str
   if (rc != SLLM_OK) return rc;
   const dim3 grid((unsigned)chunks, (unsigned)p.H);
   launch_kernel(ssd_state_kernel<DK, DV>, dim3((unsigned)chunks, (unsigned)(p.H + p.groups)), 2 * DK, smem_state, stream, p);
-  launch_kernel(ssd_scan_kernel, dim3((unsigned)((p.dk * p.dv + RC_SCAN_THREADS - 1) / RC_SCAN_THREADS), (unsigned)p.H, (unsigned)runs), RC_SCAN_THREADS, 0, stream, p);
+  const int size = p.dk * p.dv;
+  const bool vec = size % 4 == 0 && (((uintptr_t)p.state | (uintptr_t)p.scratch) & 15) == 0;
+  const int per_cta = RC_SCAN_THREADS * (vec ? 4 : 1);
+  const dim3 scan((unsigned)((size + per_cta - 1) / per_cta), (unsigned)p.H, (unsigned)runs);
+  if (vec) launch_kernel(ssd_scan_kernel<4>, scan, RC_SCAN_THREADS, 0, stream, p);
+  else launch_kernel(ssd_scan_kernel<1>, scan, RC_SCAN_THREADS, 0, stream, p);
   launch_kernel(ssd_out_kernel<DK, DV>, grid, RC_OUT_THREADS, smem_out, stream, p);
   return launch_status("state_space_chunked");
 }
