@@ -520,7 +520,7 @@ def muzulorn_config(sz: dict) -> dict:
         else:
             layers.append({"type": "attention", "mixer": dict(attention, kv_from=i - 3) if kind else attention, "mlp": dense})
     return {"architecture": "Muzulorn", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "streams": 4, "residual_mult": 0.5,
-            "embedding": {"bigram": {"buckets": 65536, "mul_prev": 31, "mul_cur": 17}}, "layers": layers}
+            "embedding": {"bigram": {"buckets": 65536, "mul_prev": 37, "mul_cur": 19}}, "layers": layers}
 
 
 def design_run(args) -> dict:

@@ -105,7 +105,7 @@ MID = _config(1000, 352, 4, 0.6, [                 # a few hundred channels, no 
     _layer(_ssm(10, 48, 64, 2, 4, 2), _moe(8, 3, 96, 160)),
     _layer(_att(12, 3, 64, 64, 0.12, 48, 20.0, None, kv_from=0), _dense(512)),
     _layer(_lat(5, 48, 16, 64, 112, 80, 0.125, 45, (20000.0, 16)), _moe(8, 2, 96, 96)),
-], pairs=(5000, 31, 17))
+], pairs=(5000, 37, 19))
 CONFIGS = {"A": (CONFIG_A, 16), "B": (CONFIG_B, 16), "odd": (ODD, 8), "bare": (BARE, 4), "six": (SIX, 32), "mid": (MID, 16)}
 
 
@@ -260,7 +260,7 @@ def test_distance_buckets():
     """The whole-number form against the formula's logarithms (where those are not within rounding of a border), and on borders that are exact:
     with 16 buckets up to 128, distances 16, 32 and 64 each open the bucket that 8 times a power of sqrt 2 names."""
     from sllm_b200.parts.side_by_side import distance_buckets
-    for B, D in ((16, 120), (16, 128), (32, 1000), (8, 5), (2, 2), (2, 50), (64, 100), (6, 4000), (12, 7), (5, 30)):
+    for B, D in ((16, 111), (16, 128), (32, 1000), (8, 5), (2, 2), (2, 50), (64, 100), (6, 4000), (12, 7), (5, 30)):
         got = distance_buckets(B, D)
         assert len(got) == D + 1 and got[-1] == B - 1 and all(b - a in range(B) for a, b in zip(got, got[1:]))
         for n in range(D + 1):
@@ -299,7 +299,7 @@ def _attend(kf, vf, tables, seq, pos, q, ps, nq, nkv, scale, cap, bias, window=N
 
 
 @pytest.mark.parametrize("D,ps,dtype,nq,nkv,cap,n,spread", [
-    (27, 4, "float32", 3, 1, 4.0, 10, 2.0), (64, 16, "bfloat16", 8, 2, 6.0, 121, 2.0), (64, 16, "bfloat16", 24, 1, 30.0, 65, 1.0),
+    (27, 4, "float32", 3, 1, 4.0, 10, 2.0), (64, 16, "bfloat16", 8, 2, 6.0, 117, 2.0), (64, 16, "bfloat16", 24, 1, 30.0, 65, 1.0),
     (128, 32, "bfloat16", 6, 3, 0.0, 300, 1.0), (32, 8, "bfloat16", 2, 2, 7.0, 33, 2.0), (56, 16, "float32", 4, 4, 0.0, 64, 2.0),
     (16, 16, "bfloat16", 5, 1, 3.0, 1, 1.0), (128, 64, "bfloat16", 16, 2, 20.0, 17, 3.0), (64, 8, "bfloat16", 3, 3, 0.0, 2, 2.0),
     (80, 16, "bfloat16", 4, 2, 8.0, 900, 1.0), (64, 16, "bfloat16", 8, 2, 6.0, 90, 30.0)])
@@ -363,7 +363,7 @@ def test_a_bias_by_distance_over_a_context_cut_into_ranges(D, nq, nkv, q_len, ct
 
 
 @pytest.mark.parametrize("H,G,dk,dv,ps,dtype,buckets,limit,every", [
-    (6, 2, 24, 40, 4, "float32", 8, 30, 16), (3, 3, 10, 7, 8, "float32", 16, 120, 5), (8, 2, 64, 48, 16, "bfloat16", 16, 60, 32), (4, 1, 96, 128, 16, "bfloat16", 32, 90, 7),
+    (6, 2, 24, 40, 4, "float32", 8, 30, 16), (3, 3, 10, 7, 8, "float32", 16, 115, 5), (8, 2, 64, 48, 16, "bfloat16", 16, 60, 32), (4, 1, 96, 128, 16, "bfloat16", 32, 90, 7),
     (2, 2, 16, 16, 16, "bfloat16", 2, 9, 64), (1, 1, 33, 12, 16, "float32", 6, 200, 1), (4, 2, 144, 100, 16, "bfloat16", 12, 40, 20)])
 def test_attention_and_a_second_layer_on_the_same_keys_and_values(dev, H, G, dk, dv, ps, dtype, buckets, limit, every):
     """The whole mixer through its part: biases, norms over all of the query and all of the key, the query's factor across many of its steps,
